@@ -233,6 +233,53 @@ RB_EXPORT int rb_rmsnorm(void* out, int out_dtype, const float* x, const float* 
 }
 
 // ---------------------------------------------------------------- rotation + cache append
+// ---------------------------------------------------------------- tanh in place of a norm
+// out = w * tanh(alpha * x) + b, value by value.  VEC: four values a thread and turn.
+template <typename TO, bool VEC>
+__global__ void __launch_bounds__(256) tanh_norm_kernel(TO* __restrict__ out, const float* __restrict__ x,
+                                                        const float* __restrict__ w, const float* __restrict__ b,
+                                                        float alpha, int64_t n, int E) {
+  rb_pdl_launch_dependents();
+  rb_pdl_wait();
+  const int64_t first = (int64_t)blockIdx.x * blockDim.x + threadIdx.x, step = (int64_t)gridDim.x * blockDim.x;
+  if (VEC) {
+    const int E4 = E / 4;
+    for (int64_t i = first; i < n / 4; i += step) {
+      const int e = (int)(i % E4) * 4;
+      float v[4], ww[4], bb[4];
+      rb_load4(x + 4 * i, v);
+      rb_load4(w + e, ww);
+      rb_load4(b + e, bb);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] = fmaf(ww[j], tanhf(alpha * v[j]), bb[j]);
+      rb_store4(out + 4 * i, v);
+    }
+  } else {
+    for (int64_t i = first; i < n; i += step) {
+      const int e = (int)(i % E);
+      out[i] = rb_from_float<TO>(fmaf(w[e], tanhf(alpha * x[i]), b[e]));
+    }
+  }
+}
+
+RB_EXPORT int rb_tanh_norm(void* out, int out_dtype, const float* x, const float* w, const float* b, float alpha, int T, int E,
+                           cudaStream_t stream) {
+  if (T == 0) return 0;
+  RB_REQUIRE(T > 0 && E > 0, "rb_tanh_norm: bad sizes T=%d E=%d", T, E);
+  const int64_t n = (int64_t)T * E;
+  const bool vec = E % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)b % 16 == 0 &&
+                   (uintptr_t)out % 16 == 0;
+  const int64_t want = ((vec ? n / 4 : n) + 255) / 256, most = (int64_t)rb_sm_count() * 8;
+  const int blocks = (int)(want < most ? want : most);
+#define GO(TO, V) RB_LAUNCH("tanh_norm_kernel", (tanh_norm_kernel<TO, V>), blocks, 256, 0, stream, (TO*)out, x, w, b, alpha, n, E)
+  if (out_dtype == RB_F32) { if (vec) GO(float, true); else GO(float, false); }
+  else if (out_dtype == RB_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }
+  else RB_FAIL("rb_tanh_norm: unknown dtype %d", out_dtype);
+#undef GO
+  RB_CHECK_LAUNCH("rb_tanh_norm");
+  return 0;
+}
+
 // ---------------------------------------------------------------- layer norm with weight and bias
 // out = (x - mean) / sqrt(var + eps) * w + b, var the mean of the squared deviations; float32 sums, two passes over
 // the row (the second over the deviations).  One block per row.
@@ -1025,12 +1072,15 @@ RB_EXPORT int rb_head_gate(void* out, const void* a, const void* gate, int64_t l
   return 0;
 }
 
-// ---------------------------------------------------------------- gated activation with a limit
-// out = g' * sigmoid(alpha * g') * (u' + shift),  g' = min(g, limit),  u' = clamp(u, -limit, limit)
-// (limit <= 0: no limit).  alpha = 1, shift = 0 without a limit is SiLU(gate) * up.  Row layouts as rb_silu_mul.
+// ---------------------------------------------------------------- gated activations
+// kind 0: out = g' * sigmoid(alpha * g') * (u' + shift),  g' = min(g, limit),  u' = clamp(u, -limit, limit)
+//         (limit <= 0: no limit).  alpha = 1, shift = 0 without a limit is SiLU(gate) * up.
+// kind 1: out = gelu_tanh(g) * u, with gelu_tanh(g) = g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3)), which is
+//         g/2 * (1 + tanh(...)) written with one exponential
+// bias (or null): a number per column of gu, added first.  Row layouts as rb_silu_mul.
 template <typename T, typename TI>
 __global__ void gated_act_kernel(T* __restrict__ out, const TI* __restrict__ gu, int64_t n, int F, int64_t ld, int block,
-                                 float alpha, float limit, float shift) {
+                                 int kind, float alpha, float limit, float shift, const float* __restrict__ bias) {
   rb_pdl_launch_dependents();
   rb_pdl_wait();
   for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
@@ -1040,6 +1090,11 @@ __global__ void gated_act_kernel(T* __restrict__ out, const TI* __restrict__ gu,
     const int64_t at_u = block > 0 ? at_g + block : (int64_t)F + j;
     float g = rb_to_float<TI>(gu[t * ld + at_g]);
     float u = rb_to_float<TI>(gu[t * ld + at_u]);
+    if (bias != nullptr) { g += bias[at_g]; u += bias[at_u]; }
+    if (kind == 1) {
+      out[i] = rb_from_float<T>(g / (1.0f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u);
+      continue;
+    }
     if (limit > 0.f) {
       g = fminf(g, limit);
       u = fminf(fmaxf(u, -limit), limit);
@@ -1049,22 +1104,21 @@ __global__ void gated_act_kernel(T* __restrict__ out, const TI* __restrict__ gu,
 }
 
 RB_EXPORT int rb_gated_act(void* out, const void* gate_up, int dtype, int in_dtype, int T, int F, int64_t ld, int block,
-                           float alpha, float limit, float shift, cudaStream_t stream) {
+                           int kind, float alpha, float limit, float shift, const float* bias, cudaStream_t stream) {
   if (T == 0) return 0;
+  RB_REQUIRE(kind == 0 || kind == 1, "rb_gated_act: activation %d is not built (0: limited swish, 1: gelu in its tanh form)", kind);
   RB_REQUIRE(block >= 0 && (block == 0 ? ld >= 2 * (int64_t)F : ld >= ((int64_t)(F + block - 1) / block) * 2 * block),
              "rb_gated_act: rows of %lld values do not hold %d features in blocks of %d", (long long)ld, F, block);
   const int64_t n = (int64_t)T * F;
   const int threads = 256;
   const int64_t most = (int64_t)rb_sm_count() * 16;
   const int blocks = (int)((n + threads - 1) / threads < most ? (n + threads - 1) / threads : most);
-  if (dtype == RB_F32 && in_dtype == RB_F32)
-    RB_LAUNCH("gated_act_kernel", (gated_act_kernel<float, float>), blocks, threads, 0, stream, (float*)out, (const float*)gate_up, n, F, ld, block, alpha, limit, shift);
-  else if (dtype == RB_BF16 && in_dtype == RB_BF16)
-    RB_LAUNCH("gated_act_kernel", (gated_act_kernel<__nv_bfloat16, __nv_bfloat16>), blocks, threads, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, n, F, ld, block, alpha, limit, shift);
-  else if (dtype == RB_BF16 && in_dtype == RB_F32)
-    RB_LAUNCH("gated_act_kernel", (gated_act_kernel<__nv_bfloat16, float>), blocks, threads, 0, stream, (__nv_bfloat16*)out, (const float*)gate_up, n, F, ld, block, alpha, limit, shift);
-  else
-    RB_FAIL("rb_gated_act: unsupported dtypes %d <- %d", dtype, in_dtype);
+#define GO(TO, TI) RB_LAUNCH("gated_act_kernel", (gated_act_kernel<TO, TI>), blocks, threads, 0, stream, (TO*)out, (const TI*)gate_up, n, F, ld, block, kind, alpha, limit, shift, bias)
+  if (dtype == RB_F32 && in_dtype == RB_F32) GO(float, float);
+  else if (dtype == RB_BF16 && in_dtype == RB_BF16) GO(__nv_bfloat16, __nv_bfloat16);
+  else if (dtype == RB_BF16 && in_dtype == RB_F32) GO(__nv_bfloat16, float);
+  else RB_FAIL("rb_gated_act: unsupported dtypes %d <- %d", dtype, in_dtype);
+#undef GO
   RB_CHECK_LAUNCH("rb_gated_act");
   return 0;
 }

@@ -13,11 +13,25 @@ namespace {
 
 constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;  // 256 threads, 4x4 outputs each
 
+// What happens to a finished sum before it is stored or added (null: nothing): bias[n] is added, and the value is
+// multiplied by sigmoid(gate[row * ldg + z * gate_batch + n]), z the number of the product (a head).
+struct Tail {
+  const float* bias = nullptr;
+  const float* gate = nullptr;
+  int64_t ldg = 0;
+  int64_t gate_batch = 0;
+};
+__device__ __forceinline__ float finished(const Tail& tail, float v, int64_t row, int n, int64_t z) {
+  if (tail.bias != nullptr) v += tail.bias[n];
+  if (tail.gate != nullptr) v *= 1.0f / (1.0f + expf(-tail.gate[row * tail.ldg + z * tail.gate_batch + n]));
+  return v;
+}
+
 template <typename TA, typename TC>
 __global__ void __launch_bounds__(256) gemm_simple_kernel(TC* __restrict__ C, int64_t ldc,
                                                          const TA* __restrict__ A, int64_t lda,
                                                          const TA* __restrict__ W, int64_t ldw, int M, int N,
-                                                         int K, int accumulate, float alpha, int64_t batch_c,
+                                                         int K, int accumulate, float alpha, Tail tail, int64_t batch_c,
                                                          int64_t batch_a, int64_t batch_w) {
   rb_pdl_launch_dependents();
   rb_pdl_wait();
@@ -67,7 +81,7 @@ __global__ void __launch_bounds__(256) gemm_simple_kernel(TC* __restrict__ C, in
       const int gn = n0 + tx * TN + j;
       if (gn >= N) continue;
       TC* p = C + (int64_t)gm * ldc + gn;
-      float v = alpha == 1.0f ? acc[i][j] : acc[i][j] * alpha;
+      float v = finished(tail, alpha == 1.0f ? acc[i][j] : acc[i][j] * alpha, gm, gn, blockIdx.z);
       if (accumulate) v += rb_to_float<TC>(*p);
       *p = rb_from_float<TC>(v);
     }
@@ -83,7 +97,7 @@ constexpr int LM = 128, LN = 128, LK = 16;
 template <typename TA, typename TC>
 __global__ void __launch_bounds__(256) gemm_simple_large_kernel(TC* __restrict__ C, int64_t ldc, const TA* __restrict__ A,
                                                                int64_t lda, const TA* __restrict__ W, int64_t ldw, int M,
-                                                               int N, int K, int accumulate, float alpha, int64_t batch_c,
+                                                               int N, int K, int accumulate, float alpha, Tail tail, int64_t batch_c,
                                                                int64_t batch_a, int64_t batch_w) {
   rb_pdl_launch_dependents();
   rb_pdl_wait();
@@ -132,7 +146,7 @@ __global__ void __launch_bounds__(256) gemm_simple_large_kernel(TC* __restrict__
       const int gn = n0 + (j < 4 ? tx * 4 + j : 64 + tx * 4 + j - 4);
       if (gn >= N) continue;
       TC* p = C + (int64_t)gm * ldc + gn;
-      float v = alpha == 1.0f ? acc[i][j] : acc[i][j] * alpha;
+      float v = finished(tail, alpha == 1.0f ? acc[i][j] : acc[i][j] * alpha, gm, gn, blockIdx.z);
       if (accumulate) v += rb_to_float<TC>(*p);
       *p = rb_from_float<TC>(v);
     }
@@ -141,47 +155,87 @@ __global__ void __launch_bounds__(256) gemm_simple_large_kernel(TC* __restrict__
 
 // Few rows (a decode step) times one matrix per head: a warp makes one output of one head for up to eight rows at a
 // time, its lanes sharing K, so that the head's matrix is read once and 8 heads x N / 8 blocks are at work instead of
-// a few tiles.  float32 sums (a lane's share in ascending order, then the lanes' shares added up).
+// a few tiles.  float32 sums (a lane's share in ascending order, then the lanes' shares added up).  Head h's input
+// values start at column h * head_a of a row.  VEC: four values a load.
 constexpr int FEW_ROWS = 8;
-template <typename TA, typename TC>
+template <typename TA, typename TC, bool VEC>
 __global__ void __launch_bounds__(256) per_head_few_rows_kernel(TC* __restrict__ C, int64_t ldc, const TA* __restrict__ A,
-                                                               int64_t lda, const TA* __restrict__ W, int M, int N, int K) {
+                                                               int64_t lda, int head_a, const TA* __restrict__ W, int M,
+                                                               int N, int K, Tail tail) {
   rb_pdl_launch_dependents();
   rb_pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, n = blockIdx.x * 8 + warp;
   if (n >= N) return;
   const TA* w = W + ((int64_t)h * N + n) * K;
-  const TA* a = A + (int64_t)h * K;
+  const TA* a = A + (int64_t)h * head_a;
   for (int m0 = 0; m0 < M; m0 += FEW_ROWS) {
     float acc[FEW_ROWS];
 #pragma unroll
     for (int i = 0; i < FEW_ROWS; ++i) acc[i] = 0.f;
-    for (int k = lane; k < K; k += 32) {
-      const float wv = rb_to_float<TA>(w[k]);
+    if (VEC) {
+      for (int k = lane * 4; k < K; k += 128) {
+        float wv[4];
+        rb_load4(w + k, wv);
 #pragma unroll
-      for (int i = 0; i < FEW_ROWS; ++i)
-        if (m0 + i < M) acc[i] = fmaf(rb_to_float<TA>(a[(int64_t)(m0 + i) * lda + k]), wv, acc[i]);
+        for (int i = 0; i < FEW_ROWS; ++i) {
+          if (m0 + i < M) {
+            float av[4];
+            rb_load4(a + (int64_t)(m0 + i) * lda + k, av);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[i] = fmaf(av[j], wv[j], acc[i]);
+          }
+        }
+      }
+    } else {
+      for (int k = lane; k < K; k += 32) {
+        const float wv = rb_to_float<TA>(w[k]);
+#pragma unroll
+        for (int i = 0; i < FEW_ROWS; ++i)
+          if (m0 + i < M) acc[i] = fmaf(rb_to_float<TA>(a[(int64_t)(m0 + i) * lda + k]), wv, acc[i]);
+      }
     }
 #pragma unroll
     for (int i = 0; i < FEW_ROWS; ++i) {
       const float v = rb_warp_sum(acc[i]);
-      if (lane == 0 && m0 + i < M) C[(int64_t)(m0 + i) * ldc + (int64_t)h * N + n] = rb_from_float<TC>(v);
+      if (lane == 0 && m0 + i < M)
+        C[(int64_t)(m0 + i) * ldc + (int64_t)h * N + n] = rb_from_float<TC>(finished(tail, v, m0 + i, n, h));
     }
   }
 }
 
+thread_local Tail t_tail;          // of this thread's next call
+Tail take_tail() {
+  const Tail t = t_tail;
+  t_tail = Tail();
+  return t;
+}
+
 }  // namespace
 
-// C[m, h * N + n] = sum_k A[m, h * K + k] * W[h, n, k] for few rows m (any number is right; up to 16 is what it is for).
-RB_EXPORT int rb_per_head_few_rows(void* C, int64_t ldc, int c_dtype, const void* A, int64_t lda, const void* W, int a_dtype,
-                                   int M, int H, int N, int K, cudaStream_t stream) {
+// The next rb_gemm_simple, rb_gemm_simple_batched or rb_per_head_few_rows call of this thread adds bias[n] (float32, or
+// null) to every finished sum and multiplies it by sigmoid(gate[row * ldg + z * gate_batch + n]) (float32, or null; z: the
+// number of the product or head).
+RB_EXPORT int rb_gemm_simple_next(const float* bias, const float* gate, int64_t ldg, int64_t gate_batch) {
+  t_tail.bias = bias; t_tail.gate = gate; t_tail.ldg = ldg; t_tail.gate_batch = gate_batch;
+  return 0;
+}
+
+// C[m, h * N + n] = sum_k A[m, h * head_a + k] * W[h, n, k] for few rows m (any number is right; up to 16 is what it is for).
+RB_EXPORT int rb_per_head_few_rows(void* C, int64_t ldc, int c_dtype, const void* A, int64_t lda, int head_a, const void* W,
+                                   int a_dtype, int M, int H, int N, int K, cudaStream_t stream) {
+  const Tail tail = take_tail();
   if (M == 0 || N == 0 || H == 0) return 0;
-  RB_REQUIRE(M > 0 && N > 0 && K > 0 && H > 0 && H <= 65535, "rb_per_head_few_rows: bad sizes M=%d H=%d N=%d K=%d", M, H, N, K);
+  RB_REQUIRE(M > 0 && N > 0 && K > 0 && H > 0 && H <= 65535 && head_a >= K, "rb_per_head_few_rows: bad sizes M=%d H=%d N=%d K=%d (%d apart)",
+             M, H, N, K, head_a);
   const dim3 grid((N + 7) / 8, H);
+  const int elem = a_dtype == RB_F32 ? 4 : 2;
+  const bool vec = K % 4 == 0 && head_a % 4 == 0 && lda % 4 == 0 && (uintptr_t)A % (4 * elem) == 0 && (uintptr_t)W % (4 * elem) == 0;
 #define LAUNCH(TA, TC)                                                                                                  \
-  RB_LAUNCH("per_head_few_rows_kernel", (per_head_few_rows_kernel<TA, TC>), grid, 256, 0, stream, (TC*)C, ldc, (const TA*)A, \
-            lda, (const TA*)W, M, N, K)
+  do {                                                                                                                  \
+    if (vec) RB_LAUNCH("per_head_few_rows_kernel", (per_head_few_rows_kernel<TA, TC, true>), grid, 256, 0, stream, (TC*)C, ldc, (const TA*)A, lda, head_a, (const TA*)W, M, N, K, tail); \
+    else RB_LAUNCH("per_head_few_rows_kernel", (per_head_few_rows_kernel<TA, TC, false>), grid, 256, 0, stream, (TC*)C, ldc, (const TA*)A, lda, head_a, (const TA*)W, M, N, K, tail);    \
+  } while (0)
   if (a_dtype == RB_F32 && c_dtype == RB_F32) LAUNCH(float, float);
   else if (a_dtype == RB_BF16 && c_dtype == RB_F32) LAUNCH(__nv_bfloat16, float);
   else if (a_dtype == RB_BF16 && c_dtype == RB_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
@@ -199,6 +253,7 @@ RB_EXPORT int rb_gemm_simple_batched(void* C, int64_t ldc, int c_dtype, const vo
                                      int64_t ldw, int a_dtype, int M, int N, int K, int accumulate, float alpha,
                                      int n_batch, int64_t batch_c, int64_t batch_a, int64_t batch_w,
                                      cudaStream_t stream) {
+  const Tail tail = take_tail();
   if (M == 0 || N == 0 || n_batch == 0) return 0;
   RB_REQUIRE(M > 0 && N > 0 && K > 0, "rb_gemm_simple: bad sizes M=%d N=%d K=%d", M, N, K);
   if (M >= 256 && N >= LN) {
@@ -207,7 +262,7 @@ RB_EXPORT int rb_gemm_simple_batched(void* C, int64_t ldc, int c_dtype, const vo
     RB_REQUIRE(lgrid.y <= 65535 && n_batch >= 1 && n_batch <= 65535, "rb_gemm_simple: M=%d, %d products: too large for one launch", M, n_batch);
 #define LLAUNCH(TA, TC)                                                                                            \
   RB_LAUNCH("gemm_simple_large_kernel", (gemm_simple_large_kernel<TA, TC>), lgrid, 256, 0, stream, (TC*)C, ldc,     \
-            (const TA*)A, lda, (const TA*)W, ldw, M, N, K, accumulate, alpha, batch_c, batch_a, batch_w)
+            (const TA*)A, lda, (const TA*)W, ldw, M, N, K, accumulate, alpha, tail, batch_c, batch_a, batch_w)
     if (a_dtype == RB_F32 && c_dtype == RB_F32) LLAUNCH(float, float);
     else if (a_dtype == RB_BF16 && c_dtype == RB_F32) LLAUNCH(__nv_bfloat16, float);
     else if (a_dtype == RB_BF16 && c_dtype == RB_BF16) LLAUNCH(__nv_bfloat16, __nv_bfloat16);
@@ -220,7 +275,7 @@ RB_EXPORT int rb_gemm_simple_batched(void* C, int64_t ldc, int c_dtype, const vo
   RB_REQUIRE(grid.y <= 65535 && n_batch >= 1 && n_batch <= 65535, "rb_gemm_simple: M=%d, %d products: too large for one launch", M, n_batch);
 #define LAUNCH(TA, TC)                                                                                     \
   RB_LAUNCH("gemm_simple_kernel", (gemm_simple_kernel<TA, TC>), grid, 256, 0, stream, (TC*)C, ldc, (const TA*)A, \
-            lda, (const TA*)W, ldw, M, N, K, accumulate, alpha, batch_c, batch_a, batch_w)
+            lda, (const TA*)W, ldw, M, N, K, accumulate, alpha, tail, batch_c, batch_a, batch_w)
   if (a_dtype == RB_F32 && c_dtype == RB_F32) LAUNCH(float, float);
   else if (a_dtype == RB_BF16 && c_dtype == RB_F32) LAUNCH(__nv_bfloat16, float);
   else if (a_dtype == RB_BF16 && c_dtype == RB_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);

@@ -104,10 +104,18 @@ struct GemmParams {
   int64_t emit_ld;
   const float* emit_g;
   float* emit_ss;
+  // With emit_b the norm that follows is a tanh in place of a norm, which needs no sums: emit_xb is
+  // bfloat16(emit_g[column] * tanh(emit_alpha * C_new) + emit_b[column]), the finished rows, and emit_ss is not used.
+  const float* emit_b;
+  float emit_alpha;
   QkvTail qkv;        // EPI_QKV only
   // EPI_GATED: out = g' / (1 + e^(-act_alpha g')) * (u' + act_shift), g' = min(g, act_limit), u' = clamp(u, +-act_limit)
   // (act_limit <= 0: no limit).  1, 0, 0 is SiLU(gate) * up.
+  // act_kind 1: out = gelu_tanh(gate) * up instead.
   float act_alpha, act_limit, act_shift;
+  int act_kind;
+  // A number per row of W (float32, or null) that is added to the finished sums (before a gated activation).
+  const float* bias;
   // EPI_STORE: the stored value is max(v, 0)^2 instead of v (square_relu != 0).
   int square_relu;
   // Grouped rows (tile_group != nullptr; one product per CTA item, K whole): the rows of X are sorted into groups
@@ -117,6 +125,13 @@ struct GemmParams {
   // group's rows, and output columns are numbered within the group.
   const int* tile_group;
   int group_rows;
+  // One matrix per head (heads > 0; EPI_STORE, K whole): W holds `heads` matrices of n_out rows one below the other,
+  // head h reads columns h * head_x .. + K - 1 of X (what a box of X holds beyond them meets zeros in the box of W)
+  // and writes columns h * head_c .. + n_out - 1 of C.  gate (or null): the values are multiplied by
+  // sigmoid(gate[token * gate_ld + h * n_out + column]).
+  int heads, head_x, head_c;
+  const float* gate;
+  int64_t gate_ld;
 };
 
 __device__ __forceinline__ float stored_value(const GemmParams& p, float v) {
@@ -127,6 +142,8 @@ __device__ __forceinline__ float stored_value(const GemmParams& p, float v) {
 // The gated epilogue's value, with the hardware's exponential and reciprocal: their error (a few units of
 // float32) is far below the rounding to bfloat16 that follows.
 __device__ __forceinline__ float gated_value(const GemmParams& p, float g, float up) {
+  // gelu_tanh(g) = g/2 (1 + tanh(s)) = g / (1 + e^(-2 s)), s = sqrt(2/pi) (g + 0.044715 g^3)
+  if (p.act_kind == 1) return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * g * (1.0f + 0.044715f * g * g))) * up;
   if (p.act_limit > 0.f) {
     g = fminf(g, p.act_limit);
     up = fminf(fmaxf(up, -p.act_limit), p.act_limit);
@@ -139,7 +156,8 @@ __device__ __forceinline__ float gated_value(const GemmParams& p, float g, float
 // number `part` (teams first_team .. first_team + parts - 1, in the order of their k blocks).
 struct Piece {
   int n0, t0, kb_begin, nkb;
-  int w0;          // first row of W of the tile (n0, or n0 within the tile's group)
+  int w0;          // first row of W of the tile (n0, or n0 within the tile's group or head)
+  int x0, c0;      // columns of X and of C that the tile's head begins at (one matrix per head), else 0
   int w_tile, part, parts, first_team;
 };
 
@@ -273,6 +291,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       s.first_team = (int)(g_begin / p.sk_len);
       s.parts = (int)((g_end - 1) / p.sk_len) - s.first_team + 1;
       s.part = sk_team - s.first_team;
+      s.x0 = s.c0 = 0;
       return true;
     }
     const int item = first_item + li * item_stride;
@@ -289,6 +308,14 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       const int g = p.tile_group[tile % p.n_t_tiles];
       if (g < 0) s.nkb = 0;
       else s.w0 = g * p.group_rows + s.n0;
+    }
+    s.x0 = s.c0 = 0;
+    if (EPI == EPI_STORE && p.heads > 0) {
+      const int per_head = (p.n_out + BM - 1) / BM, h = s.w_tile / per_head;
+      s.n0 = (s.w_tile - h * per_head) * BM;
+      s.w0 = h * p.n_out + s.n0;
+      s.x0 = h * p.head_x;
+      s.c0 = h * p.head_c;
     }
     s.part = 0; s.parts = 1; s.first_team = 0;
     return true;
@@ -313,7 +340,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         rb_pdl_wait();
         for (int i = 0; i < early; ++i) {
           uint8_t* stage = smem + (size_t)i * STAGE_BYTES;
-          tma_load_2d(stage + W_TILE_BYTES, &tmX, (s.kb_begin + i) * BK, s.t0, &full_bar[i]);
+          tma_load_2d(stage + W_TILE_BYTES, &tmX, s.x0 + (s.kb_begin + i) * BK, s.t0, &full_bar[i]);
         }
       }
       for (int li = 0; ok && piece_at(li, s); ++li) {
@@ -328,7 +355,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           mbar_expect_tx(&full_bar[st], STAGE_BYTES);
           const int k = (s.kb_begin + i) * BK;
           tma_load_2d(stage, &tmW, k, s.w0, &full_bar[st]);
-          tma_load_2d(stage + W_TILE_BYTES, &tmX, k, s.t0, &full_bar[st]);
+          tma_load_2d(stage + W_TILE_BYTES, &tmX, s.x0 + k, s.t0, &full_bar[st]);
         }
       }
     }
@@ -394,6 +421,8 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       const int b = li % NBUF;
       const int n = n0 + row;                           // output column = weight row
       const bool n_ok = n < p.n_out;
+      // (a tile whose K is shared takes the bias with its first part)
+      const float bias_n = p.bias != nullptr && n_ok && s.part == 0 ? p.bias[n] : 0.f;
       // EPI_ADD without TMA: the values to add to do not depend on the accumulator.  They are fetched
       // one chunk ahead, the first chunk while the products of this item still run, so that the
       // epilogue waits for memory once per item and not once per chunk.
@@ -468,8 +497,8 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             OutT* dst = box + (low ? 0 : OUT_COLS) + quarter * 16 + (lane & 15);
 #pragma unroll
             for (int j = 0; j < 16; j += 2) {
-              const float mine = __uint_as_float(low ? r[j] : r[j + 1]);       // gate (low) or up (high) of my token
-              const float send = __uint_as_float(low ? r[j + 1] : r[j]);       // what the partner needs
+              const float mine = __uint_as_float(low ? r[j] : r[j + 1]) + bias_n;       // gate (low) or up (high) of my token
+              const float send = __uint_as_float(low ? r[j + 1] : r[j]) + bias_n;       // what the partner needs
               const float got = __shfl_xor_sync(0xffffffffu, send, 16);
               const float g = low ? mine : got, up = low ? got : mine;
               // silu(g) * up = g * up / (1 + e^-g), with the hardware's exponential and reciprocal: their
@@ -477,9 +506,17 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               store_out<OutT>(dst + j * OUT_COLS, gated_value(p, g, up));
             }
           } else {
+            float gate[16];
+            if (EPI == EPI_STORE && p.gate != nullptr) {
+              const int left = n_ok ? p.n_tokens - (t0 + c) : 0;
+              const float* src = p.gate + (int64_t)(t0 + c) * p.gate_ld + (s.w0 + row);
+#pragma unroll
+              for (int j = 0; j < 16; ++j) gate[j] = j < left ? src[(int64_t)j * p.gate_ld] : 0.f;
+            }
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
-              const float v = __uint_as_float(r[j]) * p.alpha;
+              float v = __uint_as_float(r[j]) * p.alpha + bias_n;
+              if (EPI == EPI_STORE && p.gate != nullptr) v = __fdividef(v, 1.0f + __expf(-gate[j]));
               store_out<OutT>(box + j * OUT_COLS + row, EPI == EPI_STORE ? stored_value(p, v) : v);
             }
           }
@@ -491,7 +528,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               if (!wait_for_count(finished, s.part, 4)) epi_fail = 1;     // noticed at the next piece; the results are void
               must_wait = false;
             }
-            tma_store_2d(&tmC, box, EPI == EPI_GATED ? n0 / 2 : n0, t0 + c, EPI == EPI_ADD);
+            tma_store_2d(&tmC, box, EPI == EPI_GATED ? n0 / 2 : s.c0 + n0, t0 + c, EPI == EPI_ADD);
             bulk_commit();
           }
         }
@@ -521,7 +558,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               if (j < t_left)
-                dst[(int64_t)j * p.ldc] = old[j] + __uint_as_float(r[j]) * (normed ? p.alpha * norm_r[t0 + c + j] : p.alpha);
+                dst[(int64_t)j * p.ldc] = old[j] + (__uint_as_float(r[j]) * (normed ? p.alpha * norm_r[t0 + c + j] : p.alpha) + bias_n);
           } else if (EPI == EPI_GATED) {
             // as above, each lane storing its own values
             const bool low = lane < 16;
@@ -534,17 +571,26 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               const float send = __uint_as_float(low ? r[j + 1] : r[j]);
               const float got = __shfl_xor_sync(0xffffffffu, send, 16);
               const float rr = normed ? norm_r[t0 + c + j + (low ? 0 : 1)] : 1.0f;       // my token's pending norm
-              const float g = (low ? mine : got) * rr, up = (low ? got : mine) * rr;
+              const float bias_p = __shfl_xor_sync(0xffffffffu, bias_n, 16);
+              const float g = (low ? mine : got) * rr + (low ? bias_n : bias_p), up = (low ? got : mine) * rr + (low ? bias_p : bias_n);
               const float v = gated_value(p, g, up);
               if (j + (low ? 0 : 1) < f_left) store_out<OutT>(dst + (int64_t)j * p.ldc, v);
             }
           } else {
-            OutT* dst = (OutT*)p.C + (int64_t)(t0 + c) * p.ldc + n;
+            OutT* dst = (OutT*)p.C + (int64_t)(t0 + c) * p.ldc + s.c0 + n;
+            float gate[16];
+            if (p.gate != nullptr) {
+              const float* src = p.gate + (int64_t)(t0 + c) * p.gate_ld + (s.w0 + row);
+#pragma unroll
+              for (int j = 0; j < 16; ++j) gate[j] = j < t_left ? src[(int64_t)j * p.gate_ld] : 0.f;
+            }
 #pragma unroll
             for (int j = 0; j < 16; ++j)
-              if (j < t_left)
-                store_out<OutT>(dst + (int64_t)j * p.ldc,
-                                stored_value(p, __uint_as_float(r[j]) * (normed ? p.alpha * norm_r[t0 + c + j] : p.alpha)));
+              if (j < t_left) {
+                float v = __uint_as_float(r[j]) * (normed ? p.alpha * norm_r[t0 + c + j] : p.alpha) + bias_n;
+                if (p.gate != nullptr) v = __fdividef(v, 1.0f + __expf(-gate[j]));
+                store_out<OutT>(dst + (int64_t)j * p.ldc, stored_value(p, v));
+              }
           }
         }
       }
@@ -658,6 +704,9 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       constexpr bool CAN_EMIT = EPI == EPI_ADD && PENDING_NORM;
       const bool emit = CAN_EMIT && p.emit_xb != nullptr;
       const float g_n = emit && n_in ? p.emit_g[n] : 0.f;
+      const float bias_n = p.bias != nullptr && n_in ? p.bias[n] : 0.f;
+      const bool emit_tanh = emit && p.emit_b != nullptr;
+      const float b_n = emit_tanh && n_in ? p.emit_b[n] : 0.f;
       {
         constexpr int CPI = BN >= 64 ? 8 : (BN >= 32 ? 4 : 2);      // columns whose loads are in flight together
         for (int cb = 0; cb < BN; cb += CPI * p.splits) {
@@ -689,6 +738,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
               for (int r = 1; r < 8; ++r) v += part[h][r];
               if (normed) v *= norm_r[column ? t0 + col[h] : 0];
+              v += bias_n;
               const float up = __shfl_xor_sync(0xffffffffu, v, 16);
               const int f = (n0 + quarter * 32) / 2 + (lane & 15);
               if (ok[h] && lane < 16 && f < p.n_features)
@@ -700,17 +750,19 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               float v = part[h][0];
 #pragma unroll
               for (int r = 1; r < 8; ++r) v += part[h][r];
-              v *= normed ? p.alpha * norm_r[t0 + col[h]] : p.alpha;
+              v = v * (normed ? p.alpha * norm_r[t0 + col[h]] : p.alpha) + bias_n;
               const int64_t at = (int64_t)(t0 + col[h]) * p.ldc + n;
               if (EPI == EPI_ADD) {
                 now = old[h] + v;
                 ((float*)p.C)[at] = now;
-                if (emit) p.emit_xb[(int64_t)(t0 + col[h]) * p.emit_ld + n] = __float2bfloat16_rn(now * g_n);
+                if (emit)
+                  p.emit_xb[(int64_t)(t0 + col[h]) * p.emit_ld + n] =
+                      __float2bfloat16_rn(emit_tanh ? fmaf(g_n, tanhf(p.emit_alpha * now), b_n) : now * g_n);
               } else {
                 store_out<OutT>((OutT*)p.C + at, stored_value(p, v));
               }
             }
-            if (emit && column) {
+            if (emit && !emit_tanh && column) {
               // the squares of this warp's 32 columns of C, lane 0 .. lane 31 in a fixed tree
               float sq = now * now;
 #pragma unroll
@@ -1075,11 +1127,16 @@ namespace {
 struct NormOptions {
   const float* in_ss = nullptr; int in_parts = 0; float in_width = 0.f, in_eps = 0.f;
   void* out_xb = nullptr; int64_t out_ld = 0; const float* out_g = nullptr; float* out_ss = nullptr;
+  const float* out_b = nullptr; float out_alpha = 0.f;
 };
 thread_local NormOptions t_norm;
-struct GatedAct { float alpha = 1.f, limit = 0.f, shift = 0.f; };
+struct GatedAct { float alpha = 1.f, limit = 0.f, shift = 0.f; int kind = 0; };
 thread_local GatedAct t_act;
-struct StoreOptions { int square_relu = 0; const int* tile_group = nullptr; int group_rows = 0; };
+struct StoreOptions {
+  int square_relu = 0; const int* tile_group = nullptr; int group_rows = 0;
+  const float* bias = nullptr;
+  int heads = 0, head_x = 0, head_c = 0; const float* gate = nullptr; int64_t gate_ld = 0;
+};
 thread_local StoreOptions t_store;
 }  // namespace
 
@@ -1101,7 +1158,30 @@ RB_EXPORT int rb_gemm_tc_grouped(const int* tile_group) {
 // The next gated product (epilogue 3) of this thread applies g' sigmoid(alpha g') (u' + shift) with g' = min(g, limit)
 // and u' = clamp(u, -limit, limit) (limit <= 0: none) instead of SiLU(gate) * up.
 RB_EXPORT int rb_gemm_tc_gated_act(float alpha, float limit, float shift) {
-  t_act.alpha = alpha; t_act.limit = limit; t_act.shift = shift;
+  t_act.alpha = alpha; t_act.limit = limit; t_act.shift = shift; t_act.kind = 0;
+  return 0;
+}
+
+// The next gated product (epilogue 3) of this thread applies gelu_tanh(gate) * up.
+RB_EXPORT int rb_gemm_tc_gated_gelu() {
+  t_act.kind = 1;
+  return 0;
+}
+
+// The next product of this thread adds bias[row of W] (float32) to its finished sums; a grouped product or one matrix
+// per head has none.
+RB_EXPORT int rb_gemm_tc_bias(const float* bias) {
+  t_store.bias = bias;
+  return 0;
+}
+
+// The next stored product (epilogue 0, one split) of this thread multiplies by one matrix per head (see GemmParams): W
+// holds heads * n_out rows, X and C the heads' columns head_x and head_c apart.  A token tile of 128 and more writes
+// whole boxes of 128 columns, so it needs head_c >= n_out rounded up to 128; what it leaves in columns n_out .. of a head
+// is not defined.  gate: null, or float32 with column h * n_out + n for value n of head h.
+RB_EXPORT int rb_gemm_tc_per_head(int heads, int head_x, int head_c, const float* gate, long long gate_ld) {
+  RB_REQUIRE(heads > 0 && head_x > 0 && head_c > 0, "rb_gemm_tc_per_head: bad sizes heads=%d, %d and %d apart", heads, head_x, head_c);
+  t_store.heads = heads; t_store.head_x = head_x; t_store.head_c = head_c; t_store.gate = gate; t_store.gate_ld = gate_ld;
   return 0;
 }
 
@@ -1118,6 +1198,14 @@ RB_EXPORT int rb_gemm_tc_pending_norm(const float* ss, int parts, float width, f
 RB_EXPORT int rb_gemm_tc_leave_norm(void* xb, int64_t ld, const float* g, float* ss) {
   RB_REQUIRE(xb != nullptr && g != nullptr && ss != nullptr && ld > 0, "rb_gemm_tc_leave_norm: bad arguments");
   t_norm.out_xb = xb; t_norm.out_ld = ld; t_norm.out_g = g; t_norm.out_ss = ss;
+  t_norm.out_b = nullptr;
+  return 0;
+}
+
+// The same where the norm that follows is a tanh: xb takes bfloat16(w[column] * tanh(alpha * C_new) + b[column]).
+RB_EXPORT int rb_gemm_tc_leave_tanh(void* xb, int64_t ld, const float* w, const float* b, float alpha) {
+  RB_REQUIRE(xb != nullptr && w != nullptr && b != nullptr && ld > 0, "rb_gemm_tc_leave_tanh: bad arguments");
+  t_norm.out_xb = xb; t_norm.out_ld = ld; t_norm.out_g = w; t_norm.out_ss = nullptr; t_norm.out_b = b; t_norm.out_alpha = alpha;
   return 0;
 }
 
@@ -1150,6 +1238,12 @@ static int gemm_tc(void* C, int64_t ldc, int c_dtype, const void* X, int64_t ldx
   RB_REQUIRE(store.tile_group == nullptr || (splits == 1 && token_tile > 0 && w_rows % n_out == 0),
              "rb_gemm_tc: grouped rows want K whole, a given token tile and whole groups (splits %d, tile %d, %d rows of %d)",
              splits, token_tile, w_rows, n_out);
+  RB_REQUIRE(store.bias == nullptr || (epilogue != EPI_QKV && store.tile_group == nullptr && store.heads == 0),
+             "rb_gemm_tc: a bias goes with a plain stored, added or gated product");
+  RB_REQUIRE(store.heads == 0 || (epilogue == EPI_STORE && splits == 1 && store.tile_group == nullptr && token_tile > 0 &&
+                                  w_rows == store.heads * n_out && store.head_x >= K && store.head_x % 8 == 0 && store.head_c >= n_out),
+             "rb_gemm_tc: one matrix per head wants a stored product with K whole, a given token tile and heads a multiple of 8 "
+             "columns apart (%d heads of %d x %d, %d and %d apart, %d rows)", store.heads, n_out, K, store.head_x, store.head_c, w_rows);
   RB_REQUIRE(alpha == 1.0f || epilogue == EPI_STORE || epilogue == EPI_ADD, "rb_gemm_tc: alpha %g with epilogue %d", alpha, epilogue);
   RB_REQUIRE(n_tokens > 0 && n_out > 0 && K > 0, "rb_gemm_tc: bad sizes tokens=%d out=%d K=%d", n_tokens, n_out, K);
   RB_REQUIRE(K % 8 == 0, "rb_gemm_tc: inner size %d is not a multiple of 8", K);
@@ -1169,6 +1263,9 @@ static int gemm_tc(void* C, int64_t ldc, int c_dtype, const void* X, int64_t ldx
   // stride; an output that is not (a width of 257 bfloat16 values) takes tiles of 64, which store by themselves
   const int out_elem = (epilogue == EPI_ADD || c_dtype == RB_F32) ? 4 : 2;
   if (plan.bn >= 128 && (((uintptr_t)C & 15) != 0 || (ldc * out_elem) % 16 != 0))
+    plan = plan_for_tile(n_tokens, n_out, K, 64, rb_sm_count(), false);
+  // one matrix per head: a head's last box of 128 columns must not reach into the next head's, and starts on 16 bytes
+  if (store.heads > 0 && plan.bn >= 128 && ((n_out + BM - 1) / BM * BM > store.head_c || store.head_c % 8 != 0))
     plan = plan_for_tile(n_tokens, n_out, K, 64, rb_sm_count(), false);
   const int bn = plan.bn;
   RB_REQUIRE(epilogue != EPI_GATED || (n_out % 32 == 0 && n_features > 0 && n_features <= n_out / 2),
@@ -1201,6 +1298,7 @@ static int gemm_tc(void* C, int64_t ldc, int c_dtype, const void* X, int64_t ldx
       const int feat_main = epilogue == EPI_GATED ? (n_features < out_off ? n_features : (int)out_off) : 0;
       t_act = act;                 // both products of the pair apply the caller's activation
       t_store.square_relu = store.square_relu;
+      t_store.bias = store.bias;
       if (gemm_tc(C, ldc, c_dtype, X, ldx, n_tokens, W, ldw, rows_main, rows_main, K, epilogue, feat_main, 1, bn, nullptr,
                   alpha, stream) != 0)
         return -1;
@@ -1210,23 +1308,24 @@ static int gemm_tc(void* C, int64_t ldc, int c_dtype, const void* X, int64_t ldx
       const int per = (nkb + parts - 1) / parts;
       t_act = act;
       t_store.square_relu = store.square_relu;
+      t_store.bias = store.bias != nullptr ? store.bias + rows_main : nullptr;
       return gemm_tc(c_tail, ldc, c_dtype, X, ldx, n_tokens, w_rest, ldw, w_rows - rows_main, n_out - rows_main, K, epilogue,
                      epilogue == EPI_GATED ? n_features - (int)out_off : 0, (nkb + per - 1) / per, 64, nullptr, alpha, stream);
     }
   }
   CUtensorMap tw, tx;
   if (rb_get_tensor_map(&tw, W, w_rows, K, ldw, BM) != 0) return -1;
-  if (rb_get_tensor_map(&tx, X, n_tokens, K, ldx, bn) != 0) return -1;
+  if (rb_get_tensor_map(&tx, X, n_tokens, store.heads > 0 ? store.heads * store.head_x : K, ldx, bn) != 0) return -1;
   CUtensorMap tc = tw;               // token tiles below 128 store by themselves
   if (bn >= 128 && epilogue != EPI_QKV) {
-    const int cols = epilogue == EPI_GATED ? n_features : n_out;
+    const int cols = epilogue == EPI_GATED ? n_features : (store.heads > 0 ? store.heads * store.head_c : n_out);
     if (rb_get_output_map(&tc, C, n_tokens, cols, ldc, 16, epilogue == EPI_GATED ? BM / 2 : BM, out_elem) != 0) return -1;
   }
   GemmParams p;
   p.C = C; p.ldc = ldc; p.n_tokens = n_tokens; p.n_out = n_out; p.K = K;
   p.n_features = n_features; p.kb_per_split = (nkb + splits - 1) / splits;
   RB_REQUIRE((int64_t)(splits - 1) * p.kb_per_split < nkb, "rb_gemm_tc: a split of K would be empty");
-  const int n_w_tiles = (n_out + BM - 1) / BM, n_t_tiles = (n_tokens + bn - 1) / bn;
+  const int n_w_tiles = (n_out + BM - 1) / BM * (store.heads > 0 ? store.heads : 1), n_t_tiles = (n_tokens + bn - 1) / bn;
   const long long items = (long long)n_w_tiles * n_t_tiles * splits;
   RB_REQUIRE(items < (1ll << 30), "rb_gemm_tc: too many tiles");
   p.n_t_tiles = n_t_tiles; p.splits = splits; p.n_items = (int)items;
@@ -1234,13 +1333,18 @@ static int gemm_tc(void* C, int64_t ldc, int c_dtype, const void* X, int64_t ldx
   p.alpha = alpha;
   p.act_alpha = 1.f; p.act_limit = 0.f; p.act_shift = 0.f;
   p.square_relu = store.square_relu; p.tile_group = store.tile_group; p.group_rows = n_out;
+  p.act_kind = 0;
   if (epilogue == EPI_GATED) {
-    p.act_alpha = act.alpha; p.act_limit = act.limit; p.act_shift = act.shift;
+    p.act_alpha = act.alpha; p.act_limit = act.limit; p.act_shift = act.shift; p.act_kind = act.kind;
   }
+  p.bias = store.bias;
+  p.heads = store.heads; p.head_x = store.head_x; p.head_c = store.head_c;
+  p.gate = store.heads > 0 ? store.gate : nullptr; p.gate_ld = store.gate_ld;
   p.norm_ss = norm.in_ss; p.norm_parts = norm.in_parts; p.norm_width = norm.in_width; p.norm_eps = norm.in_eps;
   RB_REQUIRE(norm.in_ss == nullptr || (bn <= 16 && n_tokens <= 16),
              "rb_gemm_tc: a pending norm with %d tokens in tiles of %d (at most 16 tokens)", n_tokens, bn);
   p.emit_xb = (__nv_bfloat16*)norm.out_xb; p.emit_ld = norm.out_ld; p.emit_g = norm.out_g; p.emit_ss = norm.out_ss;
+  p.emit_b = norm.out_b; p.emit_alpha = norm.out_alpha;
   RB_REQUIRE(norm.out_xb == nullptr || (epilogue == EPI_ADD && p.cluster && bn <= 16),
              "rb_gemm_tc: only an added product of at most 16 tokens whose K is split into a cluster leaves a norm's inputs");
   p.n_w_tiles = n_w_tiles;

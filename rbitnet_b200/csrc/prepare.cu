@@ -15,33 +15,9 @@
 //                              under its RMS norm and the turned key part go into the cache row [c | k_r | 0], the
 //                              queries leave with their last R values turned
 //   rotate_rows_kernel         float32 rows in place: a prefix of every head turned by position
-#include "rb_common.cuh"
+#include "rb_rotary.cuh"
 
 namespace {
-
-// position * frequency in float64, brought into (-pi, pi] before the float32 sine and cosine
-__device__ __forceinline__ void angle_sincos(int pos, double freq, float magnitude, float* sn, float* cs) {
-  const double a = (double)pos * freq;
-  const double turns = rint(a * 0.15915494309189535);
-  const float r = (float)fma(-turns, 6.283185307179586, a);
-  sincosf(r, sn, cs);
-  *sn *= magnitude;
-  *cs *= magnitude;
-}
-
-// value e of a head after the rotation of its first rot_dim values; val(i) gives the head's value i before it
-template <typename F>
-__device__ __forceinline__ float turned(F val, int e, int rot_dim, int interleaved, const float* s_sincos) {
-  if (e >= rot_dim) return val(e);
-  const int rhalf = rot_dim >> 1;
-  int pair, other;
-  bool first;
-  if (interleaved) { pair = e >> 1; first = (e & 1) == 0; other = first ? e + 1 : e - 1; }
-  else { first = e < rhalf; pair = first ? e : e - rhalf; other = first ? e + rhalf : e - rhalf; }
-  const float sn = s_sincos[pair], cs = s_sincos[rhalf + pair];
-  const float me = val(e), ot = val(other);
-  return first ? me * cs - ot * sn : me * cs + ot * sn;
-}
 
 // one or two neighbouring values (two: the address is a multiple of two values)
 template <typename T> __device__ __forceinline__ void rb_store_values(T* dst, const float* y, int n);

@@ -11,6 +11,9 @@
 // Variants, each a parameter: `scoring` 1 takes s = sigmoid(z), output by output, instead of the softmax; the router's
 // matrix may hold `n_extra` further rows after the n outputs, whose sums leave as they are (a gate that reads the same
 // rows); the gather may multiply a pair's input row by the pair's weight (experts whose weight acts on the input).
+// `scoring` 2 chooses by z itself and weighs the chosen outputs with the softmax over the chosen z alone.  The weighted
+// sum may also add a further expert's result under a gate of one number per token, and leave w tanh(alpha x) + b of the
+// residual row it has made for the sublayer after it.
 //
 // The pairs whose expert has weights are sorted by expert into rows of a padded buffer in which every
 // expert's rows start on a tile border, so that a tile of rows multiplies by one expert's matrix
@@ -27,23 +30,15 @@ namespace {
 // of the block's tokens at once, so that a row of Wr is read once per block (lanes stride over k four values at a
 // time; a token's sum is the lanes' partial sums added in a fixed tree, whatever other tokens the block holds).  Then
 // warp w makes the choice of token w.  Shared memory: per token 2 n + 2 groups floats.
-__device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
-  const float4 f = *reinterpret_cast<const float4*>(p);
-  v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-}
-__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&v)[4]) {
-  const uint2 raw = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
-}
-
 // One warp: from the token's router sums z[0..n) (shared memory; choice, gscore: n and 2 groups floats of scratch) to
 // its `top` outputs and their weights.
 __device__ __forceinline__ void route_select(float* z, float* choice, float* gscore, const float* __restrict__ correction,
                                              int n, int top, int groups, int keep, int lane, int* __restrict__ ids,
                                              float* __restrict__ weights, int64_t t, int scoring = 0) {
-  if (scoring == 1) {
+  if (scoring == 2) {
+    for (int e = lane; e < n; e += 32) choice[e] = z[e] + (correction != nullptr ? correction[e] : 0.f);
+    __syncwarp();
+  } else if (scoring == 1) {
     for (int e = lane; e < n; e += 32) {
       const float s = 1.0f / (1.0f + expf(-z[e]));
       z[e] = s;
@@ -113,6 +108,18 @@ __device__ __forceinline__ void route_select(float* z, float* choice, float* gsc
     }
     __syncwarp();
   }
+  if (scoring == 2) {
+    // the softmax over the chosen outputs' z (lane 0 has left them in `weights`)
+    float* mine = weights + (int64_t)t * top;
+    float m = -INFINITY;
+    for (int j = lane; j < top; j += 32) m = fmaxf(m, mine[j]);
+    m = rb_warp_max(m);
+    float sum = 0.f;
+    for (int j = lane; j < top; j += 32) sum += expf(mine[j] - m);
+    sum = rb_warp_sum(sum);
+    __syncwarp();
+    for (int j = lane; j < top; j += 32) mine[j] = expf(mine[j] - m) / sum;
+  }
 }
 
 constexpr int ROUTE_TB = 8;
@@ -139,13 +146,13 @@ __global__ void __launch_bounds__(256) route_kernel(int* __restrict__ ids, float
 #pragma unroll 2
       for (int k = lane * 4; k < K; k += 128) {
         float hv[4];
-        load4(row + k, hv);
+        rb_load4(row + k, hv);
 #pragma unroll
         for (int a = 0; a < 4; ++a) {
           const int e = e0 + 8 * a;
           if (e < n) {
             float wv[4];
-            load4(Wr + (int64_t)e * K + k, wv);
+            rb_load4(Wr + (int64_t)e * K + k, wv);
 #pragma unroll
             for (int i = 0; i < 4; ++i) acc[a] = fmaf(hv[i], wv[i], acc[a]);
           }
@@ -167,12 +174,12 @@ __global__ void __launch_bounds__(256) route_kernel(int* __restrict__ ids, float
 #pragma unroll 4
       for (int k = lane * 4; k < K; k += 128) {
         float wv[4];
-        load4(w + k, wv);
+        rb_load4(w + k, wv);
 #pragma unroll
         for (int j = 0; j < ROUTE_TB; ++j) {
           if (j < nt) {
             float hv[4];
-            load4(h + (int64_t)(t0 + j) * ldh + k, hv);
+            rb_load4(h + (int64_t)(t0 + j) * ldh + k, hv);
 #pragma unroll
             for (int i = 0; i < 4; ++i) acc[j] = fmaf(hv[i], wv[i], acc[j]);
           }
@@ -371,14 +378,28 @@ __global__ void gather_scaled_kernel(T* __restrict__ xp, const T* __restrict__ h
 }
 
 // ---------------------------------------------------------------- weighted sum
+// What the weighted sum adds and leaves besides (null: not):
+//   shared, gate   x also takes sigmoid(gate[t * ldg]) * shared[t, :] in (a further expert that every token uses)
+//   norm_w         norm_out[t, :] = norm_w tanh(norm_alpha x[t, :]) + norm_b of the finished row
+struct CombineTail {
+  const float* shared = nullptr;
+  const float* gate = nullptr;
+  int64_t ldg = 0;
+  const float* norm_w = nullptr;
+  const float* norm_b = nullptr;
+  float norm_alpha = 0.f;
+  void* norm_out = nullptr;
+};
+
 // x[t, :] (+)= sum_j w[t, j] * (pos[t, j] >= 0 ? y[pos[t, j], :] : h[t, :]), the choices in their order.
 template <typename T>
 __global__ void combine_kernel(float* __restrict__ x, int64_t ldx, const float* __restrict__ y, const T* __restrict__ h,
                                int64_t ldh, const int* __restrict__ pos, const float* __restrict__ weights, int top, int E,
-                               int accumulate, int vec4) {
+                               int accumulate, int vec4, CombineTail tail) {
   rb_pdl_launch_dependents();
   rb_pdl_wait();
   const int t = blockIdx.x;
+  const float sg = tail.shared != nullptr ? 1.0f / (1.0f + expf(-tail.gate[(int64_t)t * tail.ldg])) : 0.f;
   if (vec4) {
     // four columns a thread: 16-byte loads of the experts' rows and of the residual stream
     for (int c = threadIdx.x * 4; c < E; c += blockDim.x * 4) {
@@ -387,18 +408,33 @@ __global__ void combine_kernel(float* __restrict__ x, int64_t ldx, const float* 
         const int r = pos[(int64_t)t * top + j];
         const float w = weights != nullptr ? weights[(int64_t)t * top + j] : 1.0f;
         float v[4];
-        if (r >= 0) load4(y + (int64_t)r * E + c, v);
-        else load4(h + (int64_t)t * ldh + c, v);
+        if (r >= 0) rb_load4(y + (int64_t)r * E + c, v);
+        else rb_load4(h + (int64_t)t * ldh + c, v);
 #pragma unroll
         for (int i = 0; i < 4; ++i) acc[i] = fmaf(w, v[i], acc[i]);
       }
-      float4* dst = reinterpret_cast<float4*>(x + (int64_t)t * ldx + c);
-      float4 out = make_float4(acc[0], acc[1], acc[2], acc[3]);
-      if (accumulate) {
-        const float4 old = *dst;
-        out = make_float4(old.x + acc[0], old.y + acc[1], old.z + acc[2], old.w + acc[3]);
+      if (tail.shared != nullptr) {
+        float v[4];
+        rb_load4(tail.shared + (int64_t)t * E + c, v);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[i] = fmaf(v[i], sg, acc[i]);
       }
-      *dst = out;
+      float* dst = x + (int64_t)t * ldx + c;
+      if (accumulate) {
+        float old[4];
+        rb_load4(dst, old);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[i] += old[i];
+      }
+      rb_store4(dst, acc);
+      if (tail.norm_w != nullptr) {
+        float ww[4], bb[4];
+        rb_load4(tail.norm_w + c, ww);
+        rb_load4(tail.norm_b + c, bb);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[i] = fmaf(ww[i], tanhf(tail.norm_alpha * acc[i]), bb[i]);
+        rb_store4((T*)tail.norm_out + (int64_t)t * E + c, acc);
+      }
     }
     return;
   }
@@ -410,8 +446,12 @@ __global__ void combine_kernel(float* __restrict__ x, int64_t ldx, const float* 
       const float v = r >= 0 ? y[(int64_t)r * E + c] : rb_to_float<T>(h[(int64_t)t * ldh + c]);
       acc = fmaf(w, v, acc);
     }
+    if (tail.shared != nullptr) acc = fmaf(tail.shared[(int64_t)t * E + c], sg, acc);
     float* dst = x + (int64_t)t * ldx + c;
-    *dst = accumulate ? *dst + acc : acc;
+    const float now = accumulate ? *dst + acc : acc;
+    *dst = now;
+    if (tail.norm_w != nullptr)
+      ((T*)tail.norm_out)[(int64_t)t * E + c] = rb_from_float<T>(fmaf(tail.norm_w[c], tanhf(tail.norm_alpha * now), tail.norm_b[c]));
   }
 }
 
@@ -497,7 +537,7 @@ static int route_impl(int* ids, float* weights, const void* h, int64_t ldh, int 
                       const float* correction, int T, int K, int n, int top, int groups, int keep, float* z_scratch,
                       int scoring, int n_extra, float* extra, cudaStream_t stream) {
   if (T == 0) return 0;
-  RB_REQUIRE(scoring == 0 || scoring == 1, "rb_route: scoring %d is not built (0: softmax, 1: sigmoid)", scoring);
+  RB_REQUIRE(scoring >= 0 && scoring <= 2, "rb_route: scoring %d is not built (0: softmax, 1: sigmoid, 2: softmax over the chosen)", scoring);
   RB_REQUIRE(n_extra >= 0 && (n_extra == 0 || extra != nullptr), "rb_route: %d extra rows and nowhere to leave them", n_extra);
   const int n_all = n + n_extra;
   RB_REQUIRE(K > 0 && n > 0 && top > 0 && top <= n, "rb_route: bad sizes K=%d outputs=%d top=%d", K, n, top);
@@ -542,7 +582,8 @@ RB_EXPORT int rb_route(int* ids, float* weights, const void* h, int64_t ldh, int
   return route_impl(ids, weights, h, ldh, h_dtype, Wr, correction, T, K, n, top, groups, keep, z_scratch, 0, 0, nullptr, stream);
 }
 
-// The same with the variants: scoring (0: softmax over the outputs, 1: a sigmoid per output); Wr holds n + n_extra rows
+// The same with the variants: scoring (0: softmax over the outputs, 1: a sigmoid per output, 2:
+// the chosen outputs' softmax); Wr holds n + n_extra rows
 // and the sums of the last n_extra leave in extra [T, n_extra]; z_scratch then holds T * (n + n_extra) floats.
 RB_EXPORT int rb_route_scored(int* ids, float* weights, const void* h, int64_t ldh, int h_dtype, const float* Wr,
                               const float* correction, int T, int K, int n, int top, int groups, int keep, float* z_scratch,
@@ -630,18 +671,34 @@ RB_EXPORT int rb_routed_gather_scaled(void* xp, const void* h, int64_t ldh, int 
   return 0;
 }
 
+// The next rb_routed_combine call of this thread also adds sigmoid(gate[t * ldg]) * shared[t, :] (float32 [T, E]; null: not)
+// and leaves norm_w tanh(norm_alpha x) + norm_b of the finished rows in norm_out ([T, E] of the input rows' type; norm_w
+// null: not).
+static thread_local CombineTail t_combine;
+RB_EXPORT int rb_routed_combine_next(const float* shared, const float* gate, int64_t ldg, const float* norm_w, const float* norm_b,
+                                     float norm_alpha, void* norm_out) {
+  t_combine.shared = shared; t_combine.gate = gate; t_combine.ldg = ldg;
+  t_combine.norm_w = norm_w; t_combine.norm_b = norm_b; t_combine.norm_alpha = norm_alpha; t_combine.norm_out = norm_out;
+  return 0;
+}
+
 RB_EXPORT int rb_routed_combine(float* x, int64_t ldx, const float* y, const void* h, int64_t ldh, int h_dtype,
                                 const int* pos, const float* weights, int T, int top, int E, int accumulate,
                                 cudaStream_t stream) {
+  const CombineTail tail = t_combine;
+  t_combine = CombineTail();
   if (T == 0) return 0;
+  RB_REQUIRE(tail.shared == nullptr || tail.gate != nullptr, "rb_routed_combine: a shared result without its gate");
+  RB_REQUIRE(tail.norm_w == nullptr || (tail.norm_b != nullptr && tail.norm_out != nullptr), "rb_routed_combine: a norm without its place");
   const int elem = h_dtype == RB_F32 ? 4 : 2;
   const int vec4 = E % 4 == 0 && ldx % 4 == 0 && ldh % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 &&
-                   (uintptr_t)h % (4 * elem) == 0;
+                   (uintptr_t)h % (4 * elem) == 0 && (uintptr_t)tail.shared % 16 == 0 && (uintptr_t)tail.norm_w % 16 == 0 &&
+                   (uintptr_t)tail.norm_b % 16 == 0 && (uintptr_t)tail.norm_out % (4 * elem) == 0;
   const int threads = vec4 ? (E >= 1024 ? 256 : (E >= 512 ? 128 : 64)) : (E >= 256 ? 256 : (E >= 128 ? 128 : 64));
   if (h_dtype == RB_F32)
-    RB_LAUNCH("combine_kernel", (combine_kernel<float>), T, threads, 0, stream, x, ldx, y, (const float*)h, ldh, pos, weights, top, E, accumulate, vec4);
+    RB_LAUNCH("combine_kernel", (combine_kernel<float>), T, threads, 0, stream, x, ldx, y, (const float*)h, ldh, pos, weights, top, E, accumulate, vec4, tail);
   else if (h_dtype == RB_BF16)
-    RB_LAUNCH("combine_kernel", (combine_kernel<__nv_bfloat16>), T, threads, 0, stream, x, ldx, y, (const __nv_bfloat16*)h, ldh, pos, weights, top, E, accumulate, vec4);
+    RB_LAUNCH("combine_kernel", (combine_kernel<__nv_bfloat16>), T, threads, 0, stream, x, ldx, y, (const __nv_bfloat16*)h, ldh, pos, weights, top, E, accumulate, vec4, tail);
   else
     RB_FAIL("rb_routed_combine: unknown dtype %d", h_dtype);
   RB_CHECK_LAUNCH("rb_routed_combine");

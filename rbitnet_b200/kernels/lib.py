@@ -22,7 +22,8 @@ _SIGNATURES = {
     "rb_gather_rows": [P, P, P, I, I, P],
     "rb_gemm_simple": [P, L, I, P, L, P, L, I, I, I, I, I, F, P],
     "rb_gemm_simple_batched": [P, L, I, P, L, P, L, I, I, I, I, I, F, I, L, L, L, P],
-    "rb_per_head_few_rows": [P, L, I, P, L, P, I, I, I, I, I, P],
+    "rb_per_head_few_rows": [P, L, I, P, L, I, P, I, I, I, I, I, P],
+    "rb_gemm_simple_next": [P, P, L, L],
     "rb_stream_step": [P, I, I, I, P, P, I, P, P, P, P, F, P, I, P, P],
     "rb_streams_expand": [P, P, I, I, I, P],
     "rb_streams_sum": [P, P, I, I, I, P],
@@ -30,7 +31,8 @@ _SIGNATURES = {
     "rb_streams_max_results": [],
     "rb_norm_rotate_append": [P, P, L, I, P, P, F, P, F, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, P],
     "rb_head_gate": [P, P, P, L, I, I, I, I, I, I, P],
-    "rb_gated_act": [P, P, I, I, I, I, L, I, F, F, F, P],
+    "rb_gated_act": [P, P, I, I, I, I, L, I, I, F, F, F, P, P],
+    "rb_tanh_norm": [P, I, P, P, P, F, I, I, P],
     "rb_conv_causal": [P, P, L, I, I, P, P, P, P, P, P, P, I, I, I, I, P],
     "rb_conv_tail_update": [P, P, L, I, I, P, P, P, P, P, I, I, I, P],
     "rb_delta_prepare": [P, L, P, L, I, I, P, P, P, P, P, P, I, I, I, I, F, F, P],
@@ -71,7 +73,10 @@ _SIGNATURES = {
     "rb_gla_chunk_floats": [I],
     "rb_gla_chunked": [P, P, L, I, I, I, P, F, P, P, P, P, P, P, P, P, I, I, I, I, I, P],
     "rb_gla_scan": [P, P, L, I, I, I, P, F, P, P, P, P, I, I, I, I, P],
-    "rb_latent_norm_append": [P, I, P, L, I, I, I, I, P, P, F, P, P, I, I, I, P, P, I, P],
+    "rb_latent_norm_append": [P, I, P, L, I, I, I, I, I, P, P, F, P, F, I, P, P, I, I, I, P, P, I, P],
+    "rb_latent_queries_few": [P, P, P, I, P, F, I, P, I, I, I, I, I, I, P],
+    "rb_latent_turn": [P, P, I, P, F, I, P, I, I, I, I, I, I, P],
+    "rb_routed_combine_next": [P, P, L, P, P, F, P],
     "rb_route_scored": [P, P, P, L, I, P, P, I, I, I, I, I, I, P, I, I, P, P],
     "rb_routed_gather_scaled": [P, P, L, I, P, P, P, I, I, I, P],
     "rb_attention_simple": [P, P, I, P, P, P, I, I, P, P, I, I, I, I, F, I, P],
@@ -138,6 +143,10 @@ class KernelLibrary:
         self.declare("rb_gemm_tc_leave_norm", [P, L, P, P])
         self.declare("rb_gemm_tc_norm_parts", [I])
         self.declare("rb_gemm_tc_gated_act", [F, F, F])
+        self.declare("rb_gemm_tc_gated_gelu", [])
+        self.declare("rb_gemm_tc_bias", [P])
+        self.declare("rb_gemm_tc_per_head", [I, I, I, P, L])
+        self.declare("rb_gemm_tc_leave_tanh", [P, L, P, P, F])
         self.declare("rb_device_sm_count", [])
         self.declare("rb_is_checked_build", [])
         for tu in CHECKED_FILES:

@@ -20,6 +20,7 @@ from .lib import load, KernelError
 
 F32, BF16 = 0, 1
 _CODE = {torch.float32: F32, torch.bfloat16: BF16}
+_SCORING = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
 
 
 def _ptr(t: Optional[torch.Tensor]):
@@ -40,11 +41,13 @@ class GateUpWeight:
 
     ``block == 0``: rows [gate | up].  ``block == 16``: for every 16 output features, their 16 gate
     rows followed by their 16 up rows (the last group padded with zero rows), which is how the
-    tensor-core product pairs gate and up inside one warp of its epilogue."""
+    tensor-core product pairs gate and up inside one warp of its epilogue.  ``bias``: float32, a number per
+    row of ``w`` (None: no biases)."""
     w: torch.Tensor
     inner: int
     n_in: int
     block: int = 0
+    bias: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -78,6 +81,16 @@ class NormRequest:
     weight: torch.Tensor          # float32 [width]
     eps: float
     result: Optional["NormedRows"] = None
+
+
+@dataclass
+class TanhRequest:
+    """Asks the operation that adds to the residual stream to leave the rows w tanh(alpha x) + b for whoever reads them
+    next.  Nothing is pending afterwards: ``result`` is the rows themselves in the compute dtype, if it did."""
+    weight: torch.Tensor          # float32 [width]
+    bias: torch.Tensor            # float32 [width]
+    alpha: float
+    result: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -154,6 +167,8 @@ class CudaOps:
         self.fuse_norm_filter = True
         #: rows from which a scored router's sums are a tensor-core product (where that product gives the same sums)
         self.router_tc_from = 1
+        #: products with one matrix per head of many rows run on the tensor cores where the sizes allow it
+        self.per_head_on_tensor_cores = True
         #: so does gated linear attention
         self.gla_in_chunks = True
         #: a decode step's delta rule (convolution to gate) is one kernel while rows x heads fit the SMs
@@ -210,9 +225,14 @@ class CudaOps:
         """Output rows first .. first+count-1 of a prepared matrix, sharing its memory."""
         return LinearWeight(weight.w[first:first + count], count, weight.n_in)
 
-    def prepare_gate_up(self, gate: torch.Tensor, up: torch.Tensor) -> GateUpWeight:
+    def prepare_gate_up(self, gate: torch.Tensor, up: torch.Tensor, gate_bias: Optional[torch.Tensor] = None,
+                        up_bias: Optional[torch.Tensor] = None) -> GateUpWeight:
         gate, up = self.to_compute(gate), self.to_compute(up)
         F, K = gate.shape
+        bias = None
+        if gate_bias is not None:
+            gb, ub = (t.to(device=self.device, dtype=torch.float32).reshape(F) for t in (gate_bias, up_bias))
+            bias = torch.cat([gb, ub]).contiguous()
         if self.dtype == torch.bfloat16 and K % 8 == 0:
             # the layout of the tensor-core gated product: groups of 16 gate rows and their 16 up rows
             groups = -(-F // 16)
@@ -222,8 +242,13 @@ class CudaOps:
                 w[:whole, half] = m[:whole * 16].view(whole, 16, K)
                 if F % 16:
                     w[whole, half, :F % 16] = m[whole * 16:]
-            return GateUpWeight(w.view(groups * 32, K), F, K, 16)
-        return GateUpWeight(torch.cat([gate, up], dim=0).contiguous(), F, K, 0)
+            if bias is not None:
+                rows = torch.zeros((groups, 2, 16), dtype=torch.float32, device=self.device)
+                for half, v in ((0, gb), (1, ub)):
+                    rows[:, half] = torch.nn.functional.pad(v, (0, groups * 16 - F)).view(groups, 16)
+                bias = rows.view(groups * 32)
+            return GateUpWeight(w.view(groups * 32, K), F, K, 16, bias)
+        return GateUpWeight(torch.cat([gate, up], dim=0).contiguous(), F, K, 0, bias)
 
     # ------------------------------------------------------------------ ops
     def embed(self, ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
@@ -239,6 +264,14 @@ class CudaOps:
         T, E = x.shape
         out = torch.empty((T, E), dtype=out_dtype or self.dtype, device=self.device)
         self.lib.call("rb_rmsnorm", _ptr(out), _CODE[out.dtype], _ptr(x), _ptr(w), T, E, float(eps), self._stream())
+        return out
+
+    def tanh_norm(self, x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, alpha: float, out_dtype=None) -> torch.Tensor:
+        """w * tanh(alpha * x) + b, value by value in float32; the result in the compute dtype."""
+        self._check(x, torch.float32, "tanh_norm input")
+        T, E = x.shape
+        out = torch.empty((T, E), dtype=out_dtype or self.dtype, device=self.device)
+        self.lib.call("rb_tanh_norm", _ptr(out), _CODE[out.dtype], _ptr(x), _ptr(w), _ptr(b), float(alpha), T, E, self._stream())
         return out
 
     def layernorm(self, x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: float, out_dtype=None) -> torch.Tensor:
@@ -259,10 +292,11 @@ class CudaOps:
         return x
 
     def linear(self, x, weight: LinearWeight, out_dtype=None, accumulate_into: Optional[torch.Tensor] = None,
-               scale: float = 1.0, then_norm: Optional[NormRequest] = None, act: Optional[str] = None) -> torch.Tensor:
-        """scale * x[T, in] * W[out, in]^T (the scale multiplies the finished float32 sums).  With
+               scale: float = 1.0, then_norm=None, act: Optional[str] = None,
+               bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """scale * x[T, in] * W[out, in]^T + bias (the scale multiplies the finished float32 sums; bias: float32 [out]).  With
         ``accumulate_into`` (float32 [T, out]) the product is added to it in float32 and it is returned.
-        ``x`` may be ``NormedRows``.  ``then_norm``: see ``NormRequest`` (granted for a few tokens, where
+        ``x`` may be ``NormedRows``.  ``then_norm``: see ``NormRequest`` and ``TanhRequest`` (granted for a few tokens, where
         the product's parts along the inner dimension meet on chip).  ``act`` "relu2": max(v, 0)^2 of the
         finished float32 sums is stored (in the tensor-core product's epilogue, else by a kernel after it)."""
         if act not in (None, "relu2"):
@@ -297,10 +331,14 @@ class CudaOps:
                 then_norm.result = self._leave_norm(out, then_norm, T, N)
             if act is not None:
                 self.lib.call("rb_gemm_tc_square_relu", launches=0)
+            if bias is not None:
+                self.lib.call("rb_gemm_tc_bias", _ptr(bias), launches=0)
             self.lib.call("rb_gemm_tc", _ptr(out), out.stride(0), _CODE[out.dtype], _ptr(x), x.stride(0), T,
                           _ptr(weight.w), weight.w.stride(0), N, N, K, acc, 0, splits,
                           64 if 64 < T <= 256 else 0, float(scale), self._stream())
         else:
+            if bias is not None:
+                self.lib.call("rb_gemm_simple_next", _ptr(bias), c_void_p(0), 0, 0, launches=0)
             self.lib.call("rb_gemm_simple", _ptr(out), out.stride(0), _CODE[out.dtype], _ptr(x), x.stride(0),
                           _ptr(weight.w), weight.w.stride(0), self.code, T, N, K, acc, float(scale), self._stream())
             if act is not None:
@@ -315,6 +353,12 @@ class CudaOps:
             return None
         return NormRequest(weight, float(eps))
 
+    def tanh_request(self, weight: torch.Tensor, bias: torch.Tensor, alpha: float) -> Optional[TanhRequest]:
+        """The same for a tanh in place of a norm (``TanhRequest``)."""
+        if self.dtype != torch.bfloat16 or not self.fold_norms:
+            return None
+        return TanhRequest(weight, bias, float(alpha))
+
     def normed(self, rows: NormedRows) -> torch.Tensor:
         """The normed rows themselves, for whoever does not take ``NormedRows``."""
         return self.rmsnorm(rows.x, rows.weight, rows.eps)
@@ -327,8 +371,13 @@ class CudaOps:
         self.lib.call("rb_gemm_tc_pending_norm", _ptr(rows.squares), rows.squares.shape[0], float(rows.x.shape[1]),
                       float(rows.eps), launches=0)
 
-    def _leave_norm(self, out: torch.Tensor, request: NormRequest, T: int, N: int) -> NormedRows:
+    def _leave_norm(self, out: torch.Tensor, request, T: int, N: int):
         """For the next tensor-core product of this thread (one that adds into ``out``)."""
+        if isinstance(request, TanhRequest):
+            rows = torch.empty((T, N), dtype=torch.bfloat16, device=self.device)
+            self.lib.call("rb_gemm_tc_leave_tanh", _ptr(rows), rows.stride(0), _ptr(request.weight), _ptr(request.bias),
+                          float(request.alpha), launches=0)
+            return rows
         parts = self.lib.raw("rb_gemm_tc_norm_parts")(N)
         scaled = torch.empty((T, N), dtype=torch.bfloat16, device=self.device)
         squares = torch.empty((parts, T), dtype=torch.float32, device=self.device)
@@ -349,15 +398,33 @@ class CudaOps:
                 and w.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
                 and x.stride(1) == 1 and w.stride(1) == 1)
 
+    def _gated_act(self, out: torch.Tensor, gu: torch.Tensor, inner: int, block: int, act, bias=None) -> None:
+        """out = the gated activation ``act`` of float32 rows [gate | up], by a kernel of its own."""
+        kind, (alpha, limit, shift) = (1, (1.0, 0.0, 0.0)) if act == "gelu_tanh" else (0, act)
+        self.lib.call("rb_gated_act", _ptr(out), _ptr(gu), self.code, F32, gu.shape[0], inner, gu.stride(0), block, kind,
+                      float(alpha), float(limit), float(shift), _ptr(bias), self._stream())
+
+    def _next_gated_act(self, act) -> None:
+        """For the next gated tensor-core product of this thread."""
+        if act == "gelu_tanh":
+            self.lib.call("rb_gemm_tc_gated_gelu", launches=0)
+        else:
+            self.lib.call("rb_gemm_tc_gated_act", float(act[0]), float(act[1]), float(act[2]), launches=0)
+
     def gated_linear(self, x: torch.Tensor, weight: GateUpWeight, act=None) -> torch.Tensor:
         """silu(x Wg^T) * (x Wu^T) -> [T, inner] in the compute dtype.  ``act`` = (alpha, limit, shift):
-        g' sigmoid(alpha g') (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit) instead."""
+        g' sigmoid(alpha g') (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit) instead (limit 0: none);
+        "gelu_tanh": gelu(g) u, gelu in its tanh form.  The weight's biases are added to g and u first."""
+        if act is None and weight.bias is not None:
+            act = (1.0, 0.0, 0.0)
         if act is not None and weight.block == 16 and not isinstance(x, NormedRows) and self.fuse_gated_act \
                 and self._tensor_core_ok(x, weight.w):
-            # the tensor-core gated product with the limited activation in its epilogue
+            # the tensor-core gated product with the activation in its epilogue
             T, rows = x.shape[0], weight.w.shape[0]
             out = torch.empty((T, weight.inner), dtype=self.dtype, device=self.device)
-            self.lib.call("rb_gemm_tc_gated_act", float(act[0]), float(act[1]), float(act[2]), launches=0)
+            self._next_gated_act(act)
+            if weight.bias is not None:
+                self.lib.call("rb_gemm_tc_bias", _ptr(weight.bias), launches=0)
             self.lib.call("rb_gemm_tc", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), T,
                           _ptr(weight.w), weight.w.stride(0), rows, rows, weight.n_in, 3, weight.inner, 1, 0,
                           1.0, self._stream())
@@ -368,9 +435,7 @@ class CudaOps:
             T, rows = x.shape[0], weight.w.shape[0]
             gu = self.linear(x, LinearWeight(weight.w, rows, weight.n_in), out_dtype=torch.float32)
             out = torch.empty((T, weight.inner), dtype=self.dtype, device=self.device)
-            alpha, limit, shift = act
-            self.lib.call("rb_gated_act", _ptr(out), _ptr(gu), self.code, F32, T, weight.inner, gu.stride(0),
-                          weight.block, float(alpha), float(limit), float(shift), self._stream())
+            self._gated_act(out, gu, weight.inner, weight.block, act, weight.bias)
             return out
         pending = x if isinstance(x, NormedRows) else None
         if pending is not None:
@@ -1017,37 +1082,93 @@ class CudaOps:
 
     # ------------------------------------------------------------------ attention through latents
     def latent_norm_append(self, down: torch.Tensor, q_rank: int, kv_rank: int, wq: torch.Tensor, wkv: torch.Tensor,
-                           eps: float, meta, view) -> torch.Tensor:
-        """From float32 rows [query latent | key/value latent]: each under its RMS norm and weight; the query latent is
-        returned ([T, q_rank], compute dtype), the other goes to the sequence's page (``view.head_dim`` wide, padded
-        with zeros)."""
+                           eps: float, meta, view, rot_dim: int = 0, table=None) -> torch.Tensor:
+        """From float32 rows [query latent | key/value latent | key part of rot_dim]: each latent under its RMS norm and
+        weight, the key part turned by position (``table``); the query latent is returned ([T, q_rank], compute dtype),
+        the others go to the sequence's page as [c | k_r | zeros] (``view.head_dim`` wide)."""
         self._check(down, torch.float32, "latent_norm_append rows")
         T = down.shape[0]
+        freq, magnitude, interleaved = self._whole_turn(table, rot_dim, "latent_norm_append")
         cq = torch.empty((T, q_rank), dtype=self.dtype, device=self.device)
         self.lib.call("rb_latent_norm_append", _ptr(cq), self.code, _ptr(down), down.stride(0), 0, q_rank, q_rank, kv_rank,
-                      _ptr(wq), _ptr(wkv), float(eps), _ptr(view.k), _ptr(view.page_table), view.max_pages, view.page_size,
-                      view.head_dim, _ptr(meta.tok_pos), _ptr(meta.tok_slot), T, self._stream())
+                      int(rot_dim), _ptr(wq), _ptr(wkv), float(eps), _ptr(freq), float(magnitude), 1 if interleaved else 0,
+                      _ptr(view.k), _ptr(view.page_table), view.max_pages, view.page_size, view.head_dim, _ptr(meta.tok_pos),
+                      _ptr(meta.tok_slot), T, self._stream())
         return cq
+
+    @staticmethod
+    def _whole_turn(table, rot_dim: int, what: str):
+        """(frequencies, magnitude, interleaved) of a table that turns ``rot_dim`` values."""
+        if not rot_dim:
+            return None, 1.0, True
+        freq, magnitude, interleaved, turned = table
+        if turned != rot_dim:
+            raise KernelError(f"{what}: the position encoding turns {turned} of {rot_dim} values")
+        return freq, magnitude, interleaved
+
+    def latent_queries(self, q: torch.Tensor, weight: PerHeadWeight, rot_dim: int, width: int, table, meta) -> torch.Tensor:
+        """Query heads [q_c | q_r (rot_dim)] into the latent's space: [T, H * width], head h [W_h q_c | q_r turned by
+        position | zeros].  ``weight``: [H, latent, size of q_c]."""
+        self._check(q, self.dtype, "latent_queries input")
+        T, H, C, D, R = q.shape[0], weight.heads, weight.n_out, weight.n_in, int(rot_dim)
+        if q.shape[1] != H * (D + R) or width < C + R:
+            raise KernelError(f"latent_queries: rows of {q.shape[1]} values are not {H} heads of {D} + {R}, or {width} is too narrow")
+        freq, magnitude, interleaved = self._whole_turn(table, R, "latent_queries")
+        out = torch.empty((T, H * width), dtype=self.dtype, device=self.device)
+        if T <= 16:
+            self.lib.call("rb_latent_queries_few", _ptr(out), _ptr(q), _ptr(weight.w), self.code, _ptr(freq), float(magnitude),
+                          1 if interleaved else 0, _ptr(meta.tok_pos), T, H, D, R, C, int(width), self._stream())
+            return out
+        self._per_head(out, width, q, D + R, weight)
+        if width > C:
+            self.lib.call("rb_latent_turn", _ptr(out), _ptr(q), self.code, _ptr(freq), float(magnitude),
+                          1 if interleaved else 0, _ptr(meta.tok_pos), T, H, D, R, C, int(width), self._stream())
+        return out
 
     def prepare_per_head(self, w: torch.Tensor) -> PerHeadWeight:
         """[heads, n_out, n_in] -> ready for ``per_head_linear``."""
         w = self.to_compute(w)
         return PerHeadWeight(w, w.shape[0], w.shape[1], w.shape[2])
 
-    def per_head_linear(self, x: torch.Tensor, weight: PerHeadWeight) -> torch.Tensor:
-        """x [T, heads * n_in] -> [T, heads * n_out]: head h's values times its own matrix (float32 sums)."""
+    def _per_head(self, out: torch.Tensor, head_c: int, x: torch.Tensor, head_x: int, weight: PerHeadWeight, gate=None) -> None:
+        """out[:, h * head_c : + n_out] = x[:, h * head_x : + n_in] * W_h^T for many rows (the other columns of a head are
+        undefined afterwards); ``gate`` = (float32 rows, first column): times sigmoid of column h * n_out + n of them."""
+        T, H, N, K = x.shape[0], weight.heads, weight.n_out, weight.n_in
+        gate_ptr, ldg = c_void_p(0), 0
+        if gate is not None:
+            self._check(gate[0], torch.float32, "per-head gate")
+            gate_ptr, ldg = c_void_p(gate[0].data_ptr() + gate[1] * 4), gate[0].stride(0)
+        if self.per_head_on_tensor_cores and self._tensor_core_ok(x, weight.w) and K % 8 == 0 and head_x % 8 == 0:
+            whole_boxes = -(-N // 128) * 128 <= head_c and head_c % 8 == 0
+            tile = 64 if T <= 256 or not whole_boxes else 256
+            self.lib.call("rb_gemm_tc_per_head", H, int(head_x), int(head_c), gate_ptr, ldg, launches=0)
+            self.lib.call("rb_gemm_tc", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), T, _ptr(weight.w), K, H * N, N,
+                          K, 0, 0, 1, tile, 1.0, self._stream())
+            return
+        if gate is not None:
+            self.lib.call("rb_gemm_simple_next", c_void_p(0), gate_ptr, ldg, N, launches=0)
+        self.lib.call("rb_gemm_simple_batched", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), _ptr(weight.w), K,
+                      self.code, T, N, K, 0, 1.0, H, int(head_c), int(head_x), N * K, self._stream())
+
+    def per_head_linear(self, x: torch.Tensor, weight: PerHeadWeight, gate=None) -> torch.Tensor:
+        """x [T, heads * s] -> [T, heads * n_out]: the first n_in <= s values of head h times its own matrix (float32 sums).
+        ``gate`` = (float32 rows [T, ...], column): value n of head h times sigmoid(rows[:, column + h * n_out + n])."""
         self._check(x, self.dtype, "per_head_linear input")
         T, H, N, K = x.shape[0], weight.heads, weight.n_out, weight.n_in
-        if x.shape[1] != H * K:
+        head_x = x.shape[1] // H
+        if x.shape[1] != H * head_x or head_x < K:
             raise KernelError(f"per_head_linear: rows of {x.shape[1]} values are not {H} heads of {K}")
         out = torch.empty((T, H * N), dtype=self.dtype, device=self.device)
         if T <= 16:
             # a decode step: a warp per output and head instead of a few tiles
-            self.lib.call("rb_per_head_few_rows", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), _ptr(weight.w),
+            if gate is not None:
+                self._check(gate[0], torch.float32, "per-head gate")
+                self.lib.call("rb_gemm_simple_next", c_void_p(0), c_void_p(gate[0].data_ptr() + gate[1] * 4), gate[0].stride(0), N,
+                              launches=0)
+            self.lib.call("rb_per_head_few_rows", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), head_x, _ptr(weight.w),
                           self.code, T, H, N, K, self._stream())
             return out
-        self.lib.call("rb_gemm_simple_batched", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), _ptr(weight.w), K,
-                      self.code, T, N, K, 0, 1.0, H, N, K, N * K, self._stream())
+        self._per_head(out, N, x, head_x, weight, gate)
         return out
 
     # ------------------------------------------------------------------ routed experts, the variants
@@ -1063,7 +1184,8 @@ class CudaOps:
 
     def route_scored(self, h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int,
                      keep: int, scoring: str = "softmax", extra_rows: int = 0, router_tc: Optional[LinearWeight] = None):
-        """``route`` with its variants: ``scoring`` "sigmoid" takes s = sigmoid(z) output by output; the last
+        """``route`` with its variants: ``scoring`` "sigmoid" takes s = sigmoid(z) output by output, "softmax_chosen"
+        chooses by z itself and takes the softmax over the chosen z alone; the last
         ``extra_rows`` rows of ``router`` are no outputs: their float32 sums are returned as they are ([T, extra_rows],
         None without).  Returns (ids, weights, extra)."""
         self._check(h, self.dtype, "route input")
@@ -1077,13 +1199,13 @@ class CudaOps:
             # kernel that does both has a block per token (20 us at 8 tokens against 7 for the two)
             z = self.linear(h, router_tc, out_dtype=torch.float32)
             self.lib.call("rb_route_select_scored", _ptr(ids), _ptr(weights), _ptr(z), _ptr(correction), T, n, int(top),
-                          int(groups), int(keep), {"softmax": 0, "sigmoid": 1}[scoring], int(extra_rows), _ptr(extra),
+                          int(groups), int(keep), _SCORING[scoring], int(extra_rows), _ptr(extra),
                           self._stream())
             return ids, weights, extra
         z = torch.empty((T, n + extra_rows), dtype=torch.float32, device=self.device) if T >= 64 else None
         self.lib.call("rb_route_scored", _ptr(ids), _ptr(weights), _ptr(h), h.stride(0), self.code, _ptr(router),
                       _ptr(correction), T, K, n, int(top), int(groups), int(keep), _ptr(z),
-                      {"softmax": 0, "sigmoid": 1}[scoring], int(extra_rows), _ptr(extra), self._stream(),
+                      _SCORING[scoring], int(extra_rows), _ptr(extra), self._stream(),
                       launches=2 if z is not None else 1)
         return ids, weights, extra
 
@@ -1133,13 +1255,15 @@ class CudaOps:
 
     def routed_experts(self, h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up, w_down: LinearWeight,
                        n_experts: int, inner: int, accumulate_into: Optional[torch.Tensor] = None, act=None,
-                       weight_on_input: bool = False):
+                       weight_on_input: bool = False, shared=None, then_norm: Optional[TanhRequest] = None):
         """sum_j weights[t, j] * expert(ids[t, j])(h[t]) with expert e: W_down_e relu2(W_up_e h); ids >= n_experts are
         identity experts (h[t] itself).  ``w_up``: [n_experts * inner, width], ``w_down``: [n_experts * width, inner].
         Added to ``accumulate_into`` (float32), or returned as float32 rows.
         ``act`` = (alpha, limit, shift): gated experts, ``w_up`` an ``ExpertGateUp``, the inner rows
         g' sigmoid(alpha g') (u' + shift) as in ``gated_linear``.  ``weight_on_input``: sum_j expert(weights[t, j] * h[t])
-        instead (the weighted row is rounded to the compute dtype before the expert's first product)."""
+        instead (the weighted row is rounded to the compute dtype before the expert's first product).
+        ``shared`` = (float32 rows, float32 gate logits [T, 1]): sigmoid(gate) * rows is added in the same kernel as the
+        weighted sum; a ``TanhRequest`` is granted there too."""
         T, E = h.shape
         top = ids.shape[1]
         pairs = T * top
@@ -1172,7 +1296,7 @@ class CudaOps:
                 gu = None if fused else torch.empty((rows, per), dtype=torch.float32, device=self.device)
                 if fused:
                     # the activation in the grouped product's epilogue: the inner rows leave it in bfloat16
-                    self.lib.call("rb_gemm_tc_gated_act", float(act[0]), float(act[1]), float(act[2]), launches=0)
+                    self._next_gated_act(act)
                     self.lib.call("rb_gemm_tc_grouped", _ptr(tile_group), launches=0)
                     self.lib.call("rb_gemm_tc", _ptr(mid), mid.stride(0), self.code, _ptr(xp), xp.stride(0), rows, _ptr(w_up.w),
                                   w_up.w.stride(0), n_experts * per, per, E, 3, inner, 1, tile, 1.0, self._stream())
@@ -1184,8 +1308,7 @@ class CudaOps:
                     self.lib.call("rb_gemm_grouped_simple", _ptr(gu), gu.stride(0), F32, _ptr(xp), xp.stride(0), _ptr(w_up.w),
                                   w_up.w.stride(0), self.code, _ptr(tile_group), rows, per, E, 0, self._stream())
                 if not fused:
-                    self.lib.call("rb_gated_act", _ptr(mid), _ptr(gu), self.code, F32, rows, inner, gu.stride(0), w_up.block,
-                                  float(act[0]), float(act[1]), float(act[2]), self._stream())
+                    self._gated_act(mid, gu, inner, w_up.block, act)
                 if tc:
                     self.lib.call("rb_gemm_tc_grouped", _ptr(tile_group), launches=0)
                     self.lib.call("rb_gemm_tc", _ptr(y), y.stride(0), F32, _ptr(mid), mid.stride(0), rows, _ptr(w_down.w),
@@ -1208,6 +1331,16 @@ class CudaOps:
                               w_down.w.stride(0), self.code, _ptr(tile_group), rows, E, inner, 0, self._stream())
         else:
             pos = torch.full((pairs,), -1, dtype=torch.int32, device=self.device)
+        if shared is not None or isinstance(then_norm, TanhRequest):
+            z, gate = shared if shared is not None else (None, None)
+            if z is not None:
+                self._check(z, torch.float32, "shared expert's rows")
+            req = then_norm if isinstance(then_norm, TanhRequest) else None
+            if req is not None:
+                req.result = torch.empty((T, E), dtype=self.dtype, device=self.device)
+            self.lib.call("rb_routed_combine_next", _ptr(z), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                          _ptr(req.weight if req else None), _ptr(req.bias if req else None), float(req.alpha if req else 0.0),
+                          _ptr(req.result if req else None), launches=0)
         self.lib.call("rb_routed_combine", _ptr(out), out.stride(0), _ptr(y), _ptr(h), h.stride(0), self.code, _ptr(pos),
                       _ptr(None if weight_on_input else weights), T, top, E, acc, self._stream())
         return out

@@ -7,12 +7,15 @@ and costs three in a chain of dependent launches.  Where the operations offer it
 sides say that they pass it on (``folds_norms``), the block asks the part before a norm to have its
 last product leave the rows times the norm's weights, with their sums of squares, and gives those
 to the part after the norm, whose first product multiplies its sums by each row's factor.  Parts
-that know nothing of this get the normed rows as before.
+that know nothing of this get the normed rows as before.  A norm that needs no sums over the row (a tanh in its place)
+asks for the finished rows themselves, which any part reads; a part that only ``passes_norms`` on may leave those too.
 
 An arrangement is a class built from a ``BlockSpec`` with ``parts()`` (name -> part, every part
 whose weights are to be bound; the names are those of ``BlockSpec.parts``) and
 ``run(ctx, x, entry)``.  ``build_parts`` makes every part a spec names, whatever it is called."""
 from __future__ import annotations
+
+import torch
 
 from .registry import register_part, build_part
 
@@ -45,8 +48,9 @@ class PreNormBlock:
 
     @staticmethod
     def _request(ctx, norm, before):
-        """A request to the part before ``norm``, if both know how."""
-        if norm is None or not getattr(before, "folds_norms", False):
+        """A request to the part before ``norm``, if both know how (a part that ``passes_norms`` on hands ``then_norm`` to
+        its last operation, but reads finished rows only)."""
+        if norm is None or not (getattr(before, "folds_norms", False) or getattr(before, "passes_norms", False)):
             return None
         deferred = getattr(norm, "deferred", None)
         return deferred(ctx.ops) if deferred is not None else None
@@ -56,6 +60,8 @@ class PreNormBlock:
         """The input of ``part``: what the part before left if ``part`` takes it, else the normed rows."""
         if pending is None:
             return norm.forward(ctx, x)
+        if isinstance(pending, torch.Tensor):
+            return pending                        # a norm that needs no sums over the row: the finished rows
         return pending if getattr(part, "folds_norms", False) else ctx.ops.normed(pending)
 
     def run(self, ctx, x, entry: int, pending=None, next_norm=None):

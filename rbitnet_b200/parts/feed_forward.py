@@ -4,6 +4,8 @@ the product are float32 before any rounding to the compute dtype.
 
 ``activation`` "swish_limited": with g' = min(gate h, limit) and u' = clamp(up h, -limit, limit),
 the inner rows are g' * sigmoid(alpha g') * (u' + shift); alpha = 1.702 and shift = 1 unless given.
+``activation`` "gelu_tanh": gelu(gate h) * (up h), gelu in its tanh form.  ``bias``: all three projections have biases,
+added to the float32 sums.
 
 ``Dense``: down(relu2(up h)), no gate.  ``RoutedExperts``: a router chooses a few of many small feed-forwards
 (and identity experts) per token; a shared expert may run beside them."""
@@ -17,24 +19,33 @@ from .registry import register_part
 
 class GatedDense(FeedForward):
     def __init__(self, width: int, inner: int, activation: str = "silu", limit: float = 0.0,
-                 alpha: float = 1.702, shift: float = 1.0):
-        if activation not in ("silu", "swish_limited"):
+                 alpha: float = 1.702, shift: float = 1.0, bias: bool = False):
+        if activation not in ("silu", "swish_limited", "gelu_tanh"):
             raise ValueError(f"gated feed-forward: activation {activation!r} is not built "
-                             "(only 'silu' and 'swish_limited')")
+                             "(only 'silu', 'swish_limited' and 'gelu_tanh')")
         self.width, self.inner, self.activation = int(width), int(inner), activation
-        #: (alpha, limit, shift) of the limited activation; None: SiLU(gate) * up
-        self.act = None if activation == "silu" else (float(alpha), float(limit), float(shift))
-        if self.act is not None and not self.act[1] > 0:
+        #: (alpha, limit, shift) of the limited activation, or "gelu_tanh"; None: SiLU(gate) * up
+        self.act = {"silu": None, "gelu_tanh": "gelu_tanh"}.get(activation, (float(alpha), float(limit), float(shift)))
+        if activation == "swish_limited" and not self.act[1] > 0:
             raise ValueError("gated feed-forward: 'swish_limited' needs a positive limit")
-        self.w_gate_up = self.w_down = None
+        self.has_bias = bool(bias)
+        self.w_gate_up = self.w_down = self.down_bias = None
 
     def weight_shapes(self):
-        return {"gate": ((self.inner, self.width), "matrix"), "up": ((self.inner, self.width), "matrix"),
-                "down": ((self.width, self.inner), "matrix")}
+        shapes = {"gate": ((self.inner, self.width), "matrix"), "up": ((self.inner, self.width), "matrix"),
+                  "down": ((self.width, self.inner), "matrix")}
+        if self.has_bias:
+            shapes.update({"gate.b": ((self.inner,), "matrix"), "up.b": ((self.inner,), "matrix"),
+                           "down.b": ((self.width,), "matrix")})
+        return shapes
 
     def bind(self, weights, ops):
-        self.w_gate_up = ops.prepare_gate_up(weights["gate"], weights["up"])
         self.w_down = ops.prepare_linear([weights["down"]])
+        if self.has_bias:
+            self.w_gate_up = ops.prepare_gate_up(weights["gate"], weights["up"], weights["gate.b"], weights["up.b"])
+            self.down_bias = weights["down.b"].to(device=ops.device, dtype=torch.float32).contiguous()
+        else:
+            self.w_gate_up = ops.prepare_gate_up(weights["gate"], weights["up"])
 
     #: ``h`` may be rows with their norm pending, and ``then_norm`` is handed to the last product
     folds_norms = True
@@ -44,12 +55,12 @@ class GatedDense(FeedForward):
             t = ctx.ops.gated_linear(h, self.w_gate_up)        # silu(gate h) * (up h)
         else:
             t = ctx.ops.gated_linear(h, self.w_gate_up, act=self.act)
+        kw = {"bias": self.down_bias} if self.has_bias else {}
         if accumulate_into is None:
-            return ctx.ops.linear(t, self.w_down, out_dtype=torch.float32)
-        if then_norm is None:
-            ctx.ops.linear(t, self.w_down, accumulate_into=accumulate_into)
-        else:
-            ctx.ops.linear(t, self.w_down, accumulate_into=accumulate_into, then_norm=then_norm)
+            return ctx.ops.linear(t, self.w_down, out_dtype=torch.float32, **kw)
+        if then_norm is not None:
+            kw["then_norm"] = then_norm
+        ctx.ops.linear(t, self.w_down, accumulate_into=accumulate_into, **kw)
 
 
 class Dense(FeedForward):
@@ -84,15 +95,16 @@ class RoutedExperts(FeedForward):
     "sigmoid": s = sigmoid(z), output by output.  The choice is made by s + correction ("correction", one number per
     output), among the outputs of the ``keep`` best of ``groups`` equal groups of neighbouring outputs (a group's score
     is its largest choice score; groups 0 or 1: no groups); the chosen outputs' weights are their s, not
-    renormalised.  ``weight_on`` "output": the result is the weighted sum of the chosen experts' results;
+    renormalised.  "softmax_chosen": the choice is made by z + correction instead, and the chosen outputs' weights are
+    the softmax over their z alone.  ``weight_on`` "output": the result is the weighted sum of the chosen experts' results;
     "input": every chosen expert runs on its weight times the input row, and the results are added up as they are.
 
     ``activation`` "relu2": an expert is down(relu2(up h)) ("e<i>.up" [inner, width], "e<i>.down" [width, inner]).
     "swish_limited": an expert is gated, down(g' sigmoid(alpha g') (u' + shift)) with g' = min(gate h, limit) and
-    u' = clamp(up h, -limit, limit) ("e<i>.gate" beside the other two).
+    u' = clamp(up h, -limit, limit) ("e<i>.gate" beside the other two).  "silu": gated, down(silu(gate h) * up h).
 
-    ``shared`` (a dict with "inner", "limit" and optionally "alpha", "shift"): one more gated expert of that form that
-    every token uses ("shared.gate", "shared.up", "shared.down"), its result multiplied by sigmoid(w_sg . h), one
+    ``shared`` (a dict with "inner" and, for the limited activation, "limit" and optionally "alpha",
+    "shift"): one more gated expert of the same form that every token uses ("shared.gate", "shared.up", "shared.down"), its result multiplied by sigmoid(w_sg . h), one
     number per token ("shared.sg" [1, width]), and added.  The gate's sum is made beside the router's, in float32.
 
     Weights: "router" [n_experts + n_identity, width], "correction" (``correction=False``: none), the experts'."""
@@ -101,26 +113,28 @@ class RoutedExperts(FeedForward):
                  keep: int = 0, correction: bool = True, activation: str = "relu2", scoring: str = "softmax",
                  weight_on: str = "output", limit: float = 0.0, alpha: float = 1.702, shift: float = 1.0,
                  shared: dict = None):
-        if activation not in ("relu2", "swish_limited"):
-            raise ValueError(f"routed experts: activation {activation!r} is not built (only 'relu2' and 'swish_limited')")
-        if scoring not in ("softmax", "sigmoid"):
-            raise ValueError(f"routed experts: scoring {scoring!r} is not built (only 'softmax' and 'sigmoid')")
+        if activation not in ("relu2", "swish_limited", "silu"):
+            raise ValueError(f"routed experts: activation {activation!r} is not built (only 'relu2', 'swish_limited' and 'silu')")
+        if scoring not in ("softmax", "sigmoid", "softmax_chosen"):
+            raise ValueError(f"routed experts: scoring {scoring!r} is not built (only 'softmax', 'sigmoid' and 'softmax_chosen')")
         if weight_on not in ("output", "input"):
             raise ValueError(f"routed experts: the weight acts on the 'output' or on the 'input', not on {weight_on!r}")
         self.width, self.inner, self.n_experts, self.top = int(width), int(inner), int(n_experts), int(top)
         self.n_identity, self.groups, self.keep = int(n_identity), int(groups or 0), int(keep or 0)
         self.has_correction = bool(correction)
         self.activation, self.scoring, self.weight_on = activation, scoring, weight_on
-        #: (alpha, limit, shift) of a gated expert's activation; None: relu2 without a gate
-        self.act = (float(alpha), float(limit), float(shift)) if activation == "swish_limited" else None
-        if self.act is not None and not self.act[1] > 0:
+        #: (alpha, limit, shift) of a gated expert's activation (limit 0: none); None: relu2 without a gate
+        self.act = {"relu2": None, "silu": (1.0, 0.0, 0.0)}.get(activation, (float(alpha), float(limit), float(shift)))
+        if activation == "swish_limited" and not self.act[1] > 0:
             raise ValueError("routed experts: 'swish_limited' needs a positive limit")
         self.shared = None
         if shared:
             self.shared = {"inner": int(shared["inner"]),
-                           "act": (float(shared.get("alpha", 1.702)), float(shared["limit"]), float(shared.get("shift", 1.0)))}
-            if self.shared["inner"] < 1 or not self.shared["act"][1] > 0:
-                raise ValueError("routed experts: the shared expert needs an inner size and a positive limit")
+                           "act": (None if activation == "silu" else
+                                   (float(shared.get("alpha", 1.702)), float(shared["limit"]), float(shared.get("shift", 1.0))))}
+            if self.shared["inner"] < 1 or not (activation == "silu" or self.shared["act"][1] > 0):
+                raise ValueError("routed experts: the shared expert needs an inner size and, with a limited activation, a "
+                                 "positive limit")
         n = self.n_experts + self.n_identity
         if self.weight_on == "input" and self.n_identity:
             raise ValueError("routed experts: identity experts go with weights on the results")
@@ -176,7 +190,10 @@ class RoutedExperts(FeedForward):
             self.shared_gate_up = ops.prepare_gate_up(weights["shared.gate"], weights["shared.up"])
             self.shared_down = ops.prepare_linear([weights["shared.down"]])
 
-    def forward(self, ctx, h, accumulate_into=None):
+    #: ``then_norm`` is handed to the weighted sum, which grants a norm that needs no sums over the row
+    passes_norms = True
+
+    def forward(self, ctx, h, accumulate_into=None, then_norm=None):
         ops = ctx.ops
         if self.plain:
             if self.router_tc is not None:
@@ -188,13 +205,16 @@ class RoutedExperts(FeedForward):
         extra = 1 if self.shared is not None else 0
         ids, weights, gate = ops.route_scored(h, self.router, self.correction, self.top, self.groups, self.keep,
                                               scoring=self.scoring, extra_rows=extra, router_tc=self.router_tc)
-        y = ops.routed_experts(h, ids, weights, self.w_up, self.w_down, self.n_experts, self.inner,
-                               accumulate_into=accumulate_into, act=self.act, weight_on_input=self.weight_on == "input")
+        kw = {}
         if self.shared is not None:
             t = ops.gated_linear(h, self.shared_gate_up, act=self.shared["act"])
-            z = ops.linear(t, self.shared_down, out_dtype=torch.float32)
-            ops.add_scaled_rows(y, z, gate)                      # y += sigmoid(gate) * z, one number per row
-        return y
+            # sigmoid(gate) * z, one number per row, is added beside the experts' results
+            kw["shared"] = (ops.linear(t, self.shared_down, out_dtype=torch.float32), gate)
+        if then_norm is not None:
+            kw["then_norm"] = then_norm
+        return ops.routed_experts(h, ids, weights, self.w_up, self.w_down, self.n_experts, self.inner,
+                                  accumulate_into=accumulate_into, act=self.act,
+                                  weight_on_input=self.weight_on == "input", **kw)
 
 
 register_part("feed_forward", "gated_dense", GatedDense)

@@ -1,7 +1,7 @@
 """``LatentAttention``: causal softmax attention whose keys and values are made from one small vector per position,
 the only thing the cache keeps.
 
-From the input rows h, without biases and without a position encoding:
+From the input rows h, without biases and (unless ``rot_dim`` is given) without a position encoding:
 
     c_q = rmsnorm(W_dq h) * w_dq          [q_rank]      the queries' latent
     q   = W_uq c_q                        [n_heads, head_dim]
@@ -23,9 +23,14 @@ Options, each off by default:
                 rows after the latent's (not normed): one key part per position that all heads share.  Both are turned
                 by position (``position``: a rotary encoding over ``rot_dim`` values) and the score is
                 (q_c . W_uk c + rot(q_r) . rot(k_r)) * scale.  The cache row is [c | rot(k_r)]; a query head enters
-                the attention as [W_uk^T q_c | rot(q_r)] (the small product per head carries an identity block for
-                the turned part), and the result's columns beyond the latent are dropped by W_uv's zero columns
+                the attention as [W_uk^T q_c | rot(q_r)], and the result's columns beyond the latent meet no row of W_uv
   sinks         the softmax's denominator also holds exp(s_h), a stored number per head ("sink")
+  value_gate    the joined heads are multiplied value by value with sigmoid(W_g h) ("g", a row per value), read from the
+                same input rows; its float32 sums come out of the same product as the latents, and the sigmoid is applied
+                where the heads' results leave their matrices W_uv
+
+All options go together.  With queries through a latent AND a turned part, the turned part of the queries exists only
+after W_uq: the step that takes the query heads into the latent's space turns it (``ops.latent_queries``).
 """
 from __future__ import annotations
 
@@ -40,11 +45,12 @@ from .spec import PartSpec
 
 class LatentAttention(Mixer):
     def __init__(self, width: int, n_heads: int, head_dim: int, value_dim: int, q_rank: int, kv_rank: int,
-                 scale: float, norm_eps: float, rot_dim: int = 0, position: dict = None, sinks: bool = False):
+                 scale: float, norm_eps: float, rot_dim: int = 0, position: dict = None, sinks: bool = False,
+                 value_gate: bool = False):
         self.width, self.n_heads, self.head_dim, self.value_dim = int(width), int(n_heads), int(head_dim), int(value_dim)
         self.q_rank, self.kv_rank = int(q_rank or 0), int(kv_rank)
         self.scale, self.norm_eps = float(scale), float(norm_eps)
-        self.rot_dim, self.sinks = int(rot_dim or 0), bool(sinks)
+        self.rot_dim, self.sinks, self.value_gate = int(rot_dim or 0), bool(sinks), bool(value_gate)
         if min(self.n_heads, self.head_dim, self.value_dim, self.kv_rank) < 1 or self.q_rank < 0 or self.rot_dim < 0:
             raise ValueError("latent attention: heads, sizes and ranks are at least 1")
         self.position = None
@@ -54,7 +60,9 @@ class LatentAttention(Mixer):
             self.position = build_part("position", PartSpec(position["kind"], dict(position.get("params", {}))))
             if self.position.head_dim != self.rot_dim or self.position.rot_dim != self.rot_dim:
                 raise ValueError("latent attention: the position encoding turns the whole turned part")
-        self.direct = self.q_rank == 0 or self.rot_dim > 0 or self.sinks
+        self.direct = self.q_rank == 0
+        #: the float32 column of the stacked product at which the gate's sums begin
+        self.gate_at = (self.q_rank or self.n_heads * (self.head_dim + self.rot_dim)) + self.kv_rank + self.rot_dim
         self.sink_w = None
         self.cache_width = self.kv_rank + self.rot_dim
         self.w_down = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = self.q_norm_w = self.kv_norm_w = None
@@ -70,6 +78,8 @@ class LatentAttention(Mixer):
             shapes["q"] = ((H * (D + self.rot_dim), E), "matrix")
         if self.sinks:
             shapes["sink"] = ((H,), "matrix")
+        if self.value_gate:
+            shapes["g"] = ((H * Dv, E), "matrix")
         return shapes
 
     def cache_need(self):
@@ -78,59 +88,67 @@ class LatentAttention(Mixer):
     def bind(self, weights, ops):
         H, D, Dv, R, Rr = self.n_heads, self.head_dim, self.value_dim, self.kv_rank, self.rot_dim
         self.cache_width = Rc = ops.cache_head_width(R + Rr, R + Rr)
+        gate = [weights["g"]] if self.value_gate else []
         if self.q_rank:
-            if self.direct:
-                raise ValueError("latent attention: a turned key part or sinks go with queries made straight from the "
-                                 "input rows (q_rank = 0)")
-            self.w_down = ops.prepare_linear([weights["dq"], weights["dkv"]])
+            self.w_down = ops.prepare_linear([weights["dq"], weights["dkv"]] + gate)
             self.w_uq = ops.prepare_linear([weights["uq"]])
         else:
-            self.w_down = ops.prepare_linear([weights["q"], weights["dkv"]])
-            if self.position is not None:
-                self.position.bind({}, ops)
+            self.w_down = ops.prepare_linear([weights["q"], weights["dkv"]] + gate)
+        if self.position is not None:
+            self.position.bind({}, ops)
         if self.sinks:
             self.sink_w = weights["sink"].to(device=ops.device, dtype=torch.float32).contiguous()
         self.w_o = ops.prepare_linear([weights["o"]])
-        # per head: [Rc, D + Rr] (W_uk of the head, transposed, and an identity block that passes the turned part on)
-        # and [Dv, Rc]; the columns beyond kv_rank are zeros
-        uk = torch.zeros((H, Rc, D + Rr), dtype=weights["uk"].dtype, device=weights["uk"].device)
-        uk[:, :R, :D] = weights["uk"].view(H, D, R).transpose(1, 2)
-        if Rr:
-            uk[:, R:R + Rr, D:] = torch.eye(Rr, dtype=uk.dtype, device=uk.device)
-        uv = torch.zeros((H, Dv, Rc), dtype=weights["uv"].dtype, device=weights["uv"].device)
-        uv[:, :, :R] = weights["uv"].view(H, Dv, R)
+        # per head W_uk of the head, transposed, and W_uv.  Where the queries are turned before they enter the latent's
+        # space, the first carries an identity block that passes the turned part on, and rows of zeros up to the cache's
+        # width: [Rc, D + Rr]; else it is [R, D]
+        if self.direct:
+            uk = torch.zeros((H, Rc, D + Rr), dtype=weights["uk"].dtype, device=weights["uk"].device)
+            uk[:, :R, :D] = weights["uk"].view(H, D, R).transpose(1, 2)
+            if Rr:
+                uk[:, R:R + Rr, D:] = torch.eye(Rr, dtype=uk.dtype, device=uk.device)
+        else:
+            uk = weights["uk"].view(H, D, R).transpose(1, 2).contiguous()
         self.w_uk_t = ops.prepare_per_head(uk)
-        self.w_uv = ops.prepare_per_head(uv)
+        self.w_uv = ops.prepare_per_head(weights["uv"].view(H, Dv, R))
         f32 = dict(device=ops.device, dtype=torch.float32)
         self.q_norm_w = weights["dq.norm"].to(**f32).contiguous() if self.q_rank else None
         self.kv_norm_w = weights["dkv.norm"].to(**f32).contiguous()
 
-    def forward(self, ctx, h, entry, accumulate_into=None):
+    #: ``h`` may be rows with their norm pending, and ``then_norm`` is handed to the last product
+    folds_norms = True
+
+    def forward(self, ctx, h, entry, accumulate_into=None, then_norm=None):
         ops = ctx.ops
         view = ctx.cache_view(entry)
         if not view.writes:
             raise ValueError("latent attention reads only its own cache")
         H = self.n_heads
-        down = ops.linear(h, self.w_down, out_dtype=torch.float32)                  # [T, W_dq h (or W_q h) | W_dkv h]
+        # float32 [T, W_dq h (or W_q h) | W_dkv h | W_g h]
+        down = ops.linear(h, self.w_down, out_dtype=torch.float32)
+        table = self.position.table() if self.position is not None else None
         if self.direct:
-            table = self.position.table() if self.position is not None else None
             q = ops.latent_rotate_append(down, H, self.head_dim, self.rot_dim, self.kv_rank, table, self.kv_norm_w,
                                          self.norm_eps, ctx.meta, view)            # [T, H * (D + Rr)]; [c | k_r] is cached
+            ql = ops.per_head_linear(q, self.w_uk_t)                                # [T, H * Rc]: W_uk^T q per head
         else:
             cq = ops.latent_norm_append(down, self.q_rank, self.kv_rank, self.q_norm_w, self.kv_norm_w, self.norm_eps,
-                                        ctx.meta, view)                             # [T, q_rank]; c is in the cache
-            q = ops.linear(cq, self.w_uq)                                           # [T, H * D]
-        ql = ops.per_head_linear(q, self.w_uk_t)                                    # [T, H * Rc]: W_uk^T q per head
+                                        ctx.meta, view, rot_dim=self.rot_dim, table=table)    # [T, q_rank]; [c | k_r] is cached
+            q = ops.linear(cq, self.w_uq)                                           # [T, H * (D + Rr)]
+            ql = ops.latent_queries(q, self.w_uk_t, self.rot_dim, view.head_dim, table, ctx.meta)
         both = dataclasses.replace(view, v=view.k)                                  # keys and values: the latents
         if self.sinks:
             a = ops.attention(ql.view(ql.shape[0], H, view.head_dim), ctx.meta, both, H, self.scale, None,
                               sinks=self.sink_w)
         else:
             a = ops.attention(ql.view(ql.shape[0], H, view.head_dim), ctx.meta, both, H, self.scale, None)
-        o = ops.per_head_linear(a, self.w_uv)                                       # [T, H * Dv]
+        gate = (down, self.gate_at) if self.value_gate else None
+        o = ops.per_head_linear(a, self.w_uv, gate=gate)                            # [T, H * Dv]
         if accumulate_into is None:
             return ops.linear(o, self.w_o, out_dtype=torch.float32)
-        return ops.linear(o, self.w_o, accumulate_into=accumulate_into)
+        if then_norm is None:
+            return ops.linear(o, self.w_o, accumulate_into=accumulate_into)
+        return ops.linear(o, self.w_o, accumulate_into=accumulate_into, then_norm=then_norm)
 
 
 register_part("mixer", "latent_attention", LatentAttention)

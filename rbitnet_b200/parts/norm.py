@@ -79,5 +79,34 @@ class LayerNorm(Norm):
         return ctx.ops.layernorm(x, self.weight, self.bias, self.eps)
 
 
+class TanhNorm(Norm):
+    """A bounded curve in place of a norm: y = tanh(alpha * x) * w + b, value by value in float32, without a mean or a
+    variance ("Dynamic Tanh").  Weights "weight" and "bias" over the width and the one number "alpha".  Because a value
+    needs nothing but itself, whoever makes the new residual rows can leave the finished rows of this norm as well."""
+
+    def __init__(self, width: int):
+        self.width = int(width)
+        self.weight = self.bias = None
+        self.alpha = 0.0
+
+    def weight_shapes(self):
+        return {"weight": ((self.width,), "norm"), "bias": ((self.width,), "matrix"), "alpha": ((), "norm")}
+
+    def bind(self, weights, ops):
+        self.weight = weights["weight"].to(torch.float32).contiguous()
+        self.bias = weights["bias"].to(torch.float32).contiguous()
+        self.alpha = float(weights["alpha"].to(torch.float32).reshape(-1)[0])
+
+    def forward(self, ctx, x, out_dtype=None):
+        kw = {} if out_dtype is None else {"out_dtype": out_dtype}
+        return ctx.ops.tanh_norm(x, self.weight, self.bias, self.alpha, **kw)
+
+    def deferred(self, ops):
+        """What the operation before this norm needs to leave its rows, if the operations can do that; else None."""
+        make = getattr(ops, "tanh_request", None)
+        return make(self.weight, self.bias, self.alpha) if make is not None else None
+
+
 register_part("norm", "rmsnorm", RMSNorm)
+register_part("norm", "tanh", TanhNorm)
 register_part("norm", "layernorm", LayerNorm)

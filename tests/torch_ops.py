@@ -25,6 +25,17 @@ class _GU:
     w: torch.Tensor
     inner: int
     n_in: int
+    bias: torch.Tensor = None
+
+
+def _gated(act, g, u):
+    """The gated activation the package asks for: (alpha, limit, shift), "gelu_tanh", or None (SiLU)."""
+    if act == "gelu_tanh":
+        return 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3))) * u
+    alpha, limit, shift = act if act is not None else (1.0, 0.0, 0.0)
+    if limit > 0:
+        g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
+    return g / (1.0 + torch.exp(-alpha * g)) * (u + shift)
 
 
 class TorchOps:
@@ -46,8 +57,9 @@ class TorchOps:
     def rows_of(self, weight, first, count):
         return _W(weight.w[first:first + count], count, weight.n_in)
 
-    def prepare_gate_up(self, gate, up):
-        return _GU(torch.cat([self.to_compute(gate), self.to_compute(up)], dim=0), gate.shape[0], gate.shape[1])
+    def prepare_gate_up(self, gate, up, gate_bias=None, up_bias=None):
+        bias = torch.cat([gate_bias, up_bias]).float() if gate_bias is not None else None
+        return _GU(torch.cat([self.to_compute(gate), self.to_compute(up)], dim=0), gate.shape[0], gate.shape[1], bias)
 
     def embed(self, ids, table, scale=1.0):
         return table[ids.long()].to(torch.float32) * scale
@@ -55,6 +67,9 @@ class TorchOps:
     def rmsnorm(self, x, w, eps, out_dtype=None):
         s = (x * x).sum(-1, keepdim=True) / x.shape[-1]
         return (x * w * (1.0 / torch.sqrt(s + eps))).to(out_dtype or self.dtype)
+
+    def tanh_norm(self, x, w, b, alpha, out_dtype=None):
+        return (torch.tanh(alpha * x) * w + b).to(out_dtype or self.dtype)
 
     def layernorm(self, x, w, b, eps, out_dtype=None):
         mu = x.mean(-1, keepdim=True)
@@ -66,8 +81,10 @@ class TorchOps:
         x += y
         return x
 
-    def linear(self, x, weight, out_dtype=None, accumulate_into=None, scale=1.0, act=None):
+    def linear(self, x, weight, out_dtype=None, accumulate_into=None, scale=1.0, act=None, bias=None):
         y = x.to(torch.float32) @ weight.w.to(torch.float32).T * scale
+        if bias is not None:
+            y = y + bias
         if act == "relu2":
             y = torch.clamp(y, min=0.0) ** 2
         if accumulate_into is not None:
@@ -77,12 +94,9 @@ class TorchOps:
 
     def gated_linear(self, x, weight, act=None):
         gu = x.to(torch.float32) @ weight.w.to(torch.float32).T
-        g, u = gu[:, :weight.inner], gu[:, weight.inner:]
-        if act is not None:
-            alpha, limit, shift = act
-            g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
-            return (g / (1.0 + torch.exp(-alpha * g)) * (u + shift)).to(self.dtype)
-        return (g / (1.0 + torch.exp(-g)) * u).to(self.dtype)
+        if weight.bias is not None:
+            gu = gu + weight.bias
+        return _gated(act, gu[:, :weight.inner], gu[:, weight.inner:]).to(self.dtype)
 
     def normed(self, rows):
         return rows
@@ -314,25 +328,44 @@ class TorchOps:
         return (o.reshape(T, H * Dv) * (gate / (1.0 + torch.exp(-gate)))).to(self.dtype)
 
     # ---- attention through latents
-    def latent_norm_append(self, down, q_rank, kv_rank, wq, wkv, eps, meta, view):
+    def latent_norm_append(self, down, q_rank, kv_rank, wq, wkv, eps, meta, view, rot_dim=0, table=None):
         x = down.float()
         cq, c = x[:, :q_rank], x[:, q_rank:q_rank + kv_rank]
         cq = cq / torch.sqrt((cq * cq).mean(-1, keepdim=True) + eps) * wq
         c = c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * wkv
+        kr = x[:, q_rank + kv_rank:q_rank + kv_rank + rot_dim].reshape(x.shape[0], 1, rot_dim).clone()
+        if rot_dim:
+            self._turn(kr, table, meta.tok_pos)
         for t in range(x.shape[0]):
             p, slot = int(meta.tok_pos[t]), int(meta.tok_slot[t])
             page = int(view.page_table[slot, p // view.page_size])
             view.k[page, 0, p % view.page_size, :] = 0
             view.k[page, 0, p % view.page_size, :kv_rank] = c[t].to(view.k.dtype)
+            view.k[page, 0, p % view.page_size, kv_rank:kv_rank + rot_dim] = kr[t, 0].to(view.k.dtype)
         return cq.to(self.dtype)
+
+    def latent_queries(self, q, w, rot_dim, width, table, meta):
+        H, C, D = w.shape
+        T, R = q.shape[0], rot_dim
+        x = q.to(torch.float32).view(T, H, D + R)
+        out = torch.zeros(T, H, width)
+        out[..., :C] = torch.einsum("thk,hnk->thn", x[..., :D], w.to(torch.float32))
+        if R:
+            qr = x[..., D:].clone()
+            self._turn(qr, table, meta.tok_pos)
+            out[..., C:C + R] = qr
+        return out.reshape(T, H * width).to(self.dtype)
 
     def prepare_per_head(self, w):
         return self.to_compute(w)
 
-    def per_head_linear(self, x, w):
+    def per_head_linear(self, x, w, gate=None):
         H, N, K = w.shape
-        y = torch.einsum("thk,hnk->thn", x.to(torch.float32).view(x.shape[0], H, K), w.to(torch.float32))
-        return y.reshape(x.shape[0], H * N).to(self.dtype)
+        y = torch.einsum("thk,hnk->thn", x.to(torch.float32).view(x.shape[0], H, -1)[..., :K], w.to(torch.float32))
+        y = y.reshape(x.shape[0], H * N)
+        if gate is not None:
+            y = y * torch.sigmoid(gate[0][:, gate[1]:gate[1] + H * N])
+        return y.to(self.dtype)
 
     # ---- routed experts
     def prepare_expert_gate_up(self, gates, ups):
@@ -344,7 +377,7 @@ class TorchOps:
         n = router.shape[0] - extra_rows
         extra = z[:, n:].clone() if extra_rows else None
         z = z[:, :n]
-        s = torch.sigmoid(z) if scoring == "sigmoid" else torch.softmax(z, dim=-1)
+        s = {"sigmoid": torch.sigmoid, "softmax_chosen": lambda v: v}.get(scoring, lambda v: torch.softmax(v, dim=-1))(z)
         choice = s + correction if correction is not None else s.clone()
         if groups > 1 and keep < groups:
             per = n // groups
@@ -352,7 +385,10 @@ class TorchOps:
             kept = torch.zeros_like(best, dtype=torch.bool).scatter_(1, best.topk(keep, dim=-1).indices, True)
             choice = choice.masked_fill(~kept.repeat_interleave(per, dim=1), -math.inf)
         ids = choice.topk(top, dim=-1).indices
-        return ids.to(torch.int32), s.gather(1, ids), extra
+        weights = s.gather(1, ids)
+        if scoring == "softmax_chosen":
+            weights = torch.softmax(weights, dim=-1)
+        return ids.to(torch.int32), weights, extra
 
     def route(self, h, router, correction, top, groups, keep):
         s = torch.softmax(h.to(torch.float32) @ router.T, dim=-1)
@@ -366,7 +402,7 @@ class TorchOps:
         return ids.to(torch.int32), s.gather(1, ids)
 
     def routed_experts(self, h, ids, weights, w_up, w_down, n_experts, inner, accumulate_into=None, act=None,
-                       weight_on_input=False):
+                       weight_on_input=False, shared=None):
         T, E = h.shape
         x = h.to(torch.float32)
         out = torch.zeros(T, E)
@@ -379,13 +415,13 @@ class TorchOps:
                 xin = (w * x[t]).to(self.dtype).to(torch.float32) if weight_on_input else x[t]
                 if act is not None:
                     gu = w_up.w[e * 2 * inner:(e + 1) * 2 * inner].to(torch.float32) @ xin
-                    alpha, limit, shift = act
-                    g, u = torch.clamp(gu[:inner], max=limit), torch.clamp(gu[inner:], -limit, limit)
-                    mid = (g / (1.0 + torch.exp(-alpha * g)) * (u + shift)).to(self.dtype).to(torch.float32)
+                    mid = _gated(act, gu[:inner], gu[inner:]).to(self.dtype).to(torch.float32)
                 else:
                     up = w_up.w[e * inner:(e + 1) * inner].to(torch.float32)
                     mid = (torch.clamp(up @ xin, min=0.0) ** 2).to(self.dtype).to(torch.float32)
                 out[t] += (down @ mid) if weight_on_input else w * (down @ mid)
+        if shared is not None:
+            out += torch.sigmoid(shared[1][:, :1]) * shared[0]
         if accumulate_into is not None:
             accumulate_into += out
             return accumulate_into
