@@ -570,6 +570,24 @@ def _gozotar_shape(width, heads, kv, dim, vdim, lat_heads, lat_dim, lat_rot, kv_
             "layers": [dict((lat, att, par)[i % 3]) for i in range(layers)]}
 
 
+def _busavik_shape(width, heads, dim, rot, q_rank, kv_rank, experts, top, expert_ff, shared_ff, layers, vocab=32000, dense_every=0,
+                   ff=0):
+    """Layer sizes in the manner of a real model: attention through latents with a turned key part everywhere; every layer
+    routes `top` of `experts` gated experts beside a shared one, but for every `dense_every`-th layer (0: none), whose
+    feed-forward is dense; from four layers on, the middle two run twice."""
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared_ff}}
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": dim, "q_rank": q_rank, "kv_rank": kv_rank,
+             "scale": (dim + rot) ** -0.5, "rot": {"base": 500000.0, "dims": rot, "scaling": {
+                 "factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    ls = [{"type": "latent_attention", "mixer": mixer,
+           "mlp": {"kind": "dense", "ff": ff} if dense_every and i % dense_every == 0 else moe} for i in range(layers)]
+    cfg = {"architecture": "Busavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+           "max_positions": 8192, "layers": ls}
+    if layers >= 4:
+        cfg["loop"] = {"start": layers // 2 - 1, "stop": layers // 2 + 1, "times": 2}
+    return cfg
+
+
 DESIGN_SIZES = {
     # name: (the design's configuration, the configuration of equal width, layer runs and feed-forward size beside it)
     "w2048": (_safuvik_shape(2048, 16, 4, 128, 64, 1024, 16, 8, 128, 256, 5632, 6), _llama_like(2048, 16, 4, 128, 5632, 6)),
@@ -588,6 +606,12 @@ DESIGN_SIZES = {
                       _nifarax_shape(2048, 8, 128, 256, 16, 128, 768, 128, 32, 4, 1408, 1408, 6)),
     "gozotar_w4096": (_gozotar_shape(4096, 32, 8, 128, 128, 32, 128, 64, 192, 16, 128, 256, 14336, 3),
                       _nifarax_shape(4096, 16, 128, 256, 32, 128, 1536, 256, 64, 8, 1792, 1792, 3)),
+    # Busavik beside Nifarax (attention through latents on queries from a latent, gated experts beside a shared one): 6 runs
+    # of a layer beside 6, 3 beside 3; the cached rows (latent + turned key part) are as wide as Nifarax's latents
+    "busavik_w2048": (_busavik_shape(2048, 16, 128, 32, 768, 96, 32, 4, 1408, 1408, 4, dense_every=2, ff=5632),
+                      _nifarax_shape(2048, 8, 128, 256, 16, 128, 768, 128, 32, 4, 1408, 1408, 6)),
+    "busavik_w4096": (_busavik_shape(4096, 32, 128, 64, 1536, 192, 64, 8, 1792, 1792, 3, dense_every=3, ff=14336),
+                      _nifarax_shape(4096, 16, 128, 256, 32, 128, 1536, 256, 64, 8, 1792, 1792, 3)),
 }
 
 
@@ -597,7 +621,7 @@ class DesignTimer(KernelTimer):
                              "gated_recurrence", "matrix_memory", "layernorm", "add_rows", "gated_delta", "route", "routed_experts",
                              "rmsnorm_grouped", "input_filter", "gated_add", "add_scaled_rows", "softcap", "gated_linear_attention",
                              "latent_norm_append", "per_head_linear", "route_scored", "qk_prepare", "latent_rotate_append",
-                             "retention", "norm_add", "round_rows", "token_gate", "embed_pairs")
+                             "retention", "norm_add", "round_rows", "token_gate", "embed_pairs", "tanh_norm", "latent_queries")
 
     @staticmethod
     def _describe(name, a, kw, sync=True):
@@ -663,13 +687,23 @@ class DesignTimer(KernelTimer):
             T, E = a[0].n_tokens, a[1].shape[1]
             return f"embedding + pair embedding [{T} rows]", T * E * (2 + 2 + 4), 0.0
         if name == "latent_norm_append":
-            down, qr, kr = a[0], a[1], a[2]
+            down, qr, kr, R = a[0], a[1], a[2], kw.get("rot_dim", 0)
             T = down.shape[0]
-            return f"latents' norms + append [{T} rows of {qr}+{kr}]", el(down) + T * (qr + kr) * 2, 0.0
+            what = "latents' norms, turned key part" if R else "latents' norms"
+            return f"{what} + append [{T} rows of {qr}+{kr}{f'+{R}' if R else ''}]", T * (qr + kr + R) * (4 + 2), 0.0
+        if name == "tanh_norm":
+            return f"tanh norm [{a[0].shape[0]} rows]", el(a[0]) + a[0].numel() * 2, 0.0
+        if name == "latent_queries":
+            x, w, R, width = a[0], a[1], a[2], a[3]
+            T = x.shape[0]
+            return (f"queries into the latent's space, turned part [{T}x{w.heads}x({w.n_in}+{R})]x[{w.n_out}x{w.n_in}]",
+                    el(x) + el(w.w) + T * w.heads * width * 2, 2.0 * T * w.heads * w.n_out * w.n_in)
         if name == "per_head_linear":
             x, w = a[0], a[1]
             T = x.shape[0]
-            return (f"product per head [{T}x{w.heads}x{w.n_in}]x[{w.n_out}x{w.n_in}]", el(x) + el(w.w) + T * w.heads * w.n_out * 2,
+            gate = kw.get("gate")
+            return (f"product per head{' and gate' if gate is not None else ''} [{T}x{w.heads}x{w.n_in}]x[{w.n_out}x{w.n_in}]",
+                    el(x) + el(w.w) + T * w.heads * w.n_out * (6 if gate is not None else 2),
                     2.0 * T * w.heads * w.n_out * w.n_in)
         if name == "input_filter":
             return f"input filter [{a[0].shape[0]} rows, {a[1].shape[1]} taps]", 2 * el(a[0]), 0.0
@@ -793,7 +827,7 @@ def main():
     ap.add_argument("--workload", default=None, choices=sorted(WORKLOADS),
                     help="run one of the other generation workloads end to end instead (one short line)")
     ap.add_argument("--design", default=None, choices=sorted(DESIGN_SIZES),
-                    help="instead of the headline: prefill and decode of another design (Safuvik; vaderax_*: Vaderax; nifarax_*; gozotar_*: Gozotar beside Nifarax) beside the Llama decoder of "
+                    help="instead of the headline: prefill and decode of another design (Safuvik; vaderax_*: Vaderax; nifarax_*; gozotar_*: Gozotar beside Nifarax; busavik_*: Busavik beside Nifarax) beside the Llama decoder of "
                          "equal size at these layer sizes, nifarax_*: Nifarax beside Vaderax (uses --batch, --context, --prefill-tokens, "
                          "--steps)")
     args = ap.parse_args()
