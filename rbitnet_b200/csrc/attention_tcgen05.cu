@@ -24,6 +24,15 @@
 // shared memory, which is what bounds N = 128 products whose operands both come from there.  K is
 // K-major with the 128-byte swizzle; V, whose tile [keys, D] has D contiguous, is the MN-major B
 // operand of O += P V.  Every mbarrier wait is bounded.
+//
+// SHARED: keys and values are the same rows (attention through latents: one vector per position).  A tile is then
+// loaded once and is the B operand of both products, as it lies: K-major for S, MN-major for O.  A stage is free when
+// P V of its tile is complete.  Heads of 192 and 256 values are taken in this form only: their Q does not fit tensor
+// memory beside two S buffers and O, so it lies in shared memory, swizzled like K.  With two stages (256 values) the
+// next tile may still be on its way when this tile's P is ready: then P V goes first.
+//
+// Parts: the key tiles of a sequence may be cut into n_splits ranges, one per CTA (a decode step has few row tiles and
+// many keys).  A part leaves its maximum, sum and unnormalised O, which rb_attention_combine merges in their order.
 #include "rb_tcgen05.cuh"
 
 namespace {
@@ -32,7 +41,6 @@ constexpr int ROWS = 128;          // rows of a CTA (UMMA M)
 constexpr int TILE_KEYS = 128;     // keys per tile (UMMA N of S, K of P V)
 constexpr int PIECE = 64;          // positions per TMA piece of a tile (a page, or an aligned part of one)
 constexpr int THREADS = 320;       // loader warp, MMA warp, eight softmax warps
-constexpr int KV_STAGES = 2;
 
 struct TcAttnParams {
   const __nv_bfloat16* q;   // [T, H, D]
@@ -50,6 +58,9 @@ struct TcAttnParams {
   const float* sinks;       // [H] or null: a term exp(sinks[h]) in head h's denominator
   float softcap;            // > 0: score <- softcap * tanh(score * scale / softcap), before the mask
   float scale;
+  float* part_o;            // n_splits > 1: [T, H, n_splits, D], and
+  float* part_ml;           // [T, H, n_splits, 2] (maximum in base-2 units, sum)
+  int n_splits;
 };
 
 // 2^x for x <= 0 (and -inf -> 0) with the hardware approximation (relative error about 2^-22)
@@ -109,39 +120,45 @@ __device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, u
       : "memory");
 }
 
-template <int D>
+template <int D, bool SHARED>
 struct TcSmem {
   static constexpr int DB = D / 64;                         // 64-column blocks of a head
   static constexpr int BLOCK = ROWS * 128;                  // a block of [128 rows][128 bytes]
   static constexpr int KV_TILE_BYTES = BLOCK * DB;          // 128 keys, DB blocks
-  static constexpr int OFF_K = 0;
-  static constexpr int OFF_V = OFF_K + KV_STAGES * KV_TILE_BYTES;
-  static constexpr int OFF_MAX = OFF_V + KV_STAGES * KV_TILE_BYTES;   // float [2 tiles][2 halves][128 rows]
+  static constexpr bool Q_SMEM = 2 * TILE_KEYS + D + D / 2 > 512;      // tensor memory: two S buffers, O and Q
+  static constexpr int STAGES = !SHARED ? 2 : (D >= 256 ? 2 : (D >= 192 ? 3 : 4));
+  static constexpr int OFF_Q = 0;
+  static constexpr int OFF_K = OFF_Q + (Q_SMEM ? KV_TILE_BYTES : 0);
+  static constexpr int OFF_V = OFF_K + (SHARED ? 0 : STAGES * KV_TILE_BYTES);      // SHARED: the same tiles
+  static constexpr int OFF_MAX = OFF_V + STAGES * KV_TILE_BYTES;      // float [2 tiles][2 halves][128 rows]
   static constexpr int OFF_BAR = OFF_MAX + 2 * 2 * ROWS * 4;
-  static constexpr int BYTES = OFF_BAR + 128;
+  static constexpr int BYTES = OFF_BAR + 256;
+  static_assert(BYTES <= 227 * 1024, "shared memory");
 };
 
-template <int D>
+template <int D, bool SHARED>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, TcAttnParams p) {
-  using S = TcSmem<D>;
+  using S = TcSmem<D, SHARED>;
   constexpr int DB = S::DB;
-  // tensor memory: two S buffers in columns [0,256), O in [256, 256+D), Q (two bfloat16 a column) after it
+  constexpr int KV_STAGES = S::STAGES;
+  constexpr bool Q_SMEM = S::Q_SMEM;
+  // tensor memory: two S buffers in columns [0,256), O in [256, 256+D), Q (two bfloat16 a column) after it if it fits
   constexpr int O_COL = 2 * TILE_KEYS;
   constexpr int Q_COL = O_COL + D;
   constexpr int TMEM_COLS = 512;
-  static_assert(2 * TILE_KEYS + D + D / 2 <= 512, "tensor memory columns");
+  static_assert(2 * TILE_KEYS + D + (Q_SMEM ? 0 : D / 2) <= 512, "tensor memory columns");
   extern __shared__ __align__(1024) uint8_t smem[];
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + S::OFF_BAR);
-  uint64_t* k_full = bars;                   // [2] keys of a tile have landed
-  uint64_t* k_empty = bars + 2;              // [2] S of that tile is complete: the key stage is free
-  uint64_t* v_full = bars + 4;               // [2]
-  uint64_t* v_empty = bars + 6;              // [2] P V of that tile is complete
-  uint64_t* s_full = bars + 8;               // [2] one per S buffer
-  uint64_t* p_full = bars + 10;              // P of a tile is in tensor memory (one arrival per softmax warp)
-  uint64_t* pv_done = bars + 11;             // P V of a tile is complete: O is consistent, the P buffer is free
-  uint64_t* o_full = bars + 12;
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 13);
+  uint64_t* k_full = bars;                   // [4] keys of a tile have landed (SHARED: keys and values)
+  uint64_t* k_empty = bars + 4;              // [4] S of that tile is complete: the key stage is free
+  uint64_t* v_full = bars + 8;               // [4]
+  uint64_t* v_empty = bars + 12;             // [4] P V of that tile is complete (SHARED: its stage is free)
+  uint64_t* s_full = bars + 16;              // [2] one per S buffer
+  uint64_t* p_full = bars + 18;              // P of a tile is in tensor memory (one arrival per softmax warp)
+  uint64_t* pv_done = bars + 19;             // P V of a tile is complete: O is consistent, the P buffer is free
+  uint64_t* o_full = bars + 20;
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 21);
   float* row_max = reinterpret_cast<float*>(smem + S::OFF_MAX);
 
   rb_pdl_launch_dependents();
@@ -157,8 +174,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     for (int s = 0; s < KV_STAGES; ++s) {
       mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1);
       mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1);
-      mbar_init(&s_full[s], 1);
     }
+    mbar_init(&s_full[0], 1);
+    mbar_init(&s_full[1], 1);
     mbar_init(p_full, 8);
     mbar_init(pv_done, 1);
     mbar_init(o_full, 1);
@@ -176,7 +194,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   const int n_rows = ntok * G;
   const int key_hi = pos0 + ntok - 1;
   const int key_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-  const int kt_begin = key_lo / TILE_KEYS, kt_end = key_hi / TILE_KEYS + 1;
+  int kt_begin = key_lo / TILE_KEYS, kt_end = key_hi / TILE_KEYS + 1;
+  if (p.n_splits > 1) {                                    // this CTA's range of the key tiles (it may be empty)
+    const int per = (kt_end - kt_begin + p.n_splits - 1) / p.n_splits;
+    kt_begin += (int)blockIdx.z * per;
+    kt_end = min(kt_end, kt_begin + per);
+  }
   rb_pdl_wait();                                           // q and the cache come from earlier kernels
 
   tcgen05_fence_before();
@@ -187,7 +210,20 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   // ---- Q rows into tensor memory: the A operand of S = Q K^T is read from there, so that the
   // MMAs fetch only K from shared memory.  Row r lives in lane r, two bfloat16 per column; the two
   // softmax threads of a row write half of it each (rows beyond n_rows are zero).
-  if (warp >= 2) {
+  if (Q_SMEM && warp >= 2) {
+    // rows of 64 values (128 bytes) per block, their 16-byte pieces swizzled as TMA would leave them
+    const int quarter = warp & 3, half = (warp - 2) >> 2, r = quarter * 32 + lane;
+    const int tok = tok0 + r / G, head = kvh * G + r % G;
+    const uint4* src = reinterpret_cast<const uint4*>(p.q + ((int64_t)tok * H + head) * D + half * (D / 2));
+#pragma unroll
+    for (int i = 0; i < D / 16; ++i) {
+      const uint4 v = r < n_rows ? src[i] : make_uint4(0, 0, 0, 0);
+      const int piece = half * (D / 16) + i;               // of 8 values
+      *reinterpret_cast<uint4*>(smem + S::OFF_Q + (piece >> 3) * S::BLOCK + r * 128 + (((piece & 7) ^ (r & 7)) << 4)) = v;
+    }
+    fence_async_shared();
+  }
+  if (!Q_SMEM && warp >= 2) {
     const int quarter = warp & 3, half = (warp - 2) >> 2, r = quarter * 32 + lane;
     uint32_t w[D / 4];                                      // D/2 values = D/4 columns
     if (r < n_rows) {
@@ -227,13 +263,14 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
           const int page = p.page_table[(int64_t)slot * p.max_pages + pi];
           row[h] = (page * p.n_kv_heads + kvh) * p.page_size + key0 % p.page_size;
         }
-        if (!mbar_wait(&k_empty[s], ph, 5)) break;
+        if (!mbar_wait(SHARED ? &v_empty[s] : &k_empty[s], ph, 5)) break;
         mbar_expect_tx(&k_full[s], S::KV_TILE_BYTES);
 #pragma unroll
         for (int b = 0; b < DB; ++b)
 #pragma unroll
           for (int h = 0; h < TILE_KEYS / PIECE; ++h)
             tma_load_2d(smem + S::OFF_K + s * S::KV_TILE_BYTES + b * S::BLOCK + h * (PIECE * 128), &tmK, b * 64, row[h], &k_full[s]);
+        if (SHARED) continue;
         if (!mbar_wait(&v_empty[s], ph, 5)) break;
         mbar_expect_tx(&v_full[s], S::KV_TILE_BYTES);
 #pragma unroll
@@ -263,21 +300,27 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
           for (int k4 = 0; k4 < 4; ++k4) {
             const uint64_t koff = (uint64_t)(k4 * 32 >> 4);
             // A: 16 values of Q = 8 columns of tensor memory; B: the keys' 16 values of block b
-            umma_bf16_ts(tmem_base + (uint32_t)((j & 1) * TILE_KEYS), tmem_base + (uint32_t)(Q_COL + b * 32 + k4 * 8),
+            if (Q_SMEM)
+              umma_bf16(tmem_base + (uint32_t)((j & 1) * TILE_KEYS), smem_desc_sw128(smem_u32(smem + S::OFF_Q) + b * S::BLOCK) + koff,
+                        smem_desc_sw128(k_addr + b * S::BLOCK) + koff, idesc_s, (b > 0 || k4 > 0) ? 1u : 0u);
+            else
+              umma_bf16_ts(tmem_base + (uint32_t)((j & 1) * TILE_KEYS), tmem_base + (uint32_t)(Q_COL + b * 32 + k4 * 8),
                          smem_desc_sw128(k_addr + b * S::BLOCK) + koff, idesc_s, (b > 0 || k4 > 0) ? 1u : 0u);
           }
         tcgen05_commit(&s_full[j & 1]);
-        tcgen05_commit(&k_empty[s]);
+        if (!SHARED) tcgen05_commit(&k_empty[s]);
         return true;
       };
       if (n_tiles > 0) ok = issue_s(0);
       for (int j = 0; j < n_tiles && ok; ++j) {
-        if (j + 1 < n_tiles) ok = issue_s(j + 1);
+        // (SHARED with few stages: where the next tile has not landed yet, this tile's P V goes first)
+        const bool first = !SHARED || j + 1 >= n_tiles || mbar_try_wait(&k_full[(j + 1) % KV_STAGES], ((j + 1) / KV_STAGES) & 1, 0u);
+        if (j + 1 < n_tiles && first) ok = issue_s(j + 1);
         if (!ok) break;
         const int s = j % KV_STAGES;
         ok = mbar_wait(p_full, j & 1, 7);                    // P of this tile is in tensor memory
         if (!ok) break;
-        ok = mbar_wait(&v_full[s], (j / KV_STAGES) & 1, 6);
+        if (!SHARED) ok = mbar_wait(&v_full[s], (j / KV_STAGES) & 1, 6);
         if (!ok) break;
         tcgen05_fence_after();
         const uint32_t v_addr = smem_u32(smem + S::OFF_V + s * S::KV_TILE_BYTES);
@@ -290,6 +333,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         }
         tcgen05_commit(&v_empty[s]);
         tcgen05_commit(pv_done);
+        if (!first) ok = issue_s(j + 1);
       }
       tcgen05_commit(o_full);
     }
@@ -309,7 +353,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     constexpr int HK = TILE_KEYS / 2;                        // keys per thread and tile
     constexpr int HD = D / 2;                                // columns of O per thread
     float m_run = -INFINITY, l_run = 0.f;
-    if (p.sinks != nullptr && row_ok) {
+    if (p.sinks != nullptr && row_ok && blockIdx.z == 0) {
       // the sink: one more term of the row's denominator, counted by one of the row's two threads; both start from
       // the same reference, so that their exponents agree
       m_run = p.sinks[kvh * G + r % G] * 1.4426950408889634f;
@@ -446,7 +490,27 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     row_max[half * ROWS + r] = l_run;
     asm volatile("bar.sync 1, 256;" ::: "memory");
     const float l_all = l_run + row_max[(half ^ 1) * ROWS + r];
-    if (!failed) {
+    if (!failed && p.n_splits > 1) {
+      const int tok = tok0 + r / G, head = kvh * G + r % G;
+      const int64_t base = ((int64_t)tok * H + head) * p.n_splits + blockIdx.z;
+      const bool any = kt_end > kt_begin;                    // without keys O was never written
+      if (row_ok && half == 0) { p.part_ml[base * 2] = m_run; p.part_ml[base * 2 + 1] = l_all; }
+      float* dst = p.part_o + base * D + half * HD;
+#pragma unroll 1
+      for (int c = 0; c < HD; c += 16) {
+        uint32_t o[16];
+        __syncwarp();
+        tmem_ld16(lane_addr + O_COL + half * HD + c, o);
+        tmem_ld_wait();
+        if (row_ok) {
+#pragma unroll
+          for (int i = 0; i < 16; i += 4)
+            *reinterpret_cast<float4*>(dst + c + i) =
+                any ? make_float4(__uint_as_float(o[i]), __uint_as_float(o[i + 1]), __uint_as_float(o[i + 2]), __uint_as_float(o[i + 3]))
+                    : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+      }
+    } else if (!failed) {
       const float inv = l_all > 0.f ? 1.0f / l_all : 0.f;
       const int tok = tok0 + r / G, head = kvh * G + r % G;
       __nv_bfloat16* dst = p.out + ((int64_t)tok * H + head) * D + half * HD;
@@ -476,15 +540,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   }
 }
 
-template <int D>
+template <int D, bool SHARED>
 int launch_tc(const CUtensorMap& tk, const CUtensorMap& tv, const TcAttnParams& p, int Kh, cudaStream_t stream) {
-  auto kernel = attn_tc_kernel<D>;
-  constexpr int smem = TcSmem<D>::BYTES;
+  auto kernel = attn_tc_kernel<D, SHARED>;
+  constexpr int smem = TcSmem<D, SHARED>::BYTES;
   static RbOncePerDevice configured;
   if (configured.first()) {
     RB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   }
-  RB_LAUNCH("rb_attention_prefill_tc", (kernel), dim3(Kh, p.n_tiles), THREADS, smem, stream, tk, tv, p);
+  RB_LAUNCH("rb_attention_prefill_tc", (kernel), dim3(Kh, p.n_tiles, p.n_splits), THREADS, smem, stream, tk, tv, p);
   return 0;
 }
 
@@ -572,24 +636,39 @@ RB_EXPORT int rb_attention_decode_tma(void* out, const void* q, const void* cach
 int rb_attention_tc_error_flag(int* value, int reset) { return rb_file_error_flag(value, reset); }
 int rb_attention_tc_error_flag_address(int** out) { return rb_file_error_flag_address(out); }
 
-// Whether the tensor-memory prefill kernel takes these sizes.
-RB_EXPORT int rb_attention_prefill_tc_supports(int H, int Kh, int D, int page_size) {
+// Whether the tensor-memory kernel takes these sizes; shared: keys and values are the same rows.
+RB_EXPORT int rb_attention_prefill_tc_supports(int H, int Kh, int D, int page_size, int shared) {
   if (Kh <= 0 || H % Kh) return 0;
   const int G = H / Kh;
-  return (D == 64 || D == 128) && page_size % PIECE == 0 && G <= ROWS;
+  return (D == 64 || D == 128 || (shared && (D == 192 || D == 256))) && page_size % PIECE == 0 && G <= ROWS;
 }
 
-// Prefill over the paged cache: tile i covers tile_ntok[i] <= 128/G tokens of one sequence starting
-// at batch row tile_tok0[i].  cache_k / cache_v: [n_pages, Kh, page_size, D] bfloat16.
+// Parts to cut a step's key tiles into: `row_tiles` tiles of rows times kv heads, the longest sequence `context`
+// positions.  One where the row tiles fill the SMs; else as many as fit them, none with less than one key tile.
+RB_EXPORT int rb_attention_prefill_tc_parts(int row_tiles, int Kh, int context) {
+  const int ctas = row_tiles * Kh, key_tiles = (context + TILE_KEYS - 1) / TILE_KEYS;
+  if (ctas <= 0 || key_tiles <= 1) return 1;
+  const int room = rb_sm_count() / ctas;
+  int parts = room < key_tiles ? room : key_tiles;
+  if (parts > 16) parts = 16;                        // the merge reads 16 parts at a time
+  return parts < 1 ? 1 : parts;
+}
+
+// Attention over the paged cache: tile i covers tile_ntok[i] <= 128/G tokens of one sequence starting
+// at batch row tile_tok0[i].  cache_k / cache_v: [n_pages, Kh, page_size, D] bfloat16 (the same pointer: SHARED).
+// n_splits > 1: part_o [T, H, n_splits, D] and part_ml [T, H, n_splits, 2] float32 are scratch, T the step's rows.
 RB_EXPORT int rb_attention_prefill_tc(void* out, const void* q, const void* cache_k, const void* cache_v,
                                       long long n_pages, const int* page_table, int max_pages, int page_size,
                                       const int* tok_pos, const int* tok_slot, const int* tile_tok0,
                                       const int* tile_ntok, int n_tiles, int H, int Kh, int D, float scale,
-                                      int window, cudaStream_t stream) {
+                                      int window, float* part_o, float* part_ml, int n_splits, int T, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
+  const bool shared = cache_k == cache_v;
   RB_REQUIRE(n_tiles <= 65535, "rb_attention_prefill_tc: %d tiles in one launch", n_tiles);
-  RB_REQUIRE(rb_attention_prefill_tc_supports(H, Kh, D, page_size),
+  RB_REQUIRE(rb_attention_prefill_tc_supports(H, Kh, D, page_size, shared ? 1 : 0),
              "rb_attention_prefill_tc: sizes H=%d Kh=%d D=%d page=%d not supported", H, Kh, D, page_size);
+  RB_REQUIRE(n_splits >= 1 && n_splits <= 65535 && (n_splits == 1 || (part_o && part_ml && T > 0)),
+             "rb_attention_prefill_tc: %d parts want scratch", n_splits);
   CUtensorMap tk, tv;
   const long long rows = n_pages * Kh * page_size;
   if (rb_get_tensor_map(&tk, cache_k, rows, D, D, PIECE) != 0) return -1;
@@ -600,6 +679,13 @@ RB_EXPORT int rb_attention_prefill_tc(void* out, const void* q, const void* cach
   p.tok_pos = tok_pos; p.tok_slot = tok_slot; p.tile_tok0 = tile_tok0; p.tile_ntok = tile_ntok; p.n_tiles = n_tiles;
   p.H = H; p.G = H / Kh; p.scale_log2 = scale * 1.4426950408889634f; p.window = window;
   { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; }
-  if (D == 64) return launch_tc<64>(tk, tv, p, Kh, stream);
-  return launch_tc<128>(tk, tv, p, Kh, stream);
+  p.part_o = part_o; p.part_ml = part_ml; p.n_splits = n_splits;
+  int rc;
+  if (!shared) rc = D == 64 ? launch_tc<64, false>(tk, tv, p, Kh, stream) : launch_tc<128, false>(tk, tv, p, Kh, stream);
+  else if (D == 64) rc = launch_tc<64, true>(tk, tv, p, Kh, stream);
+  else if (D == 128) rc = launch_tc<128, true>(tk, tv, p, Kh, stream);
+  else if (D == 192) rc = launch_tc<192, true>(tk, tv, p, Kh, stream);
+  else rc = launch_tc<256, true>(tk, tv, p, Kh, stream);
+  if (rc != 0 || n_splits == 1) return rc;
+  return rb_attention_combine(out, part_o, part_ml, T, H, D, n_splits, stream);
 }

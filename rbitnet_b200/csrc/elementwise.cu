@@ -234,31 +234,31 @@ RB_EXPORT int rb_rmsnorm(void* out, int out_dtype, const float* x, const float* 
 
 // ---------------------------------------------------------------- rotation + cache append
 // ---------------------------------------------------------------- tanh in place of a norm
-// out = w * tanh(alpha * x) + b, value by value.  VEC: four values a thread and turn.
-template <typename TO, bool VEC>
+// out = w * tanh(alpha * x) + b, value by value.  A thread keeps its V columns (their w and b in registers) and takes
+// every gridDim.y-th row.
+template <typename TO, int V>
 __global__ void __launch_bounds__(256) tanh_norm_kernel(TO* __restrict__ out, const float* __restrict__ x,
                                                         const float* __restrict__ w, const float* __restrict__ b,
-                                                        float alpha, int64_t n, int E) {
+                                                        float alpha, int T, int E) {
   rb_pdl_launch_dependents();
+  const int e = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  float ww[4], bb[4];
+  if (e < E) {                                       // (weights: never written by a kernel)
+    if (V == 4) { rb_load4(w + e, ww); rb_load4(b + e, bb); }
+    else { ww[0] = w[e]; bb[0] = b[e]; }
+  }
   rb_pdl_wait();
-  const int64_t first = (int64_t)blockIdx.x * blockDim.x + threadIdx.x, step = (int64_t)gridDim.x * blockDim.x;
-  if (VEC) {
-    const int E4 = E / 4;
-    for (int64_t i = first; i < n / 4; i += step) {
-      const int e = (int)(i % E4) * 4;
-      float v[4], ww[4], bb[4];
-      rb_load4(x + 4 * i, v);
-      rb_load4(w + e, ww);
-      rb_load4(b + e, bb);
+  if (e >= E) return;
+#pragma unroll 4
+  for (int t = blockIdx.y; t < T; t += gridDim.y) {
+    const int64_t at = (int64_t)t * E + e;
+    float v[4];
+    if (V == 4) rb_load4(x + at, v);
+    else v[0] = x[at];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) v[j] = fmaf(ww[j], tanhf(alpha * v[j]), bb[j]);
-      rb_store4(out + 4 * i, v);
-    }
-  } else {
-    for (int64_t i = first; i < n; i += step) {
-      const int e = (int)(i % E);
-      out[i] = rb_from_float<TO>(fmaf(w[e], tanhf(alpha * x[i]), b[e]));
-    }
+    for (int j = 0; j < V; ++j) v[j] = fmaf(ww[j], rb_norm_tanh<TO>(alpha * v[j]), bb[j]);
+    if (V == 4) rb_store4(out + at, v);
+    else out[at] = rb_from_float<TO>(v[0]);
   }
 }
 
@@ -266,14 +266,16 @@ RB_EXPORT int rb_tanh_norm(void* out, int out_dtype, const float* x, const float
                            cudaStream_t stream) {
   if (T == 0) return 0;
   RB_REQUIRE(T > 0 && E > 0, "rb_tanh_norm: bad sizes T=%d E=%d", T, E);
-  const int64_t n = (int64_t)T * E;
   const bool vec = E % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)b % 16 == 0 &&
                    (uintptr_t)out % 16 == 0;
-  const int64_t want = ((vec ? n / 4 : n) + 255) / 256, most = (int64_t)rb_sm_count() * 8;
-  const int blocks = (int)(want < most ? want : most);
-#define GO(TO, V) RB_LAUNCH("tanh_norm_kernel", (tanh_norm_kernel<TO, V>), blocks, 256, 0, stream, (TO*)out, x, w, b, alpha, n, E)
-  if (out_dtype == RB_F32) { if (vec) GO(float, true); else GO(float, false); }
-  else if (out_dtype == RB_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }
+  const int items = vec ? E / 4 : E, threads = items >= 256 ? 256 : (items >= 128 ? 128 : 64);
+  const int bx = (items + threads - 1) / threads;
+  int by = (rb_sm_count() * (2048 / threads) + bx - 1) / bx;            // every SM's threads once
+  if (by > T) by = T;
+  const dim3 grid(bx, by);
+#define GO(TO, V) RB_LAUNCH("tanh_norm_kernel", (tanh_norm_kernel<TO, V>), grid, threads, 0, stream, (TO*)out, x, w, b, alpha, T, E)
+  if (out_dtype == RB_F32) { if (vec) GO(float, 4); else GO(float, 1); }
+  else if (out_dtype == RB_BF16) { if (vec) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 1); }
   else RB_FAIL("rb_tanh_norm: unknown dtype %d", out_dtype);
 #undef GO
   RB_CHECK_LAUNCH("rb_tanh_norm");

@@ -153,54 +153,55 @@ __global__ void __launch_bounds__(256) gemm_simple_large_kernel(TC* __restrict__
   }
 }
 
-// Few rows (a decode step) times one matrix per head: a warp makes one output of one head for up to eight rows at a
-// time, its lanes sharing K, so that the head's matrix is read once and 8 heads x N / 8 blocks are at work instead of
-// a few tiles.  float32 sums (a lane's share in ascending order, then the lanes' shares added up).  Head h's input
-// values start at column h * head_a of a row.  VEC: four values a load.
-constexpr int FEW_ROWS = 8;
+// Few rows (a decode step) times one matrix per head: a warp makes four outputs of one head for up to eight rows at a
+// time, its lanes sharing K, so that the head's matrix is read once, the rows once for four outputs, and heads x N / 16
+// blocks are at work instead of a few tiles.  float32 sums (a lane's share in ascending order, then the lanes' shares in a
+// fixed tree).  Head h's input values start at column h * head_a of a row.  VEC: four values a load.
+constexpr int FEW_ROWS = 8, FEW_OUTS = 4, FEW_WARPS = 4;
 template <typename TA, typename TC, bool VEC>
-__global__ void __launch_bounds__(256) per_head_few_rows_kernel(TC* __restrict__ C, int64_t ldc, const TA* __restrict__ A,
-                                                               int64_t lda, int head_a, const TA* __restrict__ W, int M,
-                                                               int N, int K, Tail tail) {
+__global__ void __launch_bounds__(FEW_WARPS * 32) per_head_few_rows_kernel(
+    TC* __restrict__ C, int64_t ldc, const TA* __restrict__ A, int64_t lda, int head_a, const TA* __restrict__ W, int M, int N,
+    int K, Tail tail) {
   rb_pdl_launch_dependents();
   rb_pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int h = blockIdx.y, n = blockIdx.x * 8 + warp;
-  if (n >= N) return;
-  const TA* w = W + ((int64_t)h * N + n) * K;
+  const int h = blockIdx.y, n0 = (blockIdx.x * FEW_WARPS + warp) * FEW_OUTS;
+  if (n0 >= N) return;
+  const TA* w = W + ((int64_t)h * N + n0) * K;
   const TA* a = A + (int64_t)h * head_a;
   for (int m0 = 0; m0 < M; m0 += FEW_ROWS) {
-    float acc[FEW_ROWS];
+    float acc[FEW_OUTS * FEW_ROWS];
 #pragma unroll
-    for (int i = 0; i < FEW_ROWS; ++i) acc[i] = 0.f;
-    if (VEC) {
-      for (int k = lane * 4; k < K; k += 128) {
-        float wv[4];
-        rb_load4(w + k, wv);
+    for (int i = 0; i < FEW_OUTS * FEW_ROWS; ++i) acc[i] = 0.f;
+    constexpr int V = VEC ? 4 : 1;
+    for (int k = lane * V; k < K; k += 32 * V) {
+      float wv[FEW_OUTS][4];
 #pragma unroll
-        for (int i = 0; i < FEW_ROWS; ++i) {
-          if (m0 + i < M) {
-            float av[4];
-            rb_load4(a + (int64_t)(m0 + i) * lda + k, av);
-#pragma unroll
-            for (int j = 0; j < 4; ++j) acc[i] = fmaf(av[j], wv[j], acc[i]);
-          }
+      for (int o = 0; o < FEW_OUTS; ++o) {
+        const bool have = n0 + o < N;
+        if (VEC) {
+          if (have) rb_load4(w + (int64_t)o * K + k, wv[o]);
+          else wv[o][0] = wv[o][1] = wv[o][2] = wv[o][3] = 0.f;
+        } else {
+          wv[o][0] = have ? rb_to_float<TA>(w[(int64_t)o * K + k]) : 0.f;
         }
       }
-    } else {
-      for (int k = lane; k < K; k += 32) {
-        const float wv = rb_to_float<TA>(w[k]);
 #pragma unroll
-        for (int i = 0; i < FEW_ROWS; ++i)
-          if (m0 + i < M) acc[i] = fmaf(rb_to_float<TA>(a[(int64_t)(m0 + i) * lda + k]), wv, acc[i]);
+      for (int i = 0; i < FEW_ROWS; ++i) {
+        if (m0 + i < M) {
+          float av[4];
+          if (VEC) rb_load4(a + (int64_t)(m0 + i) * lda + k, av);
+          else av[0] = rb_to_float<TA>(a[(int64_t)(m0 + i) * lda + k]);
+#pragma unroll
+          for (int o = 0; o < FEW_OUTS; ++o)
+#pragma unroll
+            for (int j = 0; j < V; ++j) acc[o * FEW_ROWS + i] = fmaf(av[j], wv[o][j], acc[o * FEW_ROWS + i]);
+        }
       }
     }
-#pragma unroll
-    for (int i = 0; i < FEW_ROWS; ++i) {
-      const float v = rb_warp_sum(acc[i]);
-      if (lane == 0 && m0 + i < M)
-        C[(int64_t)(m0 + i) * ldc + (int64_t)h * N + n] = rb_from_float<TC>(finished(tail, v, m0 + i, n, h));
-    }
+    const float v = rb_warp_sum32(acc, lane);
+    const int n = n0 + lane / FEW_ROWS, m = m0 + lane % FEW_ROWS;
+    if (n < N && m < M) C[(int64_t)m * ldc + (int64_t)h * N + n] = rb_from_float<TC>(finished(tail, v, m, n, h));
   }
 }
 
@@ -228,13 +229,13 @@ RB_EXPORT int rb_per_head_few_rows(void* C, int64_t ldc, int c_dtype, const void
   if (M == 0 || N == 0 || H == 0) return 0;
   RB_REQUIRE(M > 0 && N > 0 && K > 0 && H > 0 && H <= 65535 && head_a >= K, "rb_per_head_few_rows: bad sizes M=%d H=%d N=%d K=%d (%d apart)",
              M, H, N, K, head_a);
-  const dim3 grid((N + 7) / 8, H);
+  const dim3 grid((N + FEW_OUTS * FEW_WARPS - 1) / (FEW_OUTS * FEW_WARPS), H);
   const int elem = a_dtype == RB_F32 ? 4 : 2;
   const bool vec = K % 4 == 0 && head_a % 4 == 0 && lda % 4 == 0 && (uintptr_t)A % (4 * elem) == 0 && (uintptr_t)W % (4 * elem) == 0;
 #define LAUNCH(TA, TC)                                                                                                  \
   do {                                                                                                                  \
-    if (vec) RB_LAUNCH("per_head_few_rows_kernel", (per_head_few_rows_kernel<TA, TC, true>), grid, 256, 0, stream, (TC*)C, ldc, (const TA*)A, lda, head_a, (const TA*)W, M, N, K, tail); \
-    else RB_LAUNCH("per_head_few_rows_kernel", (per_head_few_rows_kernel<TA, TC, false>), grid, 256, 0, stream, (TC*)C, ldc, (const TA*)A, lda, head_a, (const TA*)W, M, N, K, tail);    \
+    if (vec) RB_LAUNCH("per_head_few_rows_kernel", (per_head_few_rows_kernel<TA, TC, true>), grid, FEW_WARPS * 32, 0, stream, (TC*)C, ldc, (const TA*)A, lda, head_a, (const TA*)W, M, N, K, tail); \
+    else RB_LAUNCH("per_head_few_rows_kernel", (per_head_few_rows_kernel<TA, TC, false>), grid, FEW_WARPS * 32, 0, stream, (TC*)C, ldc, (const TA*)A, lda, head_a, (const TA*)W, M, N, K, tail);    \
   } while (0)
   if (a_dtype == RB_F32 && c_dtype == RB_F32) LAUNCH(float, float);
   else if (a_dtype == RB_BF16 && c_dtype == RB_F32) LAUNCH(__nv_bfloat16, float);

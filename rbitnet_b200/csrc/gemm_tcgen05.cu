@@ -434,6 +434,15 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         for (int j = 0; j < 16; ++j) into[j] = j < left ? src[(int64_t)j * p.ldc] : 0.f;
       };
       if (EPI == EPI_ADD && !TMA_EPI && !p.cluster) fetch_old(0, ahead);
+      // the same for the gate's values of a product with one matrix per head
+      auto fetch_gate = [&](int c, float* into) {
+        const int left = n_ok ? p.n_tokens - (t0 + c) : 0;
+        const float* src = p.gate + (int64_t)(t0 + c) * p.gate_ld + (s.w0 + row);
+#pragma unroll
+        for (int j = 0; j < 16; ++j) into[j] = j < left ? src[(int64_t)j * p.gate_ld] : 0.f;
+      };
+      const bool gated = EPI == EPI_STORE && BN == 64 && p.gate != nullptr;      // (token tiles of 64 only)
+      if (gated) fetch_gate(0, ahead);
       bool ok = true;
       if (lane == 0) ok = mbar_wait(&accum_full[b], (li / NBUF) & 1, 3);
       ok = __shfl_sync(0xffffffffu, ok, 0);
@@ -506,17 +515,9 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               store_out<OutT>(dst + j * OUT_COLS, gated_value(p, g, up));
             }
           } else {
-            float gate[16];
-            if (EPI == EPI_STORE && p.gate != nullptr) {
-              const int left = n_ok ? p.n_tokens - (t0 + c) : 0;
-              const float* src = p.gate + (int64_t)(t0 + c) * p.gate_ld + (s.w0 + row);
-#pragma unroll
-              for (int j = 0; j < 16; ++j) gate[j] = j < left ? src[(int64_t)j * p.gate_ld] : 0.f;
-            }
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
-              float v = __uint_as_float(r[j]) * p.alpha + bias_n;
-              if (EPI == EPI_STORE && p.gate != nullptr) v = __fdividef(v, 1.0f + __expf(-gate[j]));
+              const float v = __uint_as_float(r[j]) * p.alpha + bias_n;
               store_out<OutT>(box + j * OUT_COLS + row, EPI == EPI_STORE ? stored_value(p, v) : v);
             }
           }
@@ -579,16 +580,16 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           } else {
             OutT* dst = (OutT*)p.C + (int64_t)(t0 + c) * p.ldc + s.c0 + n;
             float gate[16];
-            if (p.gate != nullptr) {
-              const float* src = p.gate + (int64_t)(t0 + c) * p.gate_ld + (s.w0 + row);
+            if (gated) {
 #pragma unroll
-              for (int j = 0; j < 16; ++j) gate[j] = j < t_left ? src[(int64_t)j * p.gate_ld] : 0.f;
+              for (int j = 0; j < 16; ++j) gate[j] = ahead[j];
+              if (c + 16 < BN && t0 + c + 16 < p.n_tokens) fetch_gate(c + 16, ahead);
             }
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               if (j < t_left) {
                 float v = __uint_as_float(r[j]) * (normed ? p.alpha * norm_r[t0 + c + j] : p.alpha) + bias_n;
-                if (p.gate != nullptr) v = __fdividef(v, 1.0f + __expf(-gate[j]));
+                if (gated) v = __fdividef(v, 1.0f + __expf(-gate[j]));
                 store_out<OutT>(dst + (int64_t)j * p.ldc, stored_value(p, v));
               }
           }
@@ -757,7 +758,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                 ((float*)p.C)[at] = now;
                 if (emit)
                   p.emit_xb[(int64_t)(t0 + col[h]) * p.emit_ld + n] =
-                      __float2bfloat16_rn(emit_tanh ? fmaf(g_n, tanhf(p.emit_alpha * now), b_n) : now * g_n);
+                      __float2bfloat16_rn(emit_tanh ? fmaf(g_n, rb_norm_tanh<__nv_bfloat16>(p.emit_alpha * now), b_n) : now * g_n);
               } else {
                 store_out<OutT>((OutT*)p.C + at, stored_value(p, v));
               }
@@ -1178,7 +1179,7 @@ RB_EXPORT int rb_gemm_tc_bias(const float* bias) {
 // The next stored product (epilogue 0, one split) of this thread multiplies by one matrix per head (see GemmParams): W
 // holds heads * n_out rows, X and C the heads' columns head_x and head_c apart.  A token tile of 128 and more writes
 // whole boxes of 128 columns, so it needs head_c >= n_out rounded up to 128; what it leaves in columns n_out .. of a head
-// is not defined.  gate: null, or float32 with column h * n_out + n for value n of head h.
+// is not defined.  gate (token tiles of 64 only): null, or float32 with column h * n_out + n for value n of head h.
 RB_EXPORT int rb_gemm_tc_per_head(int heads, int head_x, int head_c, const float* gate, long long gate_ld) {
   RB_REQUIRE(heads > 0 && head_x > 0 && head_c > 0, "rb_gemm_tc_per_head: bad sizes heads=%d, %d and %d apart", heads, head_x, head_c);
   t_store.heads = heads; t_store.head_x = head_x; t_store.head_c = head_c; t_store.gate = gate; t_store.gate_ld = gate_ld;
@@ -1268,6 +1269,7 @@ static int gemm_tc(void* C, int64_t ldc, int c_dtype, const void* X, int64_t ldx
   if (store.heads > 0 && plan.bn >= 128 && ((n_out + BM - 1) / BM * BM > store.head_c || store.head_c % 8 != 0))
     plan = plan_for_tile(n_tokens, n_out, K, 64, rb_sm_count(), false);
   const int bn = plan.bn;
+  RB_REQUIRE(store.heads == 0 || store.gate == nullptr || bn == 64, "rb_gemm_tc: a gate per head's value wants a token tile of 64");
   RB_REQUIRE(epilogue != EPI_GATED || (n_out % 32 == 0 && n_features > 0 && n_features <= n_out / 2),
              "rb_gemm_tc: the gated product wants rows in blocks of 32 (%d rows, %d features)", n_out, n_features);
   // A last round of few tiles.  Tiles in turn pay a whole round of the SMs for it (2,048 tokens times

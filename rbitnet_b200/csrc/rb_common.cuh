@@ -136,6 +136,25 @@ __device__ __forceinline__ void rb_store4(__nv_bfloat16* p, const float (&v)[4])
   *reinterpret_cast<uint2*>(p) = raw;
 }
 
+__device__ __forceinline__ void rb_store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void rb_store2(__nv_bfloat16* p, float a, float b) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+}
+
+// ---------------------------------------------------------------- tanh of a norm's rows
+// tanh with two of the hardware's special functions: 1 - 2 / (1 + e^(2y)), and near zero, where that difference would
+// lose digits, the first terms of tanh's series.  Error a few units of float32, far below the rounding to bfloat16 of
+// the rows it is used for (float32 rows take tanhf).
+__device__ __forceinline__ float rb_tanh_for_bf16(float y) {
+  const float y2 = y * y;
+  const float near = y * fmaf(y2, fmaf(y2, fmaf(y2, -17.0f / 315.0f, 2.0f / 15.0f), -1.0f / 3.0f), 1.0f);
+  const float far = 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * fminf(y, 40.0f)));
+  return fabsf(y) < 0.15f ? near : far;
+}
+template <typename TO> __device__ __forceinline__ float rb_norm_tanh(float y);
+template <> __device__ __forceinline__ float rb_norm_tanh<float>(float y) { return tanhf(y); }
+template <> __device__ __forceinline__ float rb_norm_tanh<__nv_bfloat16>(float y) { return rb_tanh_for_bf16(y); }
+
 // ---------------------------------------------------------------- reductions
 __device__ __forceinline__ float rb_warp_sum(float v) {
 #pragma unroll
@@ -146,6 +165,37 @@ __device__ __forceinline__ float rb_warp_max(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
+}
+
+// 32 sums over the warp's lanes at once: lane l gets the sum of everybody's v[l] (31 exchanges in all, where 32 single
+// sums take 160; every sum is taken in the same fixed tree).
+__device__ __forceinline__ float rb_warp_sum32(float (&v)[32], int lane) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool up = (lane & o) != 0;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float keep = up ? v[i + o] : v[i], send = up ? v[i] : v[i + o];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+    }
+  }
+  return v[0];
+}
+// Two sums over a block at once (`scratch`: 66 floats of shared memory).
+__device__ __forceinline__ float2 rb_block_sum2(float a, float b, float* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int nwarps = (blockDim.x + 31) >> 5;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    a += __shfl_xor_sync(0xffffffffu, a, o);
+    b += __shfl_xor_sync(0xffffffffu, b, o);
+  }
+  __syncthreads();
+  if (lane == 0) { scratch[warp] = a; scratch[33 + warp] = b; }
+  __syncthreads();
+  float ta = 0.f, tb = 0.f;
+  for (int w = 0; w < nwarps; ++w) { ta += scratch[w]; tb += scratch[33 + w]; }
+  return make_float2(ta, tb);
 }
 
 // Sum over a block of up to 1024 threads; `scratch` holds 33 floats of shared

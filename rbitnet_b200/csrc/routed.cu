@@ -402,8 +402,9 @@ __global__ void combine_kernel(float* __restrict__ x, int64_t ldx, const float* 
   const float sg = tail.shared != nullptr ? 1.0f / (1.0f + expf(-tail.gate[(int64_t)t * tail.ldg])) : 0.f;
   if (vec4) {
     // four columns a thread: 16-byte loads of the experts' rows and of the residual stream
-    for (int c = threadIdx.x * 4; c < E; c += blockDim.x * 4) {
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4; c < E; c += gridDim.y * blockDim.x * 4) {
       float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
       for (int j = 0; j < top; ++j) {
         const int r = pos[(int64_t)t * top + j];
         const float w = weights != nullptr ? weights[(int64_t)t * top + j] : 1.0f;
@@ -432,13 +433,13 @@ __global__ void combine_kernel(float* __restrict__ x, int64_t ldx, const float* 
         rb_load4(tail.norm_w + c, ww);
         rb_load4(tail.norm_b + c, bb);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) acc[i] = fmaf(ww[i], tanhf(tail.norm_alpha * acc[i]), bb[i]);
+        for (int i = 0; i < 4; ++i) acc[i] = fmaf(ww[i], rb_norm_tanh<T>(tail.norm_alpha * acc[i]), bb[i]);
         rb_store4((T*)tail.norm_out + (int64_t)t * E + c, acc);
       }
     }
     return;
   }
-  for (int c = threadIdx.x; c < E; c += blockDim.x) {
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < E; c += gridDim.y * blockDim.x) {
     float acc = 0.f;
     for (int j = 0; j < top; ++j) {
       const int r = pos[(int64_t)t * top + j];
@@ -451,7 +452,7 @@ __global__ void combine_kernel(float* __restrict__ x, int64_t ldx, const float* 
     const float now = accumulate ? *dst + acc : acc;
     *dst = now;
     if (tail.norm_w != nullptr)
-      ((T*)tail.norm_out)[(int64_t)t * E + c] = rb_from_float<T>(fmaf(tail.norm_w[c], tanhf(tail.norm_alpha * now), tail.norm_b[c]));
+      ((T*)tail.norm_out)[(int64_t)t * E + c] = rb_from_float<T>(fmaf(tail.norm_w[c], rb_norm_tanh<T>(tail.norm_alpha * now), tail.norm_b[c]));
   }
 }
 
@@ -695,10 +696,14 @@ RB_EXPORT int rb_routed_combine(float* x, int64_t ldx, const float* y, const voi
                    (uintptr_t)h % (4 * elem) == 0 && (uintptr_t)tail.shared % 16 == 0 && (uintptr_t)tail.norm_w % 16 == 0 &&
                    (uintptr_t)tail.norm_b % 16 == 0 && (uintptr_t)tail.norm_out % (4 * elem) == 0;
   const int threads = vec4 ? (E >= 1024 ? 256 : (E >= 512 ? 128 : 64)) : (E >= 256 ? 256 : (E >= 128 ? 128 : 64));
+  // few rows: a row's columns over several blocks
+  int ny = 1;
+  if (T <= rb_sm_count()) ny = (E + threads * (vec4 ? 4 : 1) - 1) / (threads * (vec4 ? 4 : 1));
+  const dim3 grid(T, ny);
   if (h_dtype == RB_F32)
-    RB_LAUNCH("combine_kernel", (combine_kernel<float>), T, threads, 0, stream, x, ldx, y, (const float*)h, ldh, pos, weights, top, E, accumulate, vec4, tail);
+    RB_LAUNCH("combine_kernel", (combine_kernel<float>), grid, threads, 0, stream, x, ldx, y, (const float*)h, ldh, pos, weights, top, E, accumulate, vec4, tail);
   else if (h_dtype == RB_BF16)
-    RB_LAUNCH("combine_kernel", (combine_kernel<__nv_bfloat16>), T, threads, 0, stream, x, ldx, y, (const __nv_bfloat16*)h, ldh, pos, weights, top, E, accumulate, vec4, tail);
+    RB_LAUNCH("combine_kernel", (combine_kernel<__nv_bfloat16>), grid, threads, 0, stream, x, ldx, y, (const __nv_bfloat16*)h, ldh, pos, weights, top, E, accumulate, vec4, tail);
   else
     RB_FAIL("rb_routed_combine: unknown dtype %d", h_dtype);
   RB_CHECK_LAUNCH("rb_routed_combine");

@@ -89,7 +89,7 @@ _SIGNATURES = {
     "rb_error_flag_addresses": [P, P],
     "rb_attention_prefill": [P, P, P, P, P, I, I, P, P, P, P, I, I, I, I, F, I, P],
     "rb_attention_decode": [P, P, P, P, P, I, I, P, P, I, I, I, I, F, I, P, P, I, P],
-    "rb_attention_prefill_tc": [P, P, P, P, L, P, I, I, P, P, P, P, I, I, I, I, F, I, P],
+    "rb_attention_prefill_tc": [P, P, P, P, L, P, I, I, P, P, P, P, I, I, I, I, F, I, P, P, I, I, P],
     "rb_attention_decode_tma": [P, P, P, P, L, P, I, I, P, P, I, I, I, I, F, I, P, P, I, P],
     "rb_attention_decode_static": [P, P, P, P, P, I, I, P, P, I, I, I, I, F, I, I, P],
     "rb_attention_next": [P, F],
@@ -125,7 +125,8 @@ class KernelLibrary:
         for name, argtypes in _SIGNATURES.items():
             self.declare(name, argtypes)
         self.declare("rb_attention_tiled_supports", [I, I, I, I, I])
-        self.declare("rb_attention_prefill_tc_supports", [I, I, I, I])
+        self.declare("rb_attention_prefill_tc_supports", [I, I, I, I, I])
+        self.declare("rb_attention_prefill_tc_parts", [I, I, I])
         self.declare("rb_gemm_tc_qkv_supports", [I, I, I])
         self.declare("rb_attention_decode_tma_supports", [I, I, I, I])
         self.declare("rb_attention_decode_tma_parts", [I, I, I])

@@ -528,9 +528,14 @@ class CudaOps:
             if sinks is not None:
                 self._check(sinks, torch.float32, "attention sinks")
             self.lib.call("rb_attention_next", _ptr(sinks), float(softcap), launches=0)
-        if self.dtype == torch.bfloat16 and meta.single_token and \
-                self.lib.raw("rb_attention_tiled_supports")(H, Kh, D, view.page_size, 1):
-            on_tma = self.decode_on_tma and self.lib.raw("rb_attention_decode_tma_supports")(H, Kh, D, view.page_size)
+        # keys and values that are the same rows (attention through latents) let the tcgen05 kernel take wider heads
+        shared = 1 if view.k.data_ptr() == view.v.data_ptr() else 0
+        on_tc = self.dtype == torch.bfloat16 and self.prefill_on_tcgen05 and \
+            self.lib.raw("rb_attention_prefill_tc_supports")(H, Kh, D, view.page_size, shared)
+        few = self.dtype == torch.bfloat16 and meta.single_token and \
+            self.lib.raw("rb_attention_tiled_supports")(H, Kh, D, view.page_size, 1)
+        on_tma = few and self.decode_on_tma and self.lib.raw("rb_attention_decode_tma_supports")(H, Kh, D, view.page_size)
+        if few and (on_tma or not (on_tc and shared)):
             if on_tma:
                 n_splits = self.lib.raw("rb_attention_decode_tma_parts")(T * Kh, max(1, -(-meta.max_context // 64)), D)
             else:
@@ -553,13 +558,19 @@ class CudaOps:
                               _ptr(view.page_table), view.max_pages, view.page_size, _ptr(meta.tok_pos),
                               _ptr(meta.tok_slot), T, H, Kh, D, float(scale), win, _ptr(part_o), _ptr(part_ml),
                               n_splits, self._stream(), launches=2 if n_splits > 1 else 1)
-        elif self.dtype == torch.bfloat16 and self.prefill_on_tcgen05 and \
-                self.lib.raw("rb_attention_prefill_tc_supports")(H, Kh, D, view.page_size):
+        elif on_tc:
             tok0, ntok, n_tiles = self._prefill_tiles(meta, 128 // (H // Kh))
+            parts, part_o, part_ml = 1, None, None
+            if meta.single_token:
+                # a decode step whose heads the decode kernels do not take: few row tiles, the keys cut into parts
+                parts = self.lib.raw("rb_attention_prefill_tc_parts")(n_tiles, Kh, int(meta.max_context))
+            if parts > 1:
+                part_o = torch.empty((T, H, parts, D), dtype=torch.float32, device=self.device)
+                part_ml = torch.empty((T, H, parts, 2), dtype=torch.float32, device=self.device)
             self.lib.call("rb_attention_prefill_tc", _ptr(out), _ptr(q), _ptr(view.k), _ptr(view.v),
                           view.k.shape[0], _ptr(view.page_table), view.max_pages, view.page_size,
                           _ptr(meta.tok_pos), _ptr(meta.tok_slot), _ptr(tok0), _ptr(ntok), n_tiles, H, Kh, D,
-                          float(scale), win, self._stream())
+                          float(scale), win, _ptr(part_o), _ptr(part_ml), parts, T, self._stream(), launches=2 if parts > 1 else 1)
         elif self.dtype == torch.bfloat16 and \
                 self.lib.raw("rb_attention_tiled_supports")(H, Kh, D, view.page_size, 0):
             tok0, ntok, n_tiles = self._prefill_tiles(meta, 64 // (H // Kh))
@@ -1140,7 +1151,7 @@ class CudaOps:
             gate_ptr, ldg = c_void_p(gate[0].data_ptr() + gate[1] * 4), gate[0].stride(0)
         if self.per_head_on_tensor_cores and self._tensor_core_ok(x, weight.w) and K % 8 == 0 and head_x % 8 == 0:
             whole_boxes = -(-N // 128) * 128 <= head_c and head_c % 8 == 0
-            tile = 64 if T <= 256 or not whole_boxes else 256
+            tile = 64 if T <= 256 or not whole_boxes or gate is not None else 256
             self.lib.call("rb_gemm_tc_per_head", H, int(head_x), int(head_c), gate_ptr, ldg, launches=0)
             self.lib.call("rb_gemm_tc", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), T, _ptr(weight.w), K, H * N, N,
                           K, 0, 0, 1, tile, 1.0, self._stream())

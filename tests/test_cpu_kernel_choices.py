@@ -40,8 +40,8 @@ def test_sizes_the_kernels_take(lib):
     assert not lib.raw("rb_attention_decode_tma_supports")(32, 8, 96, 64)      # head size
     assert not lib.raw("rb_attention_decode_tma_supports")(32, 8, 128, 16)     # pages of 16 positions
     assert not lib.raw("rb_attention_decode_tma_supports")(34, 2, 128, 64)     # 17 query heads a group
-    assert lib.raw("rb_attention_prefill_tc_supports")(32, 8, 64, 128)
-    assert not lib.raw("rb_attention_prefill_tc_supports")(7, 2, 128, 64)      # heads that are no multiple of the groups
+    assert lib.raw("rb_attention_prefill_tc_supports")(32, 8, 64, 128, 0)
+    assert not lib.raw("rb_attention_prefill_tc_supports")(7, 2, 128, 64, 0)      # heads that are no multiple of the groups
     assert lib.raw("rb_attention_tiled_supports")(6, 2, 96, 64, 1)
     assert not lib.raw("rb_attention_tiled_supports")(6, 2, 100, 64, 1)
     assert lib.raw("rb_gemm_tc_qkv_supports")(8, 128, 4)

@@ -504,3 +504,37 @@ def test_experts(dtype, T, E, F, n, top, shared, fused):
         if ask:
             assert torch.equal(request.result, ops.tanh_norm(x, nw, nb, 0.8))
     ops.check_errors()
+
+
+@pytest.mark.parametrize("H,D", [(8, 64), (16, 128), (32, 128), (3, 192), (32, 192), (32, 256), (128, 256), (20, 112)])
+@pytest.mark.parametrize("sinks,window", [(False, None), (True, None), (False, 100)])
+def test_attention_over_rows_that_are_keys_and_values(H, D, sinks, window):
+    """One key head whose keys and values are the same cached rows: prompts that begin anywhere in a page and a tile of
+    keys, and decode steps over short and long contexts (one whose keys are cut into parts of which some have none),
+    against the float32 kernel on the same rounded values."""
+    import dataclasses
+    from rbitnet_b200.cache import SequenceCache
+    from rbitnet_b200.parts.base import CacheNeed
+    runs = {"decode": [(1500, 1), (70, 1), (1, 1), (129, 1)], "one decode": [(700, 1)],
+            "prompts": [(300, 300), (1000, 37), (64, 64), (193, 2), (128, 1)], "long prompt": [(1100, 900)]}
+    results = {}
+    for dtype in (torch.float32, torch.bfloat16):
+        ops = _ops(dtype)
+        for what, seqs in runs.items():
+            cache = SequenceCache({0: CacheNeed(1, D, None, streams=((1, D),))}, {}, {}, 64 * 60, 2048, dtype, ops.device)
+            slots = [cache.alloc() for _ in seqs]
+            for s, (n, _) in zip(slots, seqs):
+                cache.reserve(s, n)
+            cache.upload_tables()
+            view = cache.view(0)
+            gen = torch.Generator().manual_seed(D + H)
+            view.k.copy_((torch.randn(view.k.shape, generator=gen) * 0.7).to(torch.bfloat16).to(dtype))
+            T = sum(n for _, n in seqs)
+            q = (torch.randn(T, H, D, generator=gen) * 0.7).to(torch.bfloat16).to(dtype).cuda()
+            sink = (torch.randn(H, generator=gen) * 3.0 + 3.0).float().cuda() if sinks else None
+            meta = _meta(ops, [(s, n - m, m) for s, (n, m) in zip(slots, seqs)])
+            got = ops.attention(q, meta, dataclasses.replace(view, v=view.k), H, 1.5 * D ** -0.5, window, sinks=sink)
+            results[dtype, what] = got.float().cpu()
+        ops.check_errors()
+    for what in runs:
+        assert rel_err(results[torch.bfloat16, what], results[torch.float32, what].double()) <= 1.5e-2, what
