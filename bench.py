@@ -299,6 +299,9 @@ class KernelTimer:
     so these are the times of the kernels alone, each starting on an idle GPU: their sum is above the
     step's own time, and a kernel's share of its roofline here is a lower bound of what it reaches
     inside the step."""
+    #: GPU clock cycles the device is kept busy before every operation, so that its launches are queued when it begins and the
+    #: time between its events is the device's and not the host's (0: not)
+    hold_cycles = 0
     decode_context = 0     # cached positions per sequence of the decode step being described without a sync
     OPS = ("embed", "rmsnorm", "linear", "gated_linear", "project_rotate_append", "rotate_append", "attention",
            "gather_rows", "sample", "decode_advance")
@@ -321,6 +324,8 @@ class KernelTimer:
                 before = self.ops.lib.launches
                 if self.events:
                     e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                    if self.hold_cycles:
+                        torch.cuda._sleep(self.hold_cycles)
                     e0.record()
                 try:
                     out = _fn(*a, **kw)
@@ -616,7 +621,9 @@ DESIGN_SIZES = {
 
 
 class DesignTimer(KernelTimer):
-    """KernelTimer with the operations of the recurrent mixers and of the residual streams."""
+    """KernelTimer with the operations of the recurrent mixers and of the residual streams, timed on a device that is kept
+    busy until an operation's launches are queued (many of these operations are shorter than their launches)."""
+    hold_cycles = 400_000
     OPS = KernelTimer.OPS + ("stream_step", "normed_mean", "streams_expand", "streams_sum", "norm_rotate_append", "head_gate",
                              "gated_recurrence", "matrix_memory", "layernorm", "add_rows", "gated_delta", "route", "routed_experts",
                              "rmsnorm_grouped", "input_filter", "gated_add", "add_scaled_rows", "softcap", "gated_linear_attention",

@@ -1149,7 +1149,7 @@ class CudaOps:
         if gate is not None:
             self._check(gate[0], torch.float32, "per-head gate")
             gate_ptr, ldg = c_void_p(gate[0].data_ptr() + gate[1] * 4), gate[0].stride(0)
-        if self.per_head_on_tensor_cores and self._tensor_core_ok(x, weight.w) and K % 8 == 0 and head_x % 8 == 0:
+        if self.per_head_on_tensor_cores and self._tensor_core_ok(x, weight.w.view(H * N, K)) and K % 8 == 0 and head_x % 8 == 0:
             whole_boxes = -(-N // 128) * 128 <= head_c and head_c % 8 == 0
             tile = 64 if T <= 256 or not whole_boxes or gate is not None else 256
             self.lib.call("rb_gemm_tc_per_head", H, int(head_x), int(head_c), gate_ptr, ldg, launches=0)

@@ -350,8 +350,11 @@ def test_a_matrix_per_head_with_strides_and_a_gate(dtype, gated, T, H, N, K, str
         want = want * torch.sigmoid(rows[:, 7:])
     for on in (True, False):
         ops.per_head_on_tensor_cores = on
+        before = ops.lib.raw("rb_gemm_tc_kernels_launched")()
         got = ops.per_head_linear(x.to(TORCH[dtype]).cuda(), weight, gate=(rows.float().cuda(), 7) if gated else None)
         assert rel_err(got.float().cpu(), want) <= (1e-5 if dtype == "float32" else 1e-2), on
+        if dtype == "bfloat16" and T > 16 and K % 8 == 0:       # the tensor-core product ran where it was asked for
+            assert (ops.lib.raw("rb_gemm_tc_kernels_launched")() > before) == on
     ops.check_errors()
 
 
