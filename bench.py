@@ -582,8 +582,8 @@ def _busavik_shape(width, heads, dim, rot, q_rank, kv_rank, experts, top, expert
     feed-forward is dense; from four layers on, the middle two run twice."""
     moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared_ff}}
     mixer = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": dim, "q_rank": q_rank, "kv_rank": kv_rank,
-             "scale": (dim + rot) ** -0.5, "rot": {"base": 500000.0, "dims": rot, "scaling": {
-                 "factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+             "scale": (dim + rot) ** -0.5, "rot": {"base": 10000.0, "dims": rot, "scaling": {
+                 "factor": 8.0, "original": 2048, "fast": 16.0, "slow": 2.0}}}
     ls = [{"type": "latent_attention", "mixer": mixer,
            "mlp": {"kind": "dense", "ff": ff} if dense_every and i % dense_every == 0 else moe} for i in range(layers)]
     cfg = {"architecture": "Busavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
@@ -626,7 +626,7 @@ class DesignTimer(KernelTimer):
     hold_cycles = 400_000
     OPS = KernelTimer.OPS + ("stream_step", "normed_mean", "streams_expand", "streams_sum", "norm_rotate_append", "head_gate",
                              "gated_recurrence", "matrix_memory", "layernorm", "add_rows", "gated_delta", "route", "routed_experts",
-                             "rmsnorm_grouped", "input_filter", "gated_add", "add_scaled_rows", "softcap", "gated_linear_attention",
+                             "rmsnorm_grouped", "input_filter", "gated_add", "softcap", "gated_linear_attention",
                              "latent_norm_append", "per_head_linear", "route_scored", "qk_prepare", "latent_rotate_append",
                              "retention", "norm_add", "round_rows", "token_gate", "embed_pairs", "tanh_norm", "latent_queries")
 
@@ -716,8 +716,6 @@ class DesignTimer(KernelTimer):
             return f"input filter [{a[0].shape[0]} rows, {a[1].shape[1]} taps]", 2 * el(a[0]), 0.0
         if name == "gated_add":
             return f"gated residual [{a[0].shape[0]} rows]", 3 * el(a[0]) + el(a[2]), 0.0
-        if name == "add_scaled_rows":
-            return f"shared expert's gate and sum [{a[0].shape[0]} rows]", 3 * el(a[0]), 0.0
         if name == "softcap":
             return f"soft cap [{a[0].shape[0]} rows]", 2 * el(a[0]), 0.0
         if name == "rmsnorm_grouped":

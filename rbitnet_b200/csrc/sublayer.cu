@@ -5,7 +5,6 @@
 //   input filter       h_t + sum_j taps[:, j] h_(t - K + 1 + j) over time on every channel (causal, zeros before a
 //                      sequence's start); the last K - 1 inputs of a sequence live in a ring of K rows by position
 //   gated residual     x += y * sigmoid(g + b), value by value
-//   scaled rows        y += sigmoid(logit_t) * z, one number per row
 //   soft cap           v <- cap * tanh(v / cap)
 //
 // All arithmetic is float32; rows enter and leave in the compute dtype where they feed a product.
@@ -284,16 +283,6 @@ __global__ void gated_add_kernel(float* __restrict__ x, const float* __restrict_
   }
 }
 
-__global__ void add_scaled_rows_kernel(float* __restrict__ y, const float* __restrict__ z, const float* __restrict__ logit,
-                                       int64_t ldl, int64_t n, int E) {
-  rb_pdl_launch_dependents();
-  rb_pdl_wait();
-  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
-    const int64_t t = i / E;
-    y[i] = fmaf(z[i], sigmoid_(logit[t * ldl]), y[i]);
-  }
-}
-
 __global__ void softcap_kernel(float* __restrict__ v, int64_t n, float cap) {
   rb_pdl_launch_dependents();
   rb_pdl_wait();
@@ -408,15 +397,6 @@ RB_EXPORT int rb_gated_add(float* x, const float* y, const void* g, int64_t ldg,
   else
     RB_FAIL("rb_gated_add: unknown dtype %d", g_dtype);
   RB_CHECK_LAUNCH("rb_gated_add");
-  return 0;
-}
-
-// y [T, E] += sigmoid(logit[t * ldl]) * z [T, E]
-RB_EXPORT int rb_add_scaled_rows(float* y, const float* z, const float* logit, int64_t ldl, int T, int E, cudaStream_t stream) {
-  if (T == 0) return 0;
-  const int64_t n = (int64_t)T * E;
-  RB_LAUNCH("add_scaled_rows_kernel", (add_scaled_rows_kernel), flat_blocks(n, 256), 256, 0, stream, y, z, logit, ldl, n, E);
-  RB_CHECK_LAUNCH("rb_add_scaled_rows");
   return 0;
 }
 

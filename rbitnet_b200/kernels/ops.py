@@ -896,14 +896,6 @@ class CudaOps:
                       self._stream())
         return x
 
-    def add_scaled_rows(self, y: torch.Tensor, z: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
-        """y += sigmoid(gate[t]) * z, one number per row; float32."""
-        self._check(y, torch.float32, "add_scaled_rows target")
-        self._check(z, torch.float32, "add_scaled_rows rows")
-        T, E = y.shape
-        self.lib.call("rb_add_scaled_rows", _ptr(y), _ptr(z), _ptr(gate), gate.stride(0), T, E, self._stream())
-        return y
-
     def softcap(self, v: torch.Tensor, cap: float) -> torch.Tensor:
         """v <- cap * tanh(v / cap), in place (float32)."""
         self._check(v, torch.float32, "softcap values")

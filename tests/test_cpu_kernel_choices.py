@@ -42,6 +42,16 @@ def test_sizes_the_kernels_take(lib):
     assert not lib.raw("rb_attention_decode_tma_supports")(34, 2, 128, 64)     # 17 query heads a group
     assert lib.raw("rb_attention_prefill_tc_supports")(32, 8, 64, 128, 0)
     assert not lib.raw("rb_attention_prefill_tc_supports")(7, 2, 128, 64, 0)      # heads that are no multiple of the groups
+    for D in (64, 128, 192, 256):                                              # keys and values that are the same rows
+        assert lib.raw("rb_attention_prefill_tc_supports")(32, 1, D, 64, 1)
+        assert bool(lib.raw("rb_attention_prefill_tc_supports")(32, 1, D, 64, 0)) == (D <= 128)
+    assert not lib.raw("rb_attention_prefill_tc_supports")(129, 1, 128, 64, 1)    # more heads than a tile has rows
+    parts = lib.raw("rb_attention_prefill_tc_parts")
+    for row_tiles in (1, 8, 100, 1000):
+        for context in (1, 128, 129, 2048, 100000):
+            n = parts(row_tiles, 1, context)
+            assert 1 <= n <= 16 and n <= -(-context // 128)                     # no part without a tile of keys to start from
+    assert parts(1, 1, 2048) == 16 and parts(1000, 1, 2048) == 1 and parts(8, 1, 128) == 1
     assert lib.raw("rb_attention_tiled_supports")(6, 2, 96, 64, 1)
     assert not lib.raw("rb_attention_tiled_supports")(6, 2, 100, 64, 1)
     assert lib.raw("rb_gemm_tc_qkv_supports")(8, 128, 4)

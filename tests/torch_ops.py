@@ -297,10 +297,6 @@ class TorchOps:
         x += y * torch.sigmoid(z)
         return x
 
-    def add_scaled_rows(self, y, z, gate):
-        y += torch.sigmoid(gate[:, :1]) * z
-        return y
-
     def softcap(self, v, cap):
         v.copy_(cap * torch.tanh(v / cap))
         return v
