@@ -13,7 +13,8 @@ A group whose layers see only the last ``window`` keys gives a sequence's pages
 back as soon as they lie wholly behind the window of the sequence's next token
 (the attention kernels start at the page that holds the first visible key), so
 a long sequence holds about ``window / page_size + 2`` pages of such a group,
-whatever its length.  The released places of a page list hold -1.
+whatever its length.  The released places of a page list hold -1.  Where the first
+``keep_first`` positions stay visible to every later token, their pages are kept.
 """
 from __future__ import annotations
 
@@ -64,12 +65,14 @@ class SlotBook:
     """Slots, their lengths and their pages in every group."""
 
     def __init__(self, n_slots: int, pages_per_group: List[int], page_size: int, max_seq: int,
-                 windows: Optional[List[Optional[int]]] = None):
+                 windows: Optional[List[Optional[int]]] = None, keeps: Optional[List[int]] = None):
         self.page_size, self.max_seq = page_size, max_seq
         self.slots = FreeList(n_slots)
         self.pools = [FreeList(n) for n in pages_per_group]
         #: per group, how many of the last keys its layers see (None: all of them)
         self.windows = list(windows) if windows is not None else [None] * len(pages_per_group)
+        #: per group, how many leading pages hold positions that stay visible
+        self.kept_pages = [-(-int(k or 0) // page_size) for k in keeps] if keeps is not None else [0] * len(pages_per_group)
         self.has_windows = any(w for w in self.windows)
         self.length: Dict[int, int] = {}
         self.pages: Dict[int, List[List[int]]] = {}
@@ -135,14 +138,15 @@ class SlotBook:
 
     def release_behind_window(self, slot: int) -> None:
         """Gives back the pages of windowed groups that no later token of the sequence can see: the
-        next token sits at position ``length`` and sees keys from ``length - window + 1`` on."""
+        next token sits at position ``length`` and sees keys from ``length - window + 1`` on (and the first ones that
+        every token sees, whose pages stay)."""
         n = self.length[slot]
         for g, w in enumerate(self.windows):
             if not w:
                 continue
             pages = self.pages[slot][g]
             first_needed = min(max(0, n - w + 1) // self.page_size, len(pages))
-            for i in range(self._released[slot][g], first_needed):
+            for i in range(max(self._released[slot][g], self.kept_pages[g]), first_needed):
                 self.pools[g].give(pages[i])
                 pages[i] = -1
             if first_needed > self._released[slot][g]:
@@ -155,7 +159,7 @@ class SlotBook:
         w = self.windows[group]
         if not w:
             return whole
-        return min(whole, max(-(-int(prompt) // self.page_size), (w - 1) // self.page_size + 2))
+        return min(whole, max(-(-int(prompt) // self.page_size), (w - 1) // self.page_size + 2 + self.kept_pages[group]))
 
     def live(self):
         return sorted(self.length)

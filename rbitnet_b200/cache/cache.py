@@ -91,7 +91,8 @@ class SequenceCache:
             g, i, _ = self._where[src]
             self._where[entry] = (g, i, False)
         self.book = SlotBook(self.n_slots, [grp.n_pages for grp in self.groups], page_size, max_seq,
-                             windows=[grp.need.window for grp in self.groups])
+                             windows=[grp.need.window for grp in self.groups],
+                             keeps=[grp.need.keep_first for grp in self.groups])
         # one tensor [n_slots, *shape] per need; a mixer that keeps several tensors per sequence names them,
         # and those are kept under (entry, name)
         self.states: Dict[object, torch.Tensor] = {}

@@ -52,6 +52,7 @@ struct Params {
   int H, G;
   float scale_log2;         // scale * log2(e)
   int window;               // 0: none
+  int keep;                 // with a window: the first so many keys stay visible
   const float* sinks;       // [H] or null: a term exp(sinks[h]) in head h's denominator
   float softcap;            // > 0: score <- softcap * tanh(score * scale / softcap)
   float scale;
@@ -109,7 +110,8 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
   const int slot = p.tok_slot[tok0];
   const int pos0 = p.tok_pos[tok0];
   const int key_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-  int kt_begin = key_lo / TILE, kt_end = pos0 / TILE + 1;
+  const RbKeyTiles tiles(key_lo, pos0, p.keep, TILE);
+  int kt_begin = 0, kt_end = tiles.n;         // numbers of the visited tiles, see RbKeyTiles
   if (p.n_splits > 1) {
     // the tiles are dealt evenly: part z takes [z*n/parts, (z+1)*n/parts), sizes that differ by at most one
     const int n = kt_end - kt_begin, z = blockIdx.z;
@@ -124,8 +126,8 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
   __syncthreads();
 
   // one thread asks for a tile: keys and values of 64 positions of this kv head, D/64 boxes each
-  auto request = [&](int kt, int buf) {
-    const int key0 = kt * TILE;
+  auto request = [&](int i, int buf) {
+    const int key0 = tiles.at(i) * TILE;
     const int page = p.page_table[(int64_t)slot * p.max_pages + key0 / p.page_size];
     const int row = (page * p.n_kv_heads + kvh) * p.page_size + key0 % p.page_size;
     mbar_expect_tx(&full[buf], 2 * S::TILE_BYTES);
@@ -141,7 +143,7 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
   int n_early = 0;                     // tiles requested before the wait (thread 0's count)
   if (threadIdx.x == 0) {
     for (int i = 0; i < NS - 1; ++i)
-      if (kt_begin + i < kt_end && kt_begin + i != newest && n_early == i) {
+      if (kt_begin + i < kt_end && tiles.at(kt_begin + i) != newest && n_early == i) {
         request(kt_begin + i, i);
         n_early = i + 1;
       }
@@ -188,7 +190,7 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
     if (!failed && !mbar_wait(&full[buf], (uint32_t)((i / NS) & 1), 14)) failed = true;
     const uint32_t tK = smem_u32(smem + S::OFF_K + buf * S::TILE_BYTES);
     const uint32_t tV = smem_u32(smem + S::OFF_V + buf * S::TILE_BYTES);
-    const int key_base = kt * TILE + kw0;
+    const int key_base = tiles.at(kt) * TILE + kw0;
     if (key_base <= pos0) {
       // ---- S = Q K^T: two accumulators per 8-key tile, over even and odd steps of d, so that the
       // chain of dependent products is half as long
@@ -212,7 +214,7 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
         for (int c = 0; c < 4; ++c) {
           const int h = c >> 1;
           const int key = key_base + n * 8 + t4 * 2 + (c & 1);
-          const bool ok = row_ok[h] && key <= pos0 && key >= key_lo;
+          const bool ok = row_ok[h] && key <= pos0 && (key >= key_lo || key < p.keep);
           const float sc = s[n][c] + s2[n][c];
           const float v = !ok ? -INFINITY : (p.softcap > 0.f ? cap_log2 * tanhf(sc * scale_over_cap) : sc * p.scale_log2);
           s[n][c] = v;

@@ -6,7 +6,7 @@
 // batched.
 //
 // Token t at position p of its sequence attends keys max(0, p-window+1)..p of
-// its own slot; query head h reads kv head h / (H/Kh); the score is
+// its own slot (and, with keep_first, the first keys whatever the window); query head h reads kv head h / (H/Kh); the score is
 // (q.k) * scale with the scale applied to the finished dot product; softmax is
 // max-subtracted.  crates/bitnet-core/src/llama/model.rs:260-289, :102-114
 #include "rb_common.cuh"
@@ -18,7 +18,7 @@ __global__ void __launch_bounds__(128) attn_simple_kernel(T* __restrict__ out, c
                                                          RbPagedLayer cache, const int* __restrict__ tok_pos,
                                                          const int* __restrict__ tok_slot, int n_tokens, int H,
                                                          float scale, int window, const float* __restrict__ sinks,
-                                                         float softcap) {
+                                                         float softcap, int keep) {
   rb_pdl_launch_dependents();
   rb_pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -43,7 +43,10 @@ __global__ void __launch_bounds__(128) attn_simple_kernel(T* __restrict__ out, c
   if (sinks != nullptr) { m = sinks[h]; l = 1.f; }     // the sink: one more term of the denominator, without a value
   const float inv_cap = softcap > 0.f ? 1.0f / softcap : 0.f;
   const int lo = window > 0 ? max(0, pos - window + 1) : 0;
-  for (int p = lo; p <= pos; ++p) {
+  // the first `keep` positions that lie before the window, then the window
+  const int n_kept = min(keep, lo);
+  for (int i = 0; i <= pos - lo + n_kept; ++i) {
+    const int p = i < n_kept ? i : lo + (i - n_kept);
     const int64_t off = rb_page_offset(cache, slot, p, kvh);
     float part = 0.f;
 #pragma unroll
@@ -82,7 +85,7 @@ int launch(T* out, const T* q, RbPagedLayer c, const int* tok_pos, const int* to
   int epl = (c.head_dim + 31) / 32;
   if (epl > 8) epl = epl <= 12 ? 12 : (epl <= 16 ? 16 : (epl <= 24 ? 24 : (epl <= 32 ? 32 : epl)));   // head sizes up to 1,024
 #define CASE(E) \
-  case E: RB_LAUNCH("attn_simple_kernel", (attn_simple_kernel<T, E>), blocks, 128, 0, stream, out, q, c, tok_pos, tok_slot, n_tokens, H, scale, window, opt.sinks, opt.softcap); break;
+  case E: RB_LAUNCH("attn_simple_kernel", (attn_simple_kernel<T, E>), blocks, 128, 0, stream, out, q, c, tok_pos, tok_slot, n_tokens, H, scale, window, opt.sinks, opt.softcap, opt.keep_first); break;
   switch (epl) {
     CASE(1) CASE(2) CASE(3) CASE(4) CASE(5) CASE(6) CASE(7) CASE(8) CASE(12) CASE(16) CASE(24) CASE(32)
     default: RB_FAIL("rb_attention_simple: head_dim %d exceeds 1024", c.head_dim);
@@ -103,8 +106,9 @@ RbAttentionOptions rb_attention_take() {
 }
 
 // For the calling thread's next attention launch (any of the library's attention entry points); see rb_common.cuh.
-RB_EXPORT int rb_attention_next(const float* sinks, float softcap) {
+RB_EXPORT int rb_attention_next(const float* sinks, float softcap, int keep_first) {
   t_next_attention.sinks = sinks;
+  t_next_attention.keep_first = keep_first > 0 ? keep_first : 0;
   t_next_attention.softcap = softcap > 0.f ? softcap : 0.f;
   return 0;
 }

@@ -55,6 +55,7 @@ struct TcAttnParams {
   int H, G;
   float scale_log2;
   int window;
+  int keep;                 // with a window: the first so many keys stay visible
   const float* sinks;       // [H] or null: a term exp(sinks[h]) in head h's denominator
   float softcap;            // > 0: score <- softcap * tanh(score * scale / softcap), before the mask
   float scale;
@@ -194,7 +195,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   const int n_rows = ntok * G;
   const int key_hi = pos0 + ntok - 1;
   const int key_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-  int kt_begin = key_lo / TILE_KEYS, kt_end = key_hi / TILE_KEYS + 1;
+  const RbKeyTiles tiles(key_lo, key_hi, p.keep, TILE_KEYS);
+  int kt_begin = 0, kt_end = tiles.n;                      // numbers of the visited tiles, see RbKeyTiles
   if (p.n_splits > 1) {                                    // this CTA's range of the key tiles (it may be empty)
     const int per = (kt_end - kt_begin + p.n_splits - 1) / p.n_splits;
     kt_begin += (int)blockIdx.z * per;
@@ -258,7 +260,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         int row[TILE_KEYS / PIECE];
 #pragma unroll
         for (int h = 0; h < TILE_KEYS / PIECE; ++h) {      // a tile is two pieces of 64 positions
-          const int key0 = kt * TILE_KEYS + h * PIECE;
+          const int key0 = tiles.at(kt) * TILE_KEYS + h * PIECE;
           const int pi = min(key0 / p.page_size, p.max_pages - 1);       // past the sequence: any page, masked later
           const int page = p.page_table[(int64_t)slot * p.max_pages + pi];
           row[h] = (page * p.n_kv_heads + kvh) * p.page_size + key0 % p.page_size;
@@ -385,11 +387,11 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
           sv[c] = fmaf(-2.0f * cap_b, rc, cap_b);
         }
       }
-      const int key_base = kt * TILE_KEYS + half * HK;
+      const int key0 = tiles.at(kt) * TILE_KEYS, key_base = key0 + half * HK;
       // a tile that every row of the CTA sees whole needs no mask (all tiles but those on the
-      // diagonal and at the window's edge)
-      const bool whole = kt * TILE_KEYS + TILE_KEYS - 1 <= pos0 &&
-                         (p.window <= 0 || kt * TILE_KEYS >= max(0, key_hi - p.window + 1));
+      // diagonal, at the window's edge and at the end of the first keys that stay visible)
+      const bool whole = key0 + TILE_KEYS - 1 <= pos0 &&
+                         (p.window <= 0 || key0 >= max(0, key_hi - p.window + 1) || key0 + TILE_KEYS <= p.keep);
       float m_half;
       if (whole) {
         float t0 = sv[0], t1 = sv[1], t2 = sv[2], t3 = sv[3];          // four chains of three-input maxima
@@ -405,8 +407,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
 #pragma unroll
         for (int c = 0; c < HK; c += 2) {
           const int key = key_base + c;
-          sv[c] = (row_ok && key <= row_pos && key >= row_lo) ? sv[c] : -INFINITY;
-          sv[c + 1] = (row_ok && key + 1 <= row_pos && key + 1 >= row_lo) ? sv[c + 1] : -INFINITY;
+          sv[c] = (row_ok && key <= row_pos && (key >= row_lo || key < p.keep)) ? sv[c] : -INFINITY;
+          sv[c + 1] = (row_ok && key + 1 <= row_pos && (key + 1 >= row_lo || key + 1 < p.keep)) ? sv[c + 1] : -INFINITY;
           t0 = fmaxf(t0, sv[c]); t1 = fmaxf(t1, sv[c + 1]);
         }
         m_half = fmaxf(t0, t1) * p.scale_log2;
@@ -625,7 +627,7 @@ RB_EXPORT int rb_attention_decode_tma(void* out, const void* q, const void* cach
   p.page_table = page_table; p.max_pages = max_pages; p.page_size = page_size; p.n_kv_heads = Kh;
   p.tok_pos = tok_pos; p.tok_slot = tok_slot; p.H = H; p.G = H / Kh;
   p.scale_log2 = scale * 1.4426950408889634f; p.window = window;
-  { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; }
+  { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; p.keep = window > 0 ? opt.keep_first : 0; }
   p.part_o = part_o; p.part_ml = part_ml; p.n_splits = n_splits; p.cluster = cluster ? 1 : 0;
   const int rc = D == 64 ? decode_tma::launch<64>(tk, tv, p, B, Kh, stream) : decode_tma::launch<128>(tk, tv, p, B, Kh, stream);
   if (rc != 0) return rc;
@@ -678,7 +680,7 @@ RB_EXPORT int rb_attention_prefill_tc(void* out, const void* q, const void* cach
   p.page_table = page_table; p.max_pages = max_pages; p.page_size = page_size; p.n_kv_heads = Kh;
   p.tok_pos = tok_pos; p.tok_slot = tok_slot; p.tile_tok0 = tile_tok0; p.tile_ntok = tile_ntok; p.n_tiles = n_tiles;
   p.H = H; p.G = H / Kh; p.scale_log2 = scale * 1.4426950408889634f; p.window = window;
-  { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; }
+  { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; p.keep = window > 0 ? opt.keep_first : 0; }
   p.part_o = part_o; p.part_ml = part_ml; p.n_splits = n_splits;
   int rc;
   if (!shared) rc = D == 64 ? launch_tc<64, false>(tk, tv, p, Kh, stream) : launch_tc<128, false>(tk, tv, p, Kh, stream);

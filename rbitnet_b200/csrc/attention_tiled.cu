@@ -63,6 +63,7 @@ struct AttnParams {
   int H, G;
   float scale_log2;         // scale * log2(e)
   int window;               // 0: none
+  int keep;                 // with a window: the first so many keys stay visible
   const float* sinks;       // [H] or null: a term exp(sinks[h]) in head h's denominator
   float softcap;            // > 0: score <- softcap * tanh(score * scale / softcap)
   float scale;
@@ -110,7 +111,8 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tiled_kernel(AttnParams p) {
   const int n_rows = ntok * G;
   const int key_hi = pos0 + ntok - 1;                                    // last key any row may see
   const int key_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;      // first key any row may see
-  int kt_begin = key_lo / TILE_KEYS, kt_end = key_hi / TILE_KEYS + 1;
+  const RbKeyTiles tiles(key_lo, key_hi, p.keep, TILE_KEYS);
+  int kt_begin = 0, kt_end = tiles.n;                                    // numbers of the visited tiles, see RbKeyTiles
   if (DECODE && p.n_splits > 1) {
     // the tiles are dealt evenly: part z takes [z*n/parts, (z+1)*n/parts), sizes that differ by at most one
     const int n = kt_end - kt_begin, z = blockIdx.z;
@@ -120,8 +122,8 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tiled_kernel(AttnParams p) {
 
   const __nv_bfloat16* Kbase = reinterpret_cast<const __nv_bfloat16*>(p.cache.k);
   const __nv_bfloat16* Vbase = reinterpret_cast<const __nv_bfloat16*>(p.cache.v);
-  auto load_tile = [&](int kt, int buf) {
-    const int key0 = kt * TILE_KEYS;
+  auto load_tile = [&](int i, int buf) {
+    const int key0 = tiles.at(i) * TILE_KEYS;
     const int page = p.cache.page_table[(int64_t)slot * p.cache.max_pages + key0 / p.cache.page_size];
     const int64_t off = (((int64_t)page * p.cache.n_kv_heads + kvh) * p.cache.page_size + key0 % p.cache.page_size) * D;
     const __nv_bfloat16* ksrc = Kbase + off;
@@ -144,7 +146,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tiled_kernel(AttnParams p) {
   if (DECODE) {
     for (int i = 0; i < NS - 1; ++i) {
       const int kt = kt_begin + i;
-      if (kt < kt_end && kt != newest && n_early == i) {
+      if (kt < kt_end && tiles.at(kt) != newest && n_early == i) {
         load_tile(kt, i);
         cp_async_commit();
         n_early = i + 1;
@@ -207,7 +209,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tiled_kernel(AttnParams p) {
     __syncthreads();
     const __nv_bfloat16* tK = sK + buf * S::KV_ELEMS;
     const __nv_bfloat16* tV = sV + buf * S::KV_ELEMS;
-    const int key_base = kt * TILE_KEYS + kw0;
+    const int key_base = tiles.at(kt) * TILE_KEYS + kw0;
 
     // a warp whose rows see none of this tile's keys skips it (prefill: tiles past the diagonal)
     const bool warp_has_rows = DECODE || rb < n_rows;
@@ -238,7 +240,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tiled_kernel(AttnParams p) {
         for (int c = 0; c < 4; ++c) {
           const int h = c >> 1;
           const int key = key_base + nt * 8 + t4 * 2 + (c & 1);
-          const bool ok = row_ok[h] && key <= row_pos[h] && key >= row_lo[h];
+          const bool ok = row_ok[h] && key <= row_pos[h] && (key >= row_lo[h] || key < p.keep);
           const float v = !ok ? -INFINITY : (p.softcap > 0.f ? cap_log2 * tanhf(s[nt][c] * scale_over_cap) : s[nt][c] * p.scale_log2);
           s[nt][c] = v;
           m_new[h] = fmaxf(m_new[h], v);
@@ -455,7 +457,7 @@ RB_EXPORT int rb_attention_prefill(void* out, const void* q, const void* cache_k
   p.cache = RbPagedLayer{(void*)cache_k, (void*)cache_v, page_table, max_pages, page_size, Kh, D};
   p.tok_pos = tok_pos; p.tok_slot = tok_slot; p.tile_tok0 = tile_tok0; p.tile_ntok = tile_ntok;
   p.H = H; p.G = H / Kh; p.scale_log2 = scale * 1.4426950408889634f; p.window = window;
-  { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; }
+  { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; p.keep = window > 0 ? opt.keep_first : 0; }
   p.part_o = nullptr; p.part_ml = nullptr; p.n_splits = 1;
   return launch_d<false>(D, p, dim3(n_tiles, Kh, 1), stream);
 }
@@ -505,7 +507,7 @@ RB_EXPORT int rb_attention_decode(void* out, const void* q, const void* cache_k,
   p.cache = RbPagedLayer{(void*)cache_k, (void*)cache_v, page_table, max_pages, page_size, Kh, D};
   p.tok_pos = tok_pos; p.tok_slot = tok_slot; p.tile_tok0 = nullptr; p.tile_ntok = nullptr;
   p.H = H; p.G = H / Kh; p.scale_log2 = scale * 1.4426950408889634f; p.window = window;
-  { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; }
+  { const RbAttentionOptions opt = rb_attention_take(); p.sinks = opt.sinks; p.softcap = opt.softcap; p.scale = scale; p.keep = window > 0 ? opt.keep_first : 0; }
   p.part_o = part_o; p.part_ml = part_ml; p.n_splits = n_splits;
   if (launch_d<true>(D, p, dim3(B, Kh, n_splits), stream) != 0) return -1;
   if (n_splits > 1) return rb_attention_combine(out, part_o, part_ml, B, H, D, n_splits, stream);

@@ -1097,6 +1097,10 @@ __global__ void gated_act_kernel(T* __restrict__ out, const TI* __restrict__ gu,
       out[i] = rb_from_float<T>(g / (1.0f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u);
       continue;
     }
+    if (kind == 2) {
+      out[i] = rb_from_float<T>(fmaxf(g, 0.f) * u);
+      continue;
+    }
     if (limit > 0.f) {
       g = fminf(g, limit);
       u = fminf(fmaxf(u, -limit), limit);
@@ -1108,7 +1112,7 @@ __global__ void gated_act_kernel(T* __restrict__ out, const TI* __restrict__ gu,
 RB_EXPORT int rb_gated_act(void* out, const void* gate_up, int dtype, int in_dtype, int T, int F, int64_t ld, int block,
                            int kind, float alpha, float limit, float shift, const float* bias, cudaStream_t stream) {
   if (T == 0) return 0;
-  RB_REQUIRE(kind == 0 || kind == 1, "rb_gated_act: activation %d is not built (0: limited swish, 1: gelu in its tanh form)", kind);
+  RB_REQUIRE(kind >= 0 && kind <= 2, "rb_gated_act: activation %d is not built (0: limited swish, 1: gelu in its tanh form, 2: relu)", kind);
   RB_REQUIRE(block >= 0 && (block == 0 ? ld >= 2 * (int64_t)F : ld >= ((int64_t)(F + block - 1) / block) * 2 * block),
              "rb_gated_act: rows of %lld values do not hold %d features in blocks of %d", (long long)ld, F, block);
   const int64_t n = (int64_t)T * F;

@@ -14,16 +14,18 @@ namespace {
 constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;  // 256 threads, 4x4 outputs each
 
 // What happens to a finished sum before it is stored or added (null: nothing): bias[n] is added, and the value is
-// multiplied by sigmoid(gate[row * ldg + z * gate_batch + n]), z the number of the product (a head).
+// multiplied by sigmoid(gate[row * ldg + z * gate_batch + n * gate_step]), z the number of the product (a head); a step of
+// 0 is one gate for all of a product's values.
 struct Tail {
   const float* bias = nullptr;
   const float* gate = nullptr;
   int64_t ldg = 0;
   int64_t gate_batch = 0;
+  int gate_step = 1;
 };
 __device__ __forceinline__ float finished(const Tail& tail, float v, int64_t row, int n, int64_t z) {
   if (tail.bias != nullptr) v += tail.bias[n];
-  if (tail.gate != nullptr) v *= 1.0f / (1.0f + expf(-tail.gate[row * tail.ldg + z * tail.gate_batch + n]));
+  if (tail.gate != nullptr) v *= 1.0f / (1.0f + expf(-tail.gate[row * tail.ldg + z * tail.gate_batch + n * tail.gate_step]));
   return v;
 }
 
@@ -215,9 +217,10 @@ Tail take_tail() {
 }  // namespace
 
 // The next rb_gemm_simple, rb_gemm_simple_batched or rb_per_head_few_rows call of this thread adds bias[n] (float32, or
-// null) to every finished sum and multiplies it by sigmoid(gate[row * ldg + z * gate_batch + n]) (float32, or null; z: the
-// number of the product or head).
-RB_EXPORT int rb_gemm_simple_next(const float* bias, const float* gate, int64_t ldg, int64_t gate_batch) {
+// null) to every finished sum and multiplies it by sigmoid(gate[row * ldg + z * gate_batch + n * gate_step]) (float32, or
+// null; z: the number of the product or head).
+RB_EXPORT int rb_gemm_simple_next(const float* bias, const float* gate, int64_t ldg, int64_t gate_batch, int gate_step) {
+  t_tail.gate_step = gate_step;
   t_tail.bias = bias; t_tail.gate = gate; t_tail.ldg = ldg; t_tail.gate_batch = gate_batch;
   return 0;
 }

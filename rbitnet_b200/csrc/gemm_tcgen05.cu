@@ -111,7 +111,7 @@ struct GemmParams {
   QkvTail qkv;        // EPI_QKV only
   // EPI_GATED: out = g' / (1 + e^(-act_alpha g')) * (u' + act_shift), g' = min(g, act_limit), u' = clamp(u, +-act_limit)
   // (act_limit <= 0: no limit).  1, 0, 0 is SiLU(gate) * up.
-  // act_kind 1: out = gelu_tanh(gate) * up instead.
+  // act_kind 1: out = gelu_tanh(gate) * up instead; 2: out = max(gate, 0) * up.
   float act_alpha, act_limit, act_shift;
   int act_kind;
   // A number per row of W (float32, or null) that is added to the finished sums (before a gated activation).
@@ -128,8 +128,8 @@ struct GemmParams {
   // One matrix per head (heads > 0; EPI_STORE, K whole): W holds `heads` matrices of n_out rows one below the other,
   // head h reads columns h * head_x .. + K - 1 of X (what a box of X holds beyond them meets zeros in the box of W)
   // and writes columns h * head_c .. + n_out - 1 of C.  gate (or null): the values are multiplied by
-  // sigmoid(gate[token * gate_ld + h * n_out + column]).
-  int heads, head_x, head_c;
+  // sigmoid(gate[token * gate_ld + h * n_out + column]), or with gate_heads by sigmoid(gate[token * gate_ld + h]).
+  int heads, head_x, head_c, gate_heads;
   const float* gate;
   int64_t gate_ld;
 };
@@ -144,6 +144,7 @@ __device__ __forceinline__ float stored_value(const GemmParams& p, float v) {
 __device__ __forceinline__ float gated_value(const GemmParams& p, float g, float up) {
   // gelu_tanh(g) = g/2 (1 + tanh(s)) = g / (1 + e^(-2 s)), s = sqrt(2/pi) (g + 0.044715 g^3)
   if (p.act_kind == 1) return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * g * (1.0f + 0.044715f * g * g))) * up;
+  if (p.act_kind == 2) return fmaxf(g, 0.f) * up;
   if (p.act_limit > 0.f) {
     g = fminf(g, p.act_limit);
     up = fminf(fmaxf(up, -p.act_limit), p.act_limit);
@@ -437,7 +438,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       // the same for the gate's values of a product with one matrix per head
       auto fetch_gate = [&](int c, float* into) {
         const int left = n_ok ? p.n_tokens - (t0 + c) : 0;
-        const float* src = p.gate + (int64_t)(t0 + c) * p.gate_ld + (s.w0 + row);
+        const float* src = p.gate + (int64_t)(t0 + c) * p.gate_ld + (p.gate_heads ? s.w0 / p.n_out : s.w0 + row);
 #pragma unroll
         for (int j = 0; j < 16; ++j) into[j] = j < left ? src[(int64_t)j * p.gate_ld] : 0.f;
       };
@@ -1136,7 +1137,7 @@ thread_local GatedAct t_act;
 struct StoreOptions {
   int square_relu = 0; const int* tile_group = nullptr; int group_rows = 0;
   const float* bias = nullptr;
-  int heads = 0, head_x = 0, head_c = 0; const float* gate = nullptr; int64_t gate_ld = 0;
+  int heads = 0, head_x = 0, head_c = 0, gate_heads = 0; const float* gate = nullptr; int64_t gate_ld = 0;
 };
 thread_local StoreOptions t_store;
 }  // namespace
@@ -1163,6 +1164,12 @@ RB_EXPORT int rb_gemm_tc_gated_act(float alpha, float limit, float shift) {
   return 0;
 }
 
+// The next gated product (epilogue 3) of this thread applies max(gate, 0) * up.
+RB_EXPORT int rb_gemm_tc_gated_relu() {
+  t_act.kind = 2;
+  return 0;
+}
+
 // The next gated product (epilogue 3) of this thread applies gelu_tanh(gate) * up.
 RB_EXPORT int rb_gemm_tc_gated_gelu() {
   t_act.kind = 1;
@@ -1179,8 +1186,10 @@ RB_EXPORT int rb_gemm_tc_bias(const float* bias) {
 // The next stored product (epilogue 0, one split) of this thread multiplies by one matrix per head (see GemmParams): W
 // holds heads * n_out rows, X and C the heads' columns head_x and head_c apart.  A token tile of 128 and more writes
 // whole boxes of 128 columns, so it needs head_c >= n_out rounded up to 128; what it leaves in columns n_out .. of a head
-// is not defined.  gate (token tiles of 64 only): null, or float32 with column h * n_out + n for value n of head h.
-RB_EXPORT int rb_gemm_tc_per_head(int heads, int head_x, int head_c, const float* gate, long long gate_ld) {
+// is not defined.  gate (token tiles of 64 only): null, or float32 with column h * n_out + n for value n of head h
+// (gate_heads: column h for all of head h's values).
+RB_EXPORT int rb_gemm_tc_per_head(int heads, int head_x, int head_c, const float* gate, long long gate_ld, int gate_heads) {
+  t_store.gate_heads = gate_heads;
   RB_REQUIRE(heads > 0 && head_x > 0 && head_c > 0, "rb_gemm_tc_per_head: bad sizes heads=%d, %d and %d apart", heads, head_x, head_c);
   t_store.heads = heads; t_store.head_x = head_x; t_store.head_c = head_c; t_store.gate = gate; t_store.gate_ld = gate_ld;
   return 0;
@@ -1340,7 +1349,7 @@ static int gemm_tc(void* C, int64_t ldc, int c_dtype, const void* X, int64_t ldx
     p.act_alpha = act.alpha; p.act_limit = act.limit; p.act_shift = act.shift; p.act_kind = act.kind;
   }
   p.bias = store.bias;
-  p.heads = store.heads; p.head_x = store.head_x; p.head_c = store.head_c;
+  p.heads = store.heads; p.head_x = store.head_x; p.head_c = store.head_c; p.gate_heads = store.gate_heads;
   p.gate = store.heads > 0 ? store.gate : nullptr; p.gate_ld = store.gate_ld;
   p.norm_ss = norm.in_ss; p.norm_parts = norm.in_parts; p.norm_width = norm.in_width; p.norm_eps = norm.in_eps;
   RB_REQUIRE(norm.in_ss == nullptr || (bn <= 16 && n_tokens <= 16),

@@ -4,6 +4,8 @@
 //
 //   round_rows_kernel          x (float32) -> compute dtype
 //   norm_add_kernel            x += y / rms(y) * w  (y a sublayer's float32 result); optionally also x in the compute dtype
+//   norm_add_norm_kernel       the same addition, and the rows of the norm after it: rounded(x / rms(x) * w2); without x:
+//                              x = y / rms(y) * w
 //   token_gate_kernel          gelu_tanh(a) * table[id]
 //   embed_pairs_kernel         table[id] * scale + pairs[(previous * a + id * b) mod n] (a sequence's first token: row n);
 //                              the sequence's last token is kept per slot
@@ -88,6 +90,85 @@ __global__ void __launch_bounds__(256) norm_add_kernel(float* __restrict__ x, co
       if (rounded != nullptr) rounded[row * E + e] = rb_from_float<T>(o);
     }
   }
+}
+
+// A block per row: x (+)= y / rms(y) * w, then h = x / rms(x) * w2.  VEC: a thread holds NV times four values of the row in
+// registers (blockDim.x * NV * 4 >= E); else the row goes through memory, each thread its own values.
+template <typename T, bool VEC, int NV>
+__global__ void __launch_bounds__(1024) norm_add_norm_kernel(float* __restrict__ x, const float* __restrict__ y,
+                                                             const float* __restrict__ w, float eps, int E, int fresh,
+                                                             T* __restrict__ h, const float* __restrict__ w2, float eps2) {
+  rb_pdl_launch_dependents();
+  __shared__ float scratch[33];
+  const int64_t row = blockIdx.x;
+  const float* yr = y + row * E;
+  float* xr = x + row * E;
+  T* hr = h + row * E;
+  if (VEC) {
+    float ww[NV][4], v[NV][4], o[NV][4];
+    // the weights do not depend on the kernel before this one
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = (i * blockDim.x + threadIdx.x) * 4;
+      if (e < E) rb_load4(w + e, ww[i]);
+    }
+    rb_pdl_wait();
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = (i * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[i][k] = o[i][k] = 0.f;
+      if (e < E) {
+        rb_load4(yr + e, v[i]);
+        if (!fresh) rb_load4(xr + e, o[i]);
+      }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) ss = fmaf(v[i][k], v[i][k], ss);
+    }
+    ss = rb_block_sum(ss, scratch);
+    const float r = 1.0f / sqrtf(ss / (float)E + eps);
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = (i * blockDim.x + threadIdx.x) * 4;
+      if (e < E) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          o[i][k] += v[i][k] * r * ww[i][k];
+          ss = fmaf(o[i][k], o[i][k], ss);
+        }
+        rb_store4(xr + e, o[i]);
+        rb_load4(w2 + e, ww[i]);
+      }
+    }
+    ss = rb_block_sum(ss, scratch);
+    const float r2 = 1.0f / sqrtf(ss / (float)E + eps2);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = (i * blockDim.x + threadIdx.x) * 4;
+      if (e < E) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) o[i][k] = o[i][k] * r2 * ww[i][k];
+        rb_store4(hr + e, o[i]);
+      }
+    }
+    return;
+  }
+  rb_pdl_wait();
+  float ss = 0.f;
+  for (int e = threadIdx.x; e < E; e += blockDim.x) ss = fmaf(yr[e], yr[e], ss);
+  ss = rb_block_sum(ss, scratch);
+  const float r = 1.0f / sqrtf(ss / (float)E + eps);
+  ss = 0.f;
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {
+    const float o = (fresh ? 0.f : xr[e]) + yr[e] * r * w[e];
+    xr[e] = o;
+    ss = fmaf(o, o, ss);
+  }
+  ss = rb_block_sum(ss, scratch);
+  const float r2 = 1.0f / sqrtf(ss / (float)E + eps2);
+  for (int e = threadIdx.x; e < E; e += blockDim.x) hr[e] = rb_from_float<T>(xr[e] * r2 * w2[e]);
 }
 
 __device__ __forceinline__ float gelu_tanh_(float z) {
@@ -370,6 +451,33 @@ RB_EXPORT int rb_norm_add(float* x, const float* y, const float* w, float eps, i
   else RB_FAIL("rb_norm_add: unknown dtype %d", rounded_dtype);
 #undef GO
   RB_CHECK_LAUNCH("rb_norm_add");
+  return 0;
+}
+
+// x [T, E] += y / rms(y) * w (fresh: x = that; x is then only written), and h [T, E] = x / rms(x) * w2 of the new rows.
+RB_EXPORT int rb_norm_add_norm(float* x, const float* y, const float* w, float eps, int T, int E, int fresh, void* h, int h_dtype,
+                               const float* w2, float eps2, cudaStream_t stream) {
+  if (T == 0) return 0;
+  RB_REQUIRE(E > 0 && h != nullptr && w2 != nullptr, "rb_norm_add_norm: bad arguments (width %d)", E);
+  RB_REQUIRE(h_dtype == RB_F32 || h_dtype == RB_BF16, "rb_norm_add_norm: unknown dtype %d", h_dtype);
+  const bool vec = E % 4 == 0 && E <= 16384 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+                   (uintptr_t)w2 % 16 == 0 && (uintptr_t)h % 16 == 0;
+  const int n4 = E / 4;
+  const int nv = n4 <= 256 ? 1 : (n4 <= 1024 ? 2 : 4);
+  const int threads = vec ? ((n4 + nv - 1) / nv + 31) / 32 * 32 : 256;
+#define GO(TT, V, N) RB_LAUNCH("norm_add_norm_kernel", (norm_add_norm_kernel<TT, V, N>), T, threads, 0, stream, x, y, w, eps, E, fresh, (TT*)h, w2, eps2)
+#define PICK(TT)                         \
+  do {                                   \
+    if (!vec) GO(TT, false, 1);          \
+    else if (nv == 1) GO(TT, true, 1);   \
+    else if (nv == 2) GO(TT, true, 2);   \
+    else GO(TT, true, 4);                \
+  } while (0)
+  if (h_dtype == RB_F32) PICK(float);
+  else PICK(__nv_bfloat16);
+#undef PICK
+#undef GO
+  RB_CHECK_LAUNCH("rb_norm_add_norm");
   return 0;
 }
 

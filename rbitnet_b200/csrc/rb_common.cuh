@@ -246,16 +246,30 @@ struct RbPagedLayer {
 };
 
 // ---------------------------------------------------------------- options of the next attention call
-// rb_attention_next(sinks, softcap) (attention_simple.cu) sets them for the calling thread's next attention launch,
+// rb_attention_next(sinks, softcap, keep_first) (attention_simple.cu) sets them for the calling thread's next attention launch,
 // which takes them with rb_attention_take (and so clears them):
 //   sinks    float32 [H] or null: the softmax's denominator of head h also holds exp(sinks[h]) (no key, no value,
 //            not scaled, counted once)
 //   softcap  > 0: score <- softcap * tanh(score / softcap), after the scale and before the softmax
+//   keep_first  > 0, with a window: the first so many positions of a sequence stay visible wherever the window is
 struct RbAttentionOptions {
   const float* sinks = nullptr;
   float softcap = 0.f;
+  int keep_first = 0;
 };
 RbAttentionOptions rb_attention_take();
+
+// The tiles of `tile` keys that a group of rows visits: those that hold keys lo .. hi, and before them those that hold
+// the first `keep` keys (tiles that are both count once).  at(i), i in 0 .. n - 1, is the number of the i-th.
+struct RbKeyTiles {
+  int kept, first, n;
+  __device__ __forceinline__ RbKeyTiles(int lo, int hi, int keep, int tile) {
+    first = lo / tile;
+    kept = min(first, (keep + tile - 1) / tile);
+    n = kept + hi / tile + 1 - first;
+  }
+  __device__ __forceinline__ int at(int i) const { return i < kept ? i : first + (i - kept); }
+};
 
 // ---------------------------------------------------------------- the checked build
 // With -DRB_CHECKED (RBITNET_CHECKED=1 when the library is built) every cache address that goes

@@ -4,7 +4,7 @@
 //   z = Wr h (float32), s = softmax(z) over all n outputs; the choice score of output e is s_e + c_e
 //   outputs form `groups` equal groups of neighbours; a group's score is its largest choice score, and
 //   only outputs of the `keep` best groups can be chosen; the `top` largest choice scores are chosen;
-//   a chosen output's weight is s_e (not renormalised)
+//   a chosen output's weight is s_e (not renormalised unless asked for, see rb_route_next)
 //   outputs n_experts .. n-1 are identity experts: their result is the input row itself
 //   result_t = sum over the chosen e of s_e * expert_e(h_t)
 //
@@ -26,6 +26,12 @@
 namespace {
 
 // ---------------------------------------------------------------- router
+// What becomes of the chosen outputs' weights: with `normalize` each is divided by their sum + floor; then times scale.
+struct RouteWeighing {
+  int normalize = 0;
+  float floor = 0.f;
+  float scale = 1.0f;
+};
 // A block of 8 warps takes TB tokens (up to 8).  Its warps share the router's outputs: a warp makes output e for all
 // of the block's tokens at once, so that a row of Wr is read once per block (lanes stride over k four values at a
 // time; a token's sum is the lanes' partial sums added in a fixed tree, whatever other tokens the block holds).  Then
@@ -34,7 +40,8 @@ namespace {
 // its `top` outputs and their weights.
 __device__ __forceinline__ void route_select(float* z, float* choice, float* gscore, const float* __restrict__ correction,
                                              int n, int top, int groups, int keep, int lane, int* __restrict__ ids,
-                                             float* __restrict__ weights, int64_t t, int scoring = 0) {
+                                             float* __restrict__ weights, int64_t t, int scoring = 0,
+                                             RouteWeighing weighing = RouteWeighing()) {
   if (scoring == 2) {
     for (int e = lane; e < n; e += 32) choice[e] = z[e] + (correction != nullptr ? correction[e] : 0.f);
     __syncwarp();
@@ -120,6 +127,25 @@ __device__ __forceinline__ void route_select(float* z, float* choice, float* gsc
     __syncwarp();
     for (int j = lane; j < top; j += 32) mine[j] = expf(mine[j] - m) / sum;
   }
+  if (weighing.normalize || weighing.scale != 1.0f) {
+    float* mine = weights + (int64_t)t * top;
+    __syncwarp();
+    float by = weighing.scale;
+    if (weighing.normalize) {
+      float sum = 0.f;
+      for (int j = lane; j < top; j += 32) sum += mine[j];
+      by /= rb_warp_sum(sum) + weighing.floor;
+      __syncwarp();
+    }
+    for (int j = lane; j < top; j += 32) mine[j] *= by;
+  }
+}
+
+thread_local RouteWeighing t_weighing;          // of this thread's next choice
+RouteWeighing take_weighing() {
+  const RouteWeighing w = t_weighing;
+  t_weighing = RouteWeighing();
+  return w;
 }
 
 constexpr int ROUTE_TB = 8;
@@ -129,7 +155,7 @@ __global__ void __launch_bounds__(256) route_kernel(int* __restrict__ ids, float
                                                     const TI* __restrict__ h, int64_t ldh,
                                                     const float* __restrict__ Wr, const float* __restrict__ correction,
                                                     int T, int K, int n_out, int top, int groups, int keep, int TB, int vec,
-                                                    int scoring, int n_extra, float* __restrict__ extra) {
+                                                    int scoring, int n_extra, float* __restrict__ extra, RouteWeighing weighing) {
   rb_pdl_launch_dependents();
   extern __shared__ float s_route[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -203,7 +229,7 @@ __global__ void __launch_bounds__(256) route_kernel(int* __restrict__ ids, float
   if (warp >= nt) return;
   float* z = s_route + (size_t)warp * per_token;     // scores, choice scores, group scores, kept groups
   for (int i = lane; i < n_extra; i += 32) extra[(int64_t)(t0 + warp) * n_extra + i] = z[n_out + i];
-  route_select(z, z + n, z + 2 * n, correction, n_out, top, groups, keep, lane, ids, weights, t0 + warp, scoring);
+  route_select(z, z + n, z + 2 * n, correction, n_out, top, groups, keep, lane, ids, weights, t0 + warp, scoring, weighing);
 }
 
 // Many tokens: the router's sums as a tiled float32 product (16 tokens by 64 outputs a block, k in steps of 32 through
@@ -266,7 +292,7 @@ __global__ void __launch_bounds__(256) route_logits_kernel(float* __restrict__ z
 __global__ void __launch_bounds__(128) route_select_kernel(int* __restrict__ ids, float* __restrict__ weights,
                                                            const float* __restrict__ zg, const float* __restrict__ correction,
                                                            int T, int n, int top, int groups, int keep, int scoring,
-                                                           int n_extra, float* __restrict__ extra) {
+                                                           int n_extra, float* __restrict__ extra, RouteWeighing weighing) {
   rb_pdl_launch_dependents();
   extern __shared__ float s_route[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -278,7 +304,7 @@ __global__ void __launch_bounds__(128) route_select_kernel(int* __restrict__ ids
   for (int e = lane; e < n; e += 32) z[e] = zg[(int64_t)t * ldz + e];
   for (int i = lane; i < n_extra; i += 32) extra[(int64_t)t * n_extra + i] = zg[(int64_t)t * ldz + n + i];
   __syncwarp();
-  route_select(z, z + n, z + 2 * n, correction, n, top, groups, keep, lane, ids, weights, t, scoring);
+  route_select(z, z + n, z + 2 * n, correction, n, top, groups, keep, lane, ids, weights, t, scoring, weighing);
 }
 
 // ---------------------------------------------------------------- plan
@@ -379,7 +405,8 @@ __global__ void gather_scaled_kernel(T* __restrict__ xp, const T* __restrict__ h
 
 // ---------------------------------------------------------------- weighted sum
 // What the weighted sum adds and leaves besides (null: not):
-//   shared, gate   x also takes sigmoid(gate[t * ldg]) * shared[t, :] in (a further expert that every token uses)
+//   shared, gate   x also takes sigmoid(gate[t * ldg]) * shared[t, :] in (a further expert that every token uses; without
+//                  a gate the whole of it)
 //   norm_w         norm_out[t, :] = norm_w tanh(norm_alpha x[t, :]) + norm_b of the finished row
 struct CombineTail {
   const float* shared = nullptr;
@@ -399,7 +426,7 @@ __global__ void combine_kernel(float* __restrict__ x, int64_t ldx, const float* 
   rb_pdl_launch_dependents();
   rb_pdl_wait();
   const int t = blockIdx.x;
-  const float sg = tail.shared != nullptr ? 1.0f / (1.0f + expf(-tail.gate[(int64_t)t * tail.ldg])) : 0.f;
+  const float sg = tail.gate == nullptr ? 1.0f : tail.shared != nullptr ? 1.0f / (1.0f + expf(-tail.gate[(int64_t)t * tail.ldg])) : 0.f;
   if (vec4) {
     // four columns a thread: 16-byte loads of the experts' rows and of the residual stream
     for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4; c < E; c += gridDim.y * blockDim.x * 4) {
@@ -537,6 +564,7 @@ __global__ void square_relu_kernel(T* __restrict__ out, const T* __restrict__ in
 static int route_impl(int* ids, float* weights, const void* h, int64_t ldh, int h_dtype, const float* Wr,
                       const float* correction, int T, int K, int n, int top, int groups, int keep, float* z_scratch,
                       int scoring, int n_extra, float* extra, cudaStream_t stream) {
+  const RouteWeighing weighing = take_weighing();
   if (T == 0) return 0;
   RB_REQUIRE(scoring >= 0 && scoring <= 2, "rb_route: scoring %d is not built (0: softmax, 1: sigmoid, 2: softmax over the chosen)", scoring);
   RB_REQUIRE(n_extra >= 0 && (n_extra == 0 || extra != nullptr), "rb_route: %d extra rows and nowhere to leave them", n_extra);
@@ -557,7 +585,7 @@ static int route_impl(int* ids, float* weights, const void* h, int64_t ldh, int 
       RB_FAIL("rb_route: unknown dtype %d", h_dtype);
     RB_CHECK_LAUNCH("rb_route");
     RB_LAUNCH("route_select_kernel", (route_select_kernel), (T + 3) / 4, 128, smem_sel, stream, ids, weights, z_scratch, correction, T, n, top,
-              groups, keep, scoring, n_extra, extra);
+              groups, keep, scoring, n_extra, extra, weighing);
     RB_CHECK_LAUNCH("rb_route");
     return 0;
   }
@@ -568,9 +596,9 @@ static int route_impl(int* ids, float* weights, const void* h, int64_t ldh, int 
   const int elem = h_dtype == RB_F32 ? 4 : 2;
   const int vec = K % 4 == 0 && ldh % 4 == 0 && (uintptr_t)h % (4 * elem) == 0 && (uintptr_t)Wr % 16 == 0;
   if (h_dtype == RB_F32)
-    RB_LAUNCH("route_kernel", (route_kernel<float>), blocks, 256, smem, stream, ids, weights, (const float*)h, ldh, Wr, correction, T, K, n, top, groups, keep, TB, vec, scoring, n_extra, extra);
+    RB_LAUNCH("route_kernel", (route_kernel<float>), blocks, 256, smem, stream, ids, weights, (const float*)h, ldh, Wr, correction, T, K, n, top, groups, keep, TB, vec, scoring, n_extra, extra, weighing);
   else if (h_dtype == RB_BF16)
-    RB_LAUNCH("route_kernel", (route_kernel<__nv_bfloat16>), blocks, 256, smem, stream, ids, weights, (const __nv_bfloat16*)h, ldh, Wr, correction, T, K, n, top, groups, keep, TB, vec, scoring, n_extra, extra);
+    RB_LAUNCH("route_kernel", (route_kernel<__nv_bfloat16>), blocks, 256, smem, stream, ids, weights, (const __nv_bfloat16*)h, ldh, Wr, correction, T, K, n, top, groups, keep, TB, vec, scoring, n_extra, extra, weighing);
   else
     RB_FAIL("rb_route: unknown dtype %d", h_dtype);
   RB_CHECK_LAUNCH("rb_route");
@@ -581,6 +609,13 @@ RB_EXPORT int rb_route(int* ids, float* weights, const void* h, int64_t ldh, int
                        const float* correction, int T, int K, int n, int top, int groups, int keep, float* z_scratch,
                        cudaStream_t stream) {
   return route_impl(ids, weights, h, ldh, h_dtype, Wr, correction, T, K, n, top, groups, keep, z_scratch, 0, 0, nullptr, stream);
+}
+
+// The next rb_route_scored or rb_route_select_scored call of this thread divides the chosen outputs' weights by their sum
+// + floor (if normalize) and multiplies them by scale.
+RB_EXPORT int rb_route_next(int normalize, float floor, float scale) {
+  t_weighing.normalize = normalize; t_weighing.floor = floor; t_weighing.scale = scale;
+  return 0;
 }
 
 // The same with the variants: scoring (0: softmax over the outputs, 1: a sigmoid per output, 2:
@@ -603,7 +638,7 @@ RB_EXPORT int rb_route_select(int* ids, float* weights, const float* z, const fl
   const size_t smem_sel = (size_t)4 * (2 * n + 2 * groups) * sizeof(float);
   RB_REQUIRE(smem_sel <= 48 * 1024, "rb_route_select: %d router outputs are more than a block's shared memory holds", n);
   RB_LAUNCH("route_select_kernel", (route_select_kernel), (T + 3) / 4, 128, smem_sel, stream, ids, weights, z, correction, T, n, top,
-            groups, keep, 0, 0, (float*)nullptr);
+            groups, keep, 0, 0, (float*)nullptr, RouteWeighing());
   RB_CHECK_LAUNCH("rb_route_select");
   return 0;
 }
@@ -611,6 +646,7 @@ RB_EXPORT int rb_route_select(int* ids, float* weights, const float* z, const fl
 // The choice with the variants of rb_route_scored, from sums z [T, n + n_extra] that a product has left.
 RB_EXPORT int rb_route_select_scored(int* ids, float* weights, const float* z, const float* correction, int T, int n, int top,
                                      int groups, int keep, int scoring, int n_extra, float* extra, cudaStream_t stream) {
+  const RouteWeighing weighing = take_weighing();
   if (T == 0) return 0;
   RB_REQUIRE(n > 0 && top > 0 && top <= n && n_extra >= 0 && (n_extra == 0 || extra != nullptr),
              "rb_route_select_scored: bad sizes outputs=%d top=%d extra=%d", n, top, n_extra);
@@ -619,7 +655,7 @@ RB_EXPORT int rb_route_select_scored(int* ids, float* weights, const float* z, c
   const size_t smem_sel = (size_t)4 * (2 * n + 2 * groups) * sizeof(float);
   RB_REQUIRE(smem_sel <= 48 * 1024, "rb_route_select_scored: %d router outputs are more than a block's shared memory holds", n);
   RB_LAUNCH("route_select_kernel", (route_select_kernel), (T + 3) / 4, 128, smem_sel, stream, ids, weights, z, correction, T, n, top,
-            groups, keep, scoring, n_extra, extra);
+            groups, keep, scoring, n_extra, extra, weighing);
   RB_CHECK_LAUNCH("rb_route_select_scored");
   return 0;
 }
@@ -672,7 +708,8 @@ RB_EXPORT int rb_routed_gather_scaled(void* xp, const void* h, int64_t ldh, int 
   return 0;
 }
 
-// The next rb_routed_combine call of this thread also adds sigmoid(gate[t * ldg]) * shared[t, :] (float32 [T, E]; null: not)
+// The next rb_routed_combine call of this thread also adds sigmoid(gate[t * ldg]) * shared[t, :] (float32 [T, E]; null: not;
+// gate null: shared[t, :] as it is)
 // and leaves norm_w tanh(norm_alpha x) + norm_b of the finished rows in norm_out ([T, E] of the input rows' type; norm_w
 // null: not).
 static thread_local CombineTail t_combine;
@@ -689,7 +726,6 @@ RB_EXPORT int rb_routed_combine(float* x, int64_t ldx, const float* y, const voi
   const CombineTail tail = t_combine;
   t_combine = CombineTail();
   if (T == 0) return 0;
-  RB_REQUIRE(tail.shared == nullptr || tail.gate != nullptr, "rb_routed_combine: a shared result without its gate");
   RB_REQUIRE(tail.norm_w == nullptr || (tail.norm_b != nullptr && tail.norm_out != nullptr), "rb_routed_combine: a norm without its place");
   const int elem = h_dtype == RB_F32 ? 4 : 2;
   const int vec4 = E % 4 == 0 && ldx % 4 == 0 && ldh % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 &&

@@ -92,6 +92,9 @@ class Model:
                     if theirs is not None and theirs.window and (not need.window or need.window > theirs.window):
                         raise ValueError(f"schedule entry {e} sees {need.window or 'all'} keys but reads the cache of "
                                          f"entry {entry.reads_cache_of}, which keeps only the last {theirs.window}")
+                    if theirs is not None and theirs.window and need.keep_first > theirs.keep_first:
+                        raise ValueError(f"schedule entry {e} sees the first {need.keep_first} keys but reads the cache of "
+                                         f"entry {entry.reads_cache_of}, which keeps only the first {theirs.keep_first}")
             st = mixer.state_need()
             if st:
                 state_needs[e] = st            # one StateNeed, or several by name
@@ -154,12 +157,18 @@ class Model:
             # plus a row chosen by the pair (previous token, token); the previous token belongs to the sequence
             x = ops.embed_pairs(meta, self.embedding, self.embedding_scale, self.embedding_pairs, self.pair_hash,
                                 ctx.cache.state(PREVIOUS_TOKEN))
+        schedule, pending = self.spec.schedule, None
         if self.embedding_norm is not None:
-            x = self.embedding_norm.forward(ctx, x, out_dtype=torch.float32)
+            # together with the first block's first norm, where both are RMS norms and the block takes finished rows
+            first = self.blocks[schedule[0].layer]
+            if getattr(first, "takes_finished_rows", False) and hasattr(self.embedding_norm, "start_with") \
+                    and not schedule[0].adds_embedding:
+                x, pending = self.embedding_norm.start_with(ctx, x, first.first_norm())
+            else:
+                x = self.embedding_norm.forward(ctx, x, out_dtype=torch.float32)
         s = self.residual_streams
         if s > 1:
             x = ops.streams_expand(x, s)                                      # [T, s * E]: every stream starts as the embedding
-        schedule, pending = self.spec.schedule, None
         taps = getattr(ctx, "layer_outputs", None)                            # a list: the residual sum after every run of a layer
         # a schedule that adds the embedded rows again later keeps them (the blocks change x in place)
         x0 = x.clone() if any(en.adds_embedding for en in schedule) else None
@@ -197,15 +206,21 @@ class Model:
             after = self.blocks[schedule[e + 1].layer] if e + 1 < len(schedule) else None
             hand_on = getattr(after, "chains_norms", False) and not schedule[e + 1].adds_embedding
             next_norm = after.first_norm() if hand_on else None
+            if after is None and s == 1 and meta.want_every_row and getattr(block, "takes_finished_rows", False):
+                next_norm = self.final_norm                   # the last block leaves the head's input rows
             pending = block.run(ctx, x, e, pending=pending, next_norm=next_norm)
             if taps is not None:
                 taps.append(ops.streams_sum(x, s) if s > 1 else x.clone())
         if meta.n_want == 0:
             return None
-        rows = x if meta.want_every_row else ops.gather_rows(x, meta.want_rows)
-        if s > 1:
-            rows = ops.streams_sum(rows, s)
-        h = self.final_norm.forward(ctx, rows)
+        if isinstance(pending, torch.Tensor) and meta.want_every_row and \
+                getattr(self.blocks[schedule[-1].layer], "takes_finished_rows", False):
+            h = pending
+        else:
+            rows = x if meta.want_every_row else ops.gather_rows(x, meta.want_rows)
+            if s > 1:
+                rows = ops.streams_sum(rows, s)
+            h = self.final_norm.forward(ctx, rows)
         logits = ops.linear(h, self.head, out_dtype=torch.float32, scale=self.logit_scale)
         if self.logit_softcap > 0.0:
             logits = ops.softcap(logits, self.logit_softcap)          # cap * tanh(logits / cap), float32

@@ -23,7 +23,7 @@ _SIGNATURES = {
     "rb_gemm_simple": [P, L, I, P, L, P, L, I, I, I, I, I, F, P],
     "rb_gemm_simple_batched": [P, L, I, P, L, P, L, I, I, I, I, I, F, I, L, L, L, P],
     "rb_per_head_few_rows": [P, L, I, P, L, I, P, I, I, I, I, I, P],
-    "rb_gemm_simple_next": [P, P, L, L],
+    "rb_gemm_simple_next": [P, P, L, L, I],
     "rb_stream_step": [P, I, I, I, P, P, I, P, P, P, P, F, P, I, P, P],
     "rb_streams_expand": [P, P, I, I, I, P],
     "rb_streams_sum": [P, P, I, I, I, P],
@@ -91,9 +91,16 @@ _SIGNATURES = {
     "rb_attention_prefill_tc": [P, P, P, P, L, P, I, I, P, P, P, P, I, I, I, I, F, I, P, P, I, I, P],
     "rb_attention_decode_tma": [P, P, P, P, L, P, I, I, P, P, I, I, I, I, F, I, P, P, I, P],
     "rb_attention_decode_static": [P, P, P, P, P, I, I, P, P, I, I, I, I, F, I, I, P],
-    "rb_attention_next": [P, F],
+    "rb_attention_next": [P, F, I],
     "rb_gla_shared_decays": [],
+    "rb_ssd_conv": [P, I, L, P, L, I, P, P, P, P, P, P, I, I, I, P],
+    "rb_ssd_step": [P, P, L, I, I, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
+    "rb_ssd_scan": [P, P, I, L, P, L, I, I, P, P, P, P, P, P, P, I, I, I, I, I, P],
+    "rb_ssd_chunked": [P, P, L, P, L, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
+    "rb_ssd_chunked_supports": [I, I],
     "rb_round_rows": [P, I, P, L, P],
+    "rb_norm_add_norm": [P, P, P, F, I, I, I, P, I, P, F, P],
+    "rb_route_next": [I, F, F],
     "rb_norm_add": [P, P, P, F, I, I, P, I, P],
     "rb_token_gate": [P, I, P, L, P, I, P, I, I, P],
     "rb_embed_pairs": [P, P, P, I, P, P, P, P, I, I, I, F, I, I, I, I, P],
@@ -134,6 +141,7 @@ class KernelLibrary:
         self.declare("rb_gemm_tc_splits", [I, I, I])
         self.declare("rb_gemm_tc_workspace_bytes", [], restype=ctypes.c_longlong)
         self.declare("rb_gated_delta_chunk_floats", [I, I], restype=ctypes.c_longlong)
+        self.declare("rb_ssd_chunk_floats", [I, I], restype=ctypes.c_longlong)
         self.declare("rb_gemm_tc_set_workspace", [P, L])
         self.declare("rb_gemm_tc_plan", [I, I, I, I, I, I, P])
         self.declare("rb_gemm_tc_share_for_test", [I])
@@ -144,8 +152,9 @@ class KernelLibrary:
         self.declare("rb_gemm_tc_norm_parts", [I])
         self.declare("rb_gemm_tc_gated_act", [F, F, F])
         self.declare("rb_gemm_tc_gated_gelu", [])
+        self.declare("rb_gemm_tc_gated_relu", [])
         self.declare("rb_gemm_tc_bias", [P])
-        self.declare("rb_gemm_tc_per_head", [I, I, I, P, L])
+        self.declare("rb_gemm_tc_per_head", [I, I, I, P, L, I])
         self.declare("rb_gemm_tc_leave_tanh", [P, L, P, P, F])
         self.declare("rb_device_sm_count", [])
         self.declare("rb_is_checked_build", [])

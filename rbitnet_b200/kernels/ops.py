@@ -171,6 +171,8 @@ class CudaOps:
         self.per_head_on_tensor_cores = True
         #: so does gated linear attention
         self.gla_in_chunks = True
+        #: in bfloat16 mode a state-space mixer takes runs of several tokens in chunks of 64 (else token by token)
+        self.ssd_in_chunks = True
         #: a decode step's delta rule (convolution to gate) is one kernel while rows x heads fit the SMs
         self.fuse_delta_step = True
         #: tensor-core products of more than 256 tokens may share a weight tile's inner dimension
@@ -338,7 +340,7 @@ class CudaOps:
                           64 if 64 < T <= 256 else 0, float(scale), self._stream())
         else:
             if bias is not None:
-                self.lib.call("rb_gemm_simple_next", _ptr(bias), c_void_p(0), 0, 0, launches=0)
+                self.lib.call("rb_gemm_simple_next", _ptr(bias), c_void_p(0), 0, 0, 1, launches=0)
             self.lib.call("rb_gemm_simple", _ptr(out), out.stride(0), _CODE[out.dtype], _ptr(x), x.stride(0),
                           _ptr(weight.w), weight.w.stride(0), self.code, T, N, K, acc, float(scale), self._stream())
             if act is not None:
@@ -400,7 +402,7 @@ class CudaOps:
 
     def _gated_act(self, out: torch.Tensor, gu: torch.Tensor, inner: int, block: int, act, bias=None) -> None:
         """out = the gated activation ``act`` of float32 rows [gate | up], by a kernel of its own."""
-        kind, (alpha, limit, shift) = (1, (1.0, 0.0, 0.0)) if act == "gelu_tanh" else (0, act)
+        kind, (alpha, limit, shift) = ({"gelu_tanh": 1, "relu": 2}[act], (1.0, 0.0, 0.0)) if isinstance(act, str) else (0, act)
         self.lib.call("rb_gated_act", _ptr(out), _ptr(gu), self.code, F32, gu.shape[0], inner, gu.stride(0), block, kind,
                       float(alpha), float(limit), float(shift), _ptr(bias), self._stream())
 
@@ -408,13 +410,15 @@ class CudaOps:
         """For the next gated tensor-core product of this thread."""
         if act == "gelu_tanh":
             self.lib.call("rb_gemm_tc_gated_gelu", launches=0)
+        elif act == "relu":
+            self.lib.call("rb_gemm_tc_gated_relu", launches=0)
         else:
             self.lib.call("rb_gemm_tc_gated_act", float(act[0]), float(act[1]), float(act[2]), launches=0)
 
     def gated_linear(self, x: torch.Tensor, weight: GateUpWeight, act=None) -> torch.Tensor:
         """silu(x Wg^T) * (x Wu^T) -> [T, inner] in the compute dtype.  ``act`` = (alpha, limit, shift):
         g' sigmoid(alpha g') (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit) instead (limit 0: none);
-        "gelu_tanh": gelu(g) u, gelu in its tanh form.  The weight's biases are added to g and u first."""
+        "gelu_tanh": gelu(g) u, gelu in its tanh form; "relu": max(g, 0) u.  The weight's biases are added to g and u first."""
         if act is None and weight.bias is not None:
             act = (1.0, 0.0, 0.0)
         if act is not None and weight.block == 16 and not isinstance(x, NormedRows) and self.fuse_gated_act \
@@ -516,18 +520,23 @@ class CudaOps:
         return z
 
     def attention(self, q: torch.Tensor, meta, view, n_heads: int, scale: float,
-                  window: Optional[int], sinks: Optional[torch.Tensor] = None, softcap: float = 0.0) -> torch.Tensor:
+                  window: Optional[int], sinks: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                  keep_first: int = 0) -> torch.Tensor:
         """Each new token's queries over its sequence's cached keys up to its own position.  ``sinks`` (float32 [H]):
         head h's softmax denominator also holds exp(sinks[h]); ``softcap`` > 0: score <- softcap * tanh(score /
-        softcap).  Every attention kernel of the library takes both."""
+        softcap); ``keep_first`` > 0 with a window: the sequence's first so many positions stay visible wherever the window
+        is.  Every attention kernel of the library takes them all."""
         T, H, D = q.shape
         Kh = view.n_kv_heads
         out = torch.empty((T, H * D), dtype=self.dtype, device=self.device)
         win = int(window or 0)
-        if sinks is not None or softcap > 0.0:
+        keep = int(keep_first or 0) if win else 0
+        if sinks is not None or softcap > 0.0 or keep > 0:
             if sinks is not None:
                 self._check(sinks, torch.float32, "attention sinks")
-            self.lib.call("rb_attention_next", _ptr(sinks), float(softcap), launches=0)
+            self.lib.call("rb_attention_next", _ptr(sinks), float(softcap), keep, launches=0)
+        # the most keys a new token can have to visit, in whole tiles
+        context = int(meta.max_context) if not win else min(int(meta.max_context), win + 126 + (keep + 63) // 64 * 64)
         # keys and values that are the same rows (attention through latents) let the tcgen05 kernel take wider heads
         shared = 1 if view.k.data_ptr() == view.v.data_ptr() else 0
         on_tc = self.dtype == torch.bfloat16 and self.prefill_on_tcgen05 and \
@@ -537,9 +546,9 @@ class CudaOps:
         on_tma = few and self.decode_on_tma and self.lib.raw("rb_attention_decode_tma_supports")(H, Kh, D, view.page_size)
         if few and (on_tma or not (on_tc and shared)):
             if on_tma:
-                n_splits = self.lib.raw("rb_attention_decode_tma_parts")(T * Kh, max(1, -(-meta.max_context // 64)), D)
+                n_splits = self.lib.raw("rb_attention_decode_tma_parts")(T * Kh, max(1, -(-context // 64)), D)
             else:
-                n_splits = self.lib.raw("rb_attention_decode_parts")(T, Kh, meta.max_context)
+                n_splits = self.lib.raw("rb_attention_decode_parts")(T, Kh, context)
             part_o = part_ml = None
             # the parts of a small grid are a thread-block cluster and merge on chip
             on_chip = on_tma and bool(self.lib.raw("rb_attention_decode_tma_on_chip")(T * Kh, n_splits, D))
@@ -563,7 +572,7 @@ class CudaOps:
             parts, part_o, part_ml = 1, None, None
             if meta.single_token:
                 # a decode step whose heads the decode kernels do not take: few row tiles, the keys cut into parts
-                parts = self.lib.raw("rb_attention_prefill_tc_parts")(n_tiles, Kh, int(meta.max_context))
+                parts = self.lib.raw("rb_attention_prefill_tc_parts")(n_tiles, Kh, context)
             if parts > 1:
                 part_o = torch.empty((T, H, parts, D), dtype=torch.float32, device=self.device)
                 part_ml = torch.empty((T, H, parts, 2), dtype=torch.float32, device=self.device)
@@ -963,6 +972,23 @@ class CudaOps:
             return None
         return x if rounded is None else rounded
 
+    def norm_add_norm(self, x: Optional[torch.Tensor], y: torch.Tensor, w: torch.Tensor, eps: float, next_w: torch.Tensor,
+                      next_eps: float):
+        """In one launch: x += y / rms(y) * w, row by row in float32 (``x`` None: x is that alone), and the rows
+        x / rms(x) * next_w of the norm after it in the compute dtype.  Returns (x, those rows)."""
+        self._check(y, torch.float32, "norm_add_norm result")
+        T, E = y.shape
+        fresh = x is None
+        if fresh:
+            x = torch.empty_like(y)
+        self._check(x, torch.float32, "norm_add_norm target")
+        if y.shape != x.shape or w.shape[0] != E or next_w.shape[0] != E:
+            raise KernelError(f"norm_add_norm: shapes {tuple(x.shape)}, {tuple(y.shape)}, {tuple(w.shape)}, {tuple(next_w.shape)}")
+        h = torch.empty((T, E), dtype=self.dtype, device=self.device)
+        self.lib.call("rb_norm_add_norm", _ptr(x), _ptr(y), _ptr(w), float(eps), T, E, 1 if fresh else 0, _ptr(h), self.code,
+                      _ptr(next_w), float(next_eps), self._stream())
+        return x, h
+
     def token_gate(self, a: torch.Tensor, table: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
         """gelu_tanh(a[t]) * table[ids[t]] -> [T, dim] in the compute dtype (a: float32 [T, dim])."""
         self._check(a, torch.float32, "token_gate rows")
@@ -1083,6 +1109,45 @@ class CudaOps:
                       at["g"], T, H, Dv, float(p.norm_eps), 1, 1, self._stream())
         return out
 
+    # ------------------------------------------------------------------ state space with a decay per head and token
+    def state_space(self, proj: torch.Tensor, p, state, meta) -> torch.Tensor:
+        """The recurrence of ``parts.ssd.StateSpace`` ``p`` on float32 rows [z | x | B | C | dt] of its stacked projection:
+        convolution and SiLU of [x | B | C], the state's steps with their read-out and the heads' own terms, times
+        silu(z), as float32 [T, H * value_dim] (the norm over it is the caller's).  ``state["S"]`` [slots, H, state rows,
+        value_dim] and ``state["tail"]`` move on."""
+        self._check(proj, torch.float32, "state_space projections")
+        T, H, P, N, G, K = proj.shape[0], p.n_heads, p.value_dim, p.state_dim, p.n_groups, p.taps
+        at, C = p.offsets(), H * P + 2 * G * N
+        first, count, tok_first, n_runs = self._runs(meta)
+        tail = state.get("tail")
+        out = torch.empty((T, H * P), dtype=torch.float32, device=self.device)
+        if first is None:
+            # one token per sequence: convolution to gate in one launch
+            self.lib.call("rb_ssd_step", _ptr(out), _ptr(proj), proj.stride(0), at["z"], at["x"], at["dt"], _ptr(p.conv_w),
+                          _ptr(p.conv_b), _ptr(p.dt_bias), _ptr(p.a_log), _ptr(p.d_skip), _ptr(state["S"]), _ptr(tail),
+                          _ptr(meta.tok_slot), _ptr(meta.tok_pos), T, H, P, N, G, K, self._stream())
+            return out
+        u = torch.empty((T, -(-C // 8) * 8), dtype=self.dtype, device=self.device)
+        self.lib.call("rb_ssd_conv", _ptr(u), self.code, u.stride(0), _ptr(proj), proj.stride(0), at["x"], _ptr(p.conv_w),
+                      _ptr(p.conv_b), _ptr(tail), _ptr(tok_first), _ptr(meta.tok_slot), _ptr(meta.tok_pos), T, C, K,
+                      self._stream())
+        if K > 1:
+            self.lib.call("rb_conv_tail_update", _ptr(tail), _ptr(proj), proj.stride(0), at["x"], F32, c_void_p(0), _ptr(first),
+                          _ptr(count), _ptr(meta.tok_slot), _ptr(meta.tok_pos), n_runs, C, K, self._stream())
+        if self.dtype == torch.bfloat16 and self.ssd_in_chunks and self.lib.raw("rb_ssd_chunked_supports")(P, N):
+            run_chunk0, chunk_row, chunk_len, n_chunks = self._delta_chunks(meta, 64)
+            scratch = torch.empty((n_chunks * H * self.lib.raw("rb_ssd_chunk_floats")(P, N),), dtype=torch.float32,
+                                  device=self.device)
+            self.lib.call("rb_ssd_chunked", _ptr(out), _ptr(u), u.stride(0), _ptr(proj), proj.stride(0), at["z"], at["dt"],
+                          _ptr(p.dt_bias), _ptr(p.a_log), _ptr(p.d_skip), _ptr(state["S"]), _ptr(scratch), _ptr(first), _ptr(count),
+                          _ptr(run_chunk0), _ptr(chunk_row), _ptr(chunk_len), _ptr(meta.tok_slot), n_runs, n_chunks, H, P, N, G,
+                          self._stream(), launches=3)
+        else:
+            self.lib.call("rb_ssd_scan", _ptr(out), _ptr(u), self.code, u.stride(0), _ptr(proj), proj.stride(0), at["z"], at["dt"],
+                          _ptr(p.dt_bias), _ptr(p.a_log), _ptr(p.d_skip), _ptr(state["S"]), _ptr(first), _ptr(count),
+                          _ptr(meta.tok_slot), n_runs, H, P, N, G, self._stream())
+        return out
+
     # ------------------------------------------------------------------ attention through latents
     def latent_norm_append(self, down: torch.Tensor, q_rank: int, kv_rank: int, wq: torch.Tensor, wkv: torch.Tensor,
                            eps: float, meta, view, rot_dim: int = 0, table=None) -> torch.Tensor:
@@ -1135,27 +1200,29 @@ class CudaOps:
 
     def _per_head(self, out: torch.Tensor, head_c: int, x: torch.Tensor, head_x: int, weight: PerHeadWeight, gate=None) -> None:
         """out[:, h * head_c : + n_out] = x[:, h * head_x : + n_in] * W_h^T for many rows (the other columns of a head are
-        undefined afterwards); ``gate`` = (float32 rows, first column): times sigmoid of column h * n_out + n of them."""
+        undefined afterwards); ``gate`` = (float32 rows, first column[, "head"]): see ``per_head_linear``."""
         T, H, N, K = x.shape[0], weight.heads, weight.n_out, weight.n_in
-        gate_ptr, ldg = c_void_p(0), 0
+        gate_ptr, ldg, by_head = c_void_p(0), 0, gate is not None and gate[2:] == ("head",)
         if gate is not None:
             self._check(gate[0], torch.float32, "per-head gate")
             gate_ptr, ldg = c_void_p(gate[0].data_ptr() + gate[1] * 4), gate[0].stride(0)
         if self.per_head_on_tensor_cores and self._tensor_core_ok(x, weight.w.view(H * N, K)) and K % 8 == 0 and head_x % 8 == 0:
             whole_boxes = -(-N // 128) * 128 <= head_c and head_c % 8 == 0
             tile = 64 if T <= 256 or not whole_boxes or gate is not None else 256
-            self.lib.call("rb_gemm_tc_per_head", H, int(head_x), int(head_c), gate_ptr, ldg, launches=0)
+            self.lib.call("rb_gemm_tc_per_head", H, int(head_x), int(head_c), gate_ptr, ldg, 1 if by_head else 0,
+                          launches=0)
             self.lib.call("rb_gemm_tc", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), T, _ptr(weight.w), K, H * N, N,
                           K, 0, 0, 1, tile, 1.0, self._stream())
             return
         if gate is not None:
-            self.lib.call("rb_gemm_simple_next", c_void_p(0), gate_ptr, ldg, N, launches=0)
+            self.lib.call("rb_gemm_simple_next", c_void_p(0), gate_ptr, ldg, 1 if by_head else N, 0 if by_head else 1, launches=0)
         self.lib.call("rb_gemm_simple_batched", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), _ptr(weight.w), K,
                       self.code, T, N, K, 0, 1.0, H, int(head_c), int(head_x), N * K, self._stream())
 
     def per_head_linear(self, x: torch.Tensor, weight: PerHeadWeight, gate=None) -> torch.Tensor:
         """x [T, heads * s] -> [T, heads * n_out]: the first n_in <= s values of head h times its own matrix (float32 sums).
-        ``gate`` = (float32 rows [T, ...], column): value n of head h times sigmoid(rows[:, column + h * n_out + n])."""
+        ``gate`` = (float32 rows [T, ...], column): value n of head h times sigmoid(rows[:, column + h * n_out + n]);
+        (rows, column, "head"): all of head h times sigmoid(rows[:, column + h])."""
         self._check(x, self.dtype, "per_head_linear input")
         T, H, N, K = x.shape[0], weight.heads, weight.n_out, weight.n_in
         head_x = x.shape[1] // H
@@ -1166,8 +1233,9 @@ class CudaOps:
             # a decode step: a warp per output and head instead of a few tiles
             if gate is not None:
                 self._check(gate[0], torch.float32, "per-head gate")
-                self.lib.call("rb_gemm_simple_next", c_void_p(0), c_void_p(gate[0].data_ptr() + gate[1] * 4), gate[0].stride(0), N,
-                              launches=0)
+                by_head = gate[2:] == ("head",)
+                self.lib.call("rb_gemm_simple_next", c_void_p(0), c_void_p(gate[0].data_ptr() + gate[1] * 4), gate[0].stride(0),
+                              1 if by_head else N, 0 if by_head else 1, launches=0)
             self.lib.call("rb_per_head_few_rows", _ptr(out), out.stride(0), self.code, _ptr(x), x.stride(0), head_x, _ptr(weight.w),
                           self.code, T, H, N, K, self._stream())
             return out
@@ -1186,12 +1254,16 @@ class CudaOps:
         return ExpertGateUp(w.contiguous(), inner, K, 2 * inner, 0)
 
     def route_scored(self, h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int,
-                     keep: int, scoring: str = "softmax", extra_rows: int = 0, router_tc: Optional[LinearWeight] = None):
+                     keep: int, scoring: str = "softmax", extra_rows: int = 0, router_tc: Optional[LinearWeight] = None,
+                     normalize: Optional[float] = None, weight_scale: float = 1.0):
         """``route`` with its variants: ``scoring`` "sigmoid" takes s = sigmoid(z) output by output, "softmax_chosen"
         chooses by z itself and takes the softmax over the chosen z alone; the last
         ``extra_rows`` rows of ``router`` are no outputs: their float32 sums are returned as they are ([T, extra_rows],
-        None without).  Returns (ids, weights, extra)."""
+        None without).  ``normalize`` (a small number): the chosen outputs' weights are divided by their sum + it; then
+        they are multiplied by ``weight_scale``.  Returns (ids, weights, extra)."""
         self._check(h, self.dtype, "route input")
+        if normalize is not None or weight_scale != 1.0:
+            self.lib.call("rb_route_next", 0 if normalize is None else 1, float(normalize or 0.0), float(weight_scale), launches=0)
         T, K = h.shape
         n = router.shape[0] - extra_rows
         ids = torch.empty((T, top), dtype=torch.int32, device=self.device)
@@ -1265,8 +1337,8 @@ class CudaOps:
         ``act`` = (alpha, limit, shift): gated experts, ``w_up`` an ``ExpertGateUp``, the inner rows
         g' sigmoid(alpha g') (u' + shift) as in ``gated_linear``.  ``weight_on_input``: sum_j expert(weights[t, j] * h[t])
         instead (the weighted row is rounded to the compute dtype before the expert's first product).
-        ``shared`` = (float32 rows, float32 gate logits [T, 1]): sigmoid(gate) * rows is added in the same kernel as the
-        weighted sum; a ``TanhRequest`` is granted there too."""
+        ``shared`` = (float32 rows, float32 gate logits [T, 1] or None): sigmoid(gate) * rows (None: the rows as they are) is
+        added in the same kernel as the weighted sum; a ``TanhRequest`` is granted there too."""
         T, E = h.shape
         top = ids.shape[1]
         pairs = T * top

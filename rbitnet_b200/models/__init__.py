@@ -5,3 +5,4 @@ from . import vaderax  # noqa: F401
 from . import nifarax  # noqa: F401
 from . import gozotar  # noqa: F401
 from . import busavik  # noqa: F401
+from . import bafulorn  # noqa: F401

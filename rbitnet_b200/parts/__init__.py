@@ -6,10 +6,11 @@ from .norm import RMSNorm, LayerNorm
 from .position import RotaryEncoding, NoPositionEncoding
 from .attention import Attention
 from .feed_forward import GatedDense, Dense, RoutedExperts
-from .block import PreNormBlock, StreamBlock, GatedPreNormBlock, PostNormBlock
+from .block import PreNormBlock, StreamBlock, GatedPreNormBlock, PostNormBlock, TwoNormBlock
 from .recurrent import GatedLinearRecurrence, MatrixMemory
 from .delta import GatedDeltaRule
 from .gla import GatedLinearAttention
+from .ssd import StateSpace
 from .latent import LatentAttention
 from .retention import Retention
 from .sublayer import CausalTapsFilter, SigmoidGate, GatedTokenEmbedding
@@ -23,4 +24,4 @@ __all__ = ["PartSpec", "BlockSpec", "ScheduleEntry", "ModelSpec", "Part", "Norm"
            "ParallelMixers", "ResidualConnection", "HyperConnection", "LayerNorm", "Dense", "RoutedExperts",
            "GatedDeltaRule", "GatedLinearAttention", "LatentAttention", "CausalTapsFilter", "SigmoidGate",
            "InputFilter", "ResultGate", "GatedPreNormBlock", "PostNormBlock", "Retention",
-           "GatedTokenEmbedding", "TokenInput"]
+           "GatedTokenEmbedding", "TokenInput", "StateSpace", "TwoNormBlock"]

@@ -34,6 +34,9 @@ kernel (``ops.qk_prepare``) does everything between it and the attention:
   value_mix        the values of the first layer of a step that has this option are kept for the step; every later
                    such layer caches (1 - l) v + l v_first instead of its own v, l its stored number "vmix"
   sinks            the softmax's denominator also holds exp(s_h), a stored number per head ("sink")
+  keep_first       with a window: the first so many positions of a sequence stay visible (and cached) wherever the window is
+  bias             the q, k (and v) projections and the output product have biases ("q.b", "k.b", "v.b", "o.b"), added to
+                   their float32 sums
 """
 from __future__ import annotations
 
@@ -53,7 +56,7 @@ class Attention(Mixer):
                  scale: Optional[float] = None, value_dim: Optional[int] = None,
                  qk_norm: Optional[str] = None, norm_eps: float = 1e-6, head_gate: bool = False,
                  value_gate: bool = False, conv_taps: int = 0, values: str = "own", softcap: float = 0.0,
-                 value_mix: bool = False, sinks: bool = False):
+                 value_mix: bool = False, sinks: bool = False, keep_first: int = 0, bias: bool = False):
         if n_heads % n_kv_heads:
             raise ValueError(f"attention: {n_heads} heads are not a multiple of {n_kv_heads} kv heads")
         self.width, self.n_heads, self.n_kv_heads, self.head_dim = width, n_heads, n_kv_heads, head_dim
@@ -68,16 +71,18 @@ class Attention(Mixer):
             raise ValueError(f"attention: values {values!r} is not built ('own', 'keys')")
         self.conv_taps, self.values_are_keys = int(conv_taps or 0), values == "keys"
         self.softcap, self.value_mix, self.sinks = float(softcap or 0.0), bool(value_mix), bool(sinks)
+        self.keep_first, self.has_bias = (int(keep_first or 0) if window else 0), bool(bias)
         if self.values_are_keys and self.value_dim != head_dim:
             raise ValueError("attention: values that are the keys have the keys' size")
         if self.values_are_keys and value_mix:
             raise ValueError("attention: values that are the keys are not mixed with another layer's")
         #: the options of the module's third paragraph: float32 projections and one kernel before the attention
         self.prepared = bool(self.conv_taps >= 1 or self.values_are_keys or self.softcap or self.value_mix or self.sinks
-                             or qk_norm == "head_weight")
+                             or self.keep_first or self.has_bias or qk_norm == "head_weight")
         if self.prepared and (qk_norm == "head" or value_gate):
             raise ValueError("attention: a weightless norm per head after the rotation and a gate per value do not go "
-                             "with the convolution, the shared values, the soft cap, the mixed values or the sinks")
+                             "with the convolution, the shared values, the soft cap, the mixed values, the sinks, the kept first "
+                             "positions or the biases")
         if head_gate and value_gate:
             raise ValueError("attention: a gate per head or a gate per value, not both")
         self.qk_norm, self.norm_eps, self.head_gate = qk_norm, float(norm_eps), bool(head_gate)
@@ -108,6 +113,8 @@ class Attention(Mixer):
         if self.conv_taps >= 1:
             shapes["q.conv"] = ((H * D, self.conv_taps), "taps")
             shapes["k.conv"] = ((K * D, self.conv_taps), "taps")
+        if self.has_bias:
+            shapes.update({f"{k}.b": (shapes[k][0][:1], "matrix") for k in ("q", "k", "v", "o") if k in shapes})
         if self.value_mix:
             shapes["vmix"] = ((), "matrix")
         if self.sinks:
@@ -119,7 +126,7 @@ class Attention(Mixer):
         return shapes
 
     def cache_need(self):
-        return CacheNeed(self.n_kv_heads, self.cache_width, self.window)
+        return CacheNeed(self.n_kv_heads, self.cache_width, self.window, keep_first=self.keep_first)
 
     def state_need(self):
         if self.conv_taps > 1:
@@ -142,6 +149,12 @@ class Attention(Mixer):
                 self.conv_w = torch.cat([weights["q.conv"], weights["k.conv"]], dim=0).to(**f32).contiguous()
             if self.value_mix:
                 self.mix_weight = float(weights["vmix"].to(torch.float32).reshape(-1)[0])
+            if self.has_bias:
+                rows = [weights[f"{k}.b"] for k in ("q", "k", "v") if f"{k}.b" in weights]
+                if self.head_gate:
+                    rows.append(torch.zeros(self.n_heads, device=weights["g"].device))
+                self.qkv_bias = torch.cat([r.to(**f32) for r in rows]).contiguous()
+                self.o_bias = weights["o.b"].to(**f32).contiguous()
             if self.sinks:
                 self.sink_w = weights["sink"].to(**f32).contiguous()
             self.cache_width = ops.cache_head_width(self.head_dim, self.value_dim)
@@ -164,7 +177,7 @@ class Attention(Mixer):
     #: ``h`` may be rows with their norm pending, and ``then_norm`` is handed to the last product
     folds_norms = True
 
-    conv_w = sink_w = None
+    conv_w = sink_w = qkv_bias = o_bias = None
     mix_weight = 0.0
 
     def _forward_prepared(self, ctx, h, entry, accumulate_into, scale_result):
@@ -174,7 +187,8 @@ class Attention(Mixer):
             raise ValueError("attention behind a convolution, with shared or mixed values, reads only its own cache")
         H, Kh, D, Dv = self.n_heads, self.n_kv_heads, self.head_dim, self.value_dim
         table = self.position.table() if hasattr(self.position, "table") else None
-        proj = ops.linear(ops.normed(h) if hasattr(h, "scaled") else h, self.w_qkv, out_dtype=torch.float32)
+        kw = {"bias": self.qkv_bias} if self.has_bias else {}
+        proj = ops.linear(ops.normed(h) if hasattr(h, "scaled") else h, self.w_qkv, out_dtype=torch.float32, **kw)
         mix = None
         if self.value_mix:
             v_at = (H + Kh) * D
@@ -190,11 +204,15 @@ class Attention(Mixer):
         q, gates = ops.qk_prepare(proj, ctx.meta, view, H, D, Dv, table, self.qk_norm, self.q_norm_w, self.k_norm_w,
                                   self.norm_eps, conv=self.conv_w, tail=tail, values_are_keys=self.values_are_keys,
                                   v_mix=mix, gate_heads=self.head_gate)
-        a = ops.attention(q, ctx.meta, view, H, self.scale, self.window, sinks=self.sink_w, softcap=self.softcap)
+        kw = {"keep_first": self.keep_first} if self.keep_first else {}
+        a = ops.attention(q, ctx.meta, view, H, self.scale, self.window, sinks=self.sink_w, softcap=self.softcap, **kw)
         a = ops.head_gate(a, gates, 0 if self.head_gate else None, H, Dv, view.head_dim)
+        kw = {}
+        if self.has_bias:
+            kw["bias"] = self.o_bias if scale_result == 1.0 else self.o_bias * scale_result
         if accumulate_into is None:
-            return ops.linear(a, self.w_o, out_dtype=torch.float32, scale=scale_result)
-        return ops.linear(a, self.w_o, accumulate_into=accumulate_into, scale=scale_result)
+            return ops.linear(a, self.w_o, out_dtype=torch.float32, scale=scale_result, **kw)
+        return ops.linear(a, self.w_o, accumulate_into=accumulate_into, scale=scale_result, **kw)
 
     def _forward_extended(self, ctx, h, entry, accumulate_into):
         ops = ctx.ops

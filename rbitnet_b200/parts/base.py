@@ -38,11 +38,14 @@ class CacheNeed:
     By default two tensors are stored per position, keys and values, each of ``n_kv_heads``
     heads of ``head_dim`` values.  ``streams`` names other contents: a tuple of (heads, width)
     pairs, one per stored tensor, for instance ``((1, 96),)`` for a mixer that keeps one vector
-    per position, or keys and values of different widths."""
+    per position, or keys and values of different widths.
+
+    ``keep_first``: with a window, the first so many positions stay visible (and stored) wherever the window is."""
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     streams: Optional[Tuple[Tuple[int, int], ...]] = None
+    keep_first: int = 0
 
     def stream_shapes(self) -> Tuple[Tuple[int, int], ...]:
         if self.streams is not None:

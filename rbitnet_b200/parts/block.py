@@ -271,7 +271,57 @@ class PostNormBlock:
         return h if want_rows else None
 
 
+class TwoNormBlock:
+    """Sublayers with a norm before and a norm after them:
+
+        x <- x + norm_b(sublayer(norm(x)))
+
+    for the mixer and, if the layer has one, the feed-forward.  Parts: "mixer" with "mixer_norm" and "mixer_result_norm";
+    optionally "feed_forward" with "ffn_norm" and "ffn_result_norm".  What lies between two sublayers (a result's norm, its
+    addition, the norm of what the next sublayer reads) is one operation of the result's norm (``add_and_norm``); the last
+    one of a block makes the rows of the block after it, whose first norm is handed in like a pending one
+    (``chains_norms``), or of the model's final norm where every row is wanted."""
+
+    chains_norms = True
+    #: what ``run`` takes as ``pending`` and returns are finished rows of a norm
+    takes_finished_rows = True
+
+    def __init__(self, spec):
+        self.spec = spec
+        self._parts = p = build_parts(spec)
+        missing = [n for n in ("mixer", "mixer_norm", "mixer_result_norm") if n not in p]
+        if missing:
+            raise ValueError(f"a two_norm block needs the parts {missing}")
+        ffn = [n for n in ("feed_forward", "ffn_norm", "ffn_result_norm") if n in p]
+        if len(ffn) not in (0, 3):
+            raise ValueError("a two_norm block has a feed-forward with its two norms, or none of them")
+        for n in ("mixer_result_norm", "ffn_result_norm"):
+            if n in p and not hasattr(p[n], "add_and_norm"):
+                raise ValueError("a two_norm block needs result norms that can be added to the residual stream (add_and_norm)")
+
+    def parts(self):
+        return self._parts
+
+    def first_norm(self):
+        return self._parts["mixer_norm"]
+
+    def run(self, ctx, x, entry: int, pending=None, next_norm=None):
+        p = self._parts
+        h = PreNormBlock._rows_for(ctx, p["mixer"], p["mixer_norm"], x, pending)
+        y = p["mixer"].forward(ctx, h, entry, accumulate_into=None)
+        last = p["mixer_result_norm"]
+        if "feed_forward" in p:
+            h = last.add_and_norm(ctx, x, y, p["ffn_norm"])
+            y = p["feed_forward"].forward(ctx, h, accumulate_into=None)
+            last = p["ffn_result_norm"]
+        if next_norm is None:
+            last.add_to(ctx, x, y)
+            return None
+        return last.add_and_norm(ctx, x, y, next_norm)
+
+
 register_part("block", "pre_norm", PreNormBlock)
+register_part("block", "two_norm", TwoNormBlock)
 register_part("block", "post_norm", PostNormBlock)
 register_part("block", "pre_norm_gated", GatedPreNormBlock)
 register_part("block", "multi_stream", StreamBlock)

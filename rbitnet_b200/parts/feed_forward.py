@@ -4,7 +4,7 @@ the product are float32 before any rounding to the compute dtype.
 
 ``activation`` "swish_limited": with g' = min(gate h, limit) and u' = clamp(up h, -limit, limit),
 the inner rows are g' * sigmoid(alpha g') * (u' + shift); alpha = 1.702 and shift = 1 unless given.
-``activation`` "gelu_tanh": gelu(gate h) * (up h), gelu in its tanh form.  ``bias``: all three projections have biases,
+``activation`` "gelu_tanh": gelu(gate h) * (up h), gelu in its tanh form; "relu": max(gate h, 0) * (up h).  ``bias``: all three projections have biases,
 added to the float32 sums.
 
 ``Dense``: down(relu2(up h)), no gate.  ``RoutedExperts``: a router chooses a few of many small feed-forwards
@@ -20,12 +20,12 @@ from .registry import register_part
 class GatedDense(FeedForward):
     def __init__(self, width: int, inner: int, activation: str = "silu", limit: float = 0.0,
                  alpha: float = 1.702, shift: float = 1.0, bias: bool = False):
-        if activation not in ("silu", "swish_limited", "gelu_tanh"):
+        if activation not in ("silu", "swish_limited", "gelu_tanh", "relu"):
             raise ValueError(f"gated feed-forward: activation {activation!r} is not built "
-                             "(only 'silu', 'swish_limited' and 'gelu_tanh')")
+                             "(only 'silu', 'swish_limited', 'gelu_tanh' and 'relu')")
         self.width, self.inner, self.activation = int(width), int(inner), activation
-        #: (alpha, limit, shift) of the limited activation, or "gelu_tanh"; None: SiLU(gate) * up
-        self.act = {"silu": None, "gelu_tanh": "gelu_tanh"}.get(activation, (float(alpha), float(limit), float(shift)))
+        #: (alpha, limit, shift) of the limited activation, or "gelu_tanh" or "relu"; None: SiLU(gate) * up
+        self.act = {"silu": None, "gelu_tanh": "gelu_tanh", "relu": "relu"}.get(activation, (float(alpha), float(limit), float(shift)))
         if activation == "swish_limited" and not self.act[1] > 0:
             raise ValueError("gated feed-forward: 'swish_limited' needs a positive limit")
         self.has_bias = bool(bias)
@@ -96,7 +96,8 @@ class RoutedExperts(FeedForward):
     output), among the outputs of the ``keep`` best of ``groups`` equal groups of neighbouring outputs (a group's score
     is its largest choice score; groups 0 or 1: no groups); the chosen outputs' weights are their s, not
     renormalised.  "softmax_chosen": the choice is made by z + correction instead, and the chosen outputs' weights are
-    the softmax over their z alone.  ``weight_on`` "output": the result is the weighted sum of the chosen experts' results;
+    the softmax over their z alone.  ``normalize`` (a small number): the chosen outputs' weights are divided by their sum
+    + it; ``weight_scale`` multiplies them after that.  ``weight_on`` "output": the result is the weighted sum of the chosen experts' results;
     "input": every chosen expert runs on its weight times the input row, and the results are added up as they are.
 
     ``activation`` "relu2": an expert is down(relu2(up h)) ("e<i>.up" [inner, width], "e<i>.down" [width, inner]).
@@ -106,13 +107,14 @@ class RoutedExperts(FeedForward):
     ``shared`` (a dict with "inner" and, for the limited activation, "limit" and optionally "alpha",
     "shift"): one more gated expert of the same form that every token uses ("shared.gate", "shared.up", "shared.down"), its result multiplied by sigmoid(w_sg . h), one
     number per token ("shared.sg" [1, width]), and added.  The gate's sum is made beside the router's, in float32.
+    With ``"gate": False`` in the dict there is no such gate and the result is added as it is.
 
     Weights: "router" [n_experts + n_identity, width], "correction" (``correction=False``: none), the experts'."""
 
     def __init__(self, width: int, inner: int, n_experts: int, top: int, n_identity: int = 0, groups: int = 0,
                  keep: int = 0, correction: bool = True, activation: str = "relu2", scoring: str = "softmax",
                  weight_on: str = "output", limit: float = 0.0, alpha: float = 1.702, shift: float = 1.0,
-                 shared: dict = None):
+                 shared: dict = None, normalize: float = None, weight_scale: float = 1.0):
         if activation not in ("relu2", "swish_limited", "silu"):
             raise ValueError(f"routed experts: activation {activation!r} is not built (only 'relu2', 'swish_limited' and 'silu')")
         if scoring not in ("softmax", "sigmoid", "softmax_chosen"):
@@ -128,8 +130,10 @@ class RoutedExperts(FeedForward):
         if activation == "swish_limited" and not self.act[1] > 0:
             raise ValueError("routed experts: 'swish_limited' needs a positive limit")
         self.shared = None
+        self.normalize = None if normalize is None else float(normalize)
+        self.weight_scale = float(weight_scale)
         if shared:
-            self.shared = {"inner": int(shared["inner"]),
+            self.shared = {"inner": int(shared["inner"]), "gate": bool(shared.get("gate", True)),
                            "act": (None if activation == "silu" else
                                    (float(shared.get("alpha", 1.702)), float(shared["limit"]), float(shared.get("shift", 1.0))))}
             if self.shared["inner"] < 1 or not (activation == "silu" or self.shared["act"][1] > 0):
@@ -151,7 +155,8 @@ class RoutedExperts(FeedForward):
     @property
     def plain(self) -> bool:
         """Softmax scores that weigh the results of ungated experts, and no shared expert."""
-        return self.act is None and self.scoring == "softmax" and self.weight_on == "output" and self.shared is None
+        return self.act is None and self.scoring == "softmax" and self.weight_on == "output" and self.shared is None \
+            and self.normalize is None and self.weight_scale == 1.0
 
     def weight_shapes(self):
         n = self.n_experts + self.n_identity
@@ -166,12 +171,14 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             f = self.shared["inner"]
             shapes.update({"shared.gate": ((f, self.width), "matrix"), "shared.up": ((f, self.width), "matrix"),
-                           "shared.down": ((self.width, f), "matrix"), "shared.sg": ((1, self.width), "matrix")})
+                           "shared.down": ((self.width, f), "matrix")})
+            if self.shared["gate"]:
+                shapes["shared.sg"] = ((1, self.width), "matrix")
         return shapes
 
     def bind(self, weights, ops):
         # the router's product is float32 whatever the compute dtype; a shared expert's gate is one more row of it
-        rows = [weights["router"]] + ([weights["shared.sg"]] if self.shared is not None else [])
+        rows = [weights["router"]] + ([weights["shared.sg"]] if self.shared is not None and self.shared["gate"] else [])
         self.router = torch.cat([r.to(device=ops.device, dtype=torch.float32) for r in rows], dim=0).contiguous()
         self.correction = (weights["correction"].to(device=ops.device, dtype=torch.float32).contiguous()
                            if self.has_correction else None)
@@ -202,9 +209,12 @@ class RoutedExperts(FeedForward):
                 ids, weights = ops.route(h, self.router, self.correction, self.top, self.groups, self.keep)
             return ops.routed_experts(h, ids, weights, self.w_up, self.w_down, self.n_experts, self.inner,
                                       accumulate_into=accumulate_into)
-        extra = 1 if self.shared is not None else 0
+        extra = 1 if self.shared is not None and self.shared["gate"] else 0
+        kw = {}
+        if self.normalize is not None or self.weight_scale != 1.0:
+            kw = {"normalize": self.normalize, "weight_scale": self.weight_scale}
         ids, weights, gate = ops.route_scored(h, self.router, self.correction, self.top, self.groups, self.keep,
-                                              scoring=self.scoring, extra_rows=extra, router_tc=self.router_tc)
+                                              scoring=self.scoring, extra_rows=extra, router_tc=self.router_tc, **kw)
         kw = {}
         if self.shared is not None:
             t = ops.gated_linear(h, self.shared_gate_up, act=self.shared["act"])

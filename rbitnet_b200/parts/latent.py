@@ -29,7 +29,11 @@ Options, each off by default:
                 same input rows; its float32 sums come out of the same product as the latents, and the sigmoid is applied
                 where the heads' results leave their matrices W_uv
 
-All options go together.  With queries through a latent AND a turned part, the turned part of the queries exists only
+  window        a position sees itself and the window - 1 positions before it; the pages behind it are given back
+  head_gate     head h's result is multiplied by sigmoid(W_g h)_h, one number per head ("g", a row per head), made and applied
+                as the gate per value is
+
+All options go together (one kind of gate at a time).  With queries through a latent AND a turned part, the turned part of the queries exists only
 after W_uq: the step that takes the query heads into the latent's space turns it (``ops.latent_queries``).
 """
 from __future__ import annotations
@@ -46,11 +50,14 @@ from .spec import PartSpec
 class LatentAttention(Mixer):
     def __init__(self, width: int, n_heads: int, head_dim: int, value_dim: int, q_rank: int, kv_rank: int,
                  scale: float, norm_eps: float, rot_dim: int = 0, position: dict = None, sinks: bool = False,
-                 value_gate: bool = False):
+                 value_gate: bool = False, window: int = None, head_gate: bool = False):
         self.width, self.n_heads, self.head_dim, self.value_dim = int(width), int(n_heads), int(head_dim), int(value_dim)
         self.q_rank, self.kv_rank = int(q_rank or 0), int(kv_rank)
         self.scale, self.norm_eps = float(scale), float(norm_eps)
         self.rot_dim, self.sinks, self.value_gate = int(rot_dim or 0), bool(sinks), bool(value_gate)
+        self.window, self.head_gate = (int(window) if window else None), bool(head_gate)
+        if self.head_gate and self.value_gate:
+            raise ValueError("latent attention: a gate per head or a gate per value, not both")
         if min(self.n_heads, self.head_dim, self.value_dim, self.kv_rank) < 1 or self.q_rank < 0 or self.rot_dim < 0:
             raise ValueError("latent attention: heads, sizes and ranks are at least 1")
         self.position = None
@@ -80,15 +87,17 @@ class LatentAttention(Mixer):
             shapes["sink"] = ((H,), "matrix")
         if self.value_gate:
             shapes["g"] = ((H * Dv, E), "matrix")
+        if self.head_gate:
+            shapes["g"] = ((H, E), "matrix")
         return shapes
 
     def cache_need(self):
-        return CacheNeed(1, self.cache_width, None, streams=((1, self.cache_width),))
+        return CacheNeed(1, self.cache_width, self.window, streams=((1, self.cache_width),))
 
     def bind(self, weights, ops):
         H, D, Dv, R, Rr = self.n_heads, self.head_dim, self.value_dim, self.kv_rank, self.rot_dim
         self.cache_width = Rc = ops.cache_head_width(R + Rr, R + Rr)
-        gate = [weights["g"]] if self.value_gate else []
+        gate = [weights["g"]] if self.value_gate or self.head_gate else []
         if self.q_rank:
             self.w_down = ops.prepare_linear([weights["dq"], weights["dkv"]] + gate)
             self.w_uq = ops.prepare_linear([weights["uq"]])
@@ -138,11 +147,11 @@ class LatentAttention(Mixer):
             ql = ops.latent_queries(q, self.w_uk_t, self.rot_dim, view.head_dim, table, ctx.meta)
         both = dataclasses.replace(view, v=view.k)                                  # keys and values: the latents
         if self.sinks:
-            a = ops.attention(ql.view(ql.shape[0], H, view.head_dim), ctx.meta, both, H, self.scale, None,
+            a = ops.attention(ql.view(ql.shape[0], H, view.head_dim), ctx.meta, both, H, self.scale, self.window,
                               sinks=self.sink_w)
         else:
-            a = ops.attention(ql.view(ql.shape[0], H, view.head_dim), ctx.meta, both, H, self.scale, None)
-        gate = (down, self.gate_at) if self.value_gate else None
+            a = ops.attention(ql.view(ql.shape[0], H, view.head_dim), ctx.meta, both, H, self.scale, self.window)
+        gate = (down, self.gate_at) if self.value_gate else (down, self.gate_at, "head") if self.head_gate else None
         o = ops.per_head_linear(a, self.w_uv, gate=gate)                            # [T, H * Dv]
         if accumulate_into is None:
             return ops.linear(o, self.w_o, out_dtype=torch.float32)

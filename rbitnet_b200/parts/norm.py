@@ -3,7 +3,8 @@
 ``groups`` > 1: the row is cut into that many equal consecutive parts, each divided by its own root mean
 square; the weight still spans the whole row.  ``one_plus``: the stored weight lies around zero and multiplies as
 1 + w.  ``layer_scale``: a second stored vector ("scale") multiplies the normed row value by value; the two are kept
-as one float32 vector.  ``add_to`` is the norm on a sublayer's RESULT: x += norm(y).
+as one float32 vector.  ``multiplier``: one number that multiplies the normed row, kept in that vector too.  ``add_to`` is
+the norm on a sublayer's RESULT: x += norm(y); ``add_and_norm`` also leaves the rows of the norm that reads the new x.
 LayerNorm: the mean taken off first, and a bias added."""
 from __future__ import annotations
 
@@ -14,7 +15,9 @@ from .registry import register_part
 
 
 class RMSNorm(Norm):
-    def __init__(self, width: int, eps: float, groups: int = 1, one_plus: bool = False, layer_scale: bool = False):
+    def __init__(self, width: int, eps: float, groups: int = 1, one_plus: bool = False, layer_scale: bool = False,
+                 multiplier: float = 1.0):
+        self.multiplier = float(multiplier)
         self.width, self.eps, self.groups = int(width), float(eps), int(groups)
         self.one_plus, self.layer_scale = bool(one_plus), bool(layer_scale)
         if self.groups < 1 or self.width % self.groups:
@@ -34,6 +37,8 @@ class RMSNorm(Norm):
             w = 1.0 + w
         if self.layer_scale:
             w = w * weights["scale"].to(torch.float32)
+        if self.multiplier != 1.0:
+            w = w * self.multiplier
         self.weight = w.contiguous()
 
     def add_to(self, ctx, x, y, want_rounded: bool = False):
@@ -42,6 +47,20 @@ class RMSNorm(Norm):
         if self.groups != 1:
             raise ValueError("rmsnorm: a norm in groups on a sublayer's result is not built")
         return ctx.ops.norm_add(x, y, self.weight, self.eps, want_rounded=want_rounded)
+
+    def add_and_norm(self, ctx, x, y, after):
+        """``add_to``, and the rows of the norm ``after`` on the new x in the compute dtype, in one operation."""
+        if self.groups != 1 or not isinstance(after, RMSNorm) or after.groups != 1:
+            self.add_to(ctx, x, y)
+            return after.forward(ctx, x)
+        return ctx.ops.norm_add_norm(x, y, self.weight, self.eps, after.weight, after.eps)[1]
+
+    def start_with(self, ctx, y, after):
+        """(norm(y) as float32 rows, the rows of the norm ``after`` on them in the compute dtype)."""
+        if self.groups != 1 or not isinstance(after, RMSNorm) or after.groups != 1:
+            x = self.forward(ctx, y, out_dtype=torch.float32)
+            return x, after.forward(ctx, x)
+        return ctx.ops.norm_add_norm(None, y, self.weight, self.eps, after.weight, after.eps)
 
     def forward(self, ctx, x, out_dtype=None):
         kw = {} if out_dtype is None else {"out_dtype": out_dtype}

@@ -29,7 +29,9 @@ class _GU:
 
 
 def _gated(act, g, u):
-    """The gated activation the package asks for: (alpha, limit, shift), "gelu_tanh", or None (SiLU)."""
+    """The gated activation the package asks for: (alpha, limit, shift), "gelu_tanh", "relu", or None (SiLU)."""
+    if act == "relu":
+        return torch.clamp(g, min=0.0) * u
     if act == "gelu_tanh":
         return 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3))) * u
     alpha, limit, shift = act if act is not None else (1.0, 0.0, 0.0)
@@ -272,6 +274,31 @@ class TorchOps:
         gate = x[:, at["g"]:at["g"] + H * Dv]
         return (o.reshape(T, H * Dv) * (gate / (1.0 + torch.exp(-gate)))).to(self.dtype)
 
+    def state_space(self, proj, p, state, meta):
+        H, P, N, G, K, C = p.n_heads, p.value_dim, p.state_dim, p.n_groups, p.taps, p.channels
+        at, inner = p.offsets(), H * P
+        x = proj.float()
+        T = x.shape[0]
+        out = torch.zeros(T, H, P)
+        share = torch.arange(H) // (H // G)
+        for first, n, slot in self._runs(meta):
+            xin = x[first:first + n, at["x"]:at["x"] + C]
+            old = state["tail"][slot][1:] if K > 1 else torch.zeros(0, C)      # this stand-in keeps the last K-1 inputs in rows 1..
+            hist = torch.cat([old, xin], dim=0)
+            S = state["S"][slot].clone()                                        # [H, N, P]
+            for t in range(n):
+                u = (hist[t:t + K] * p.conv_w.T).sum(0) + p.conv_b
+                u = u / (1.0 + torch.exp(-u))
+                v, B, Cc = u[:inner].view(H, P), u[inner:inner + G * N].view(G, N)[share], u[inner + G * N:].view(G, N)[share]
+                d = torch.nn.functional.softplus(x[first + t, at["dt"]:at["dt"] + H] + p.dt_bias)
+                S = S * torch.exp(-torch.exp(p.a_log) * d)[:, None, None] + B[:, :, None] * (d[:, None] * v)[:, None, :]
+                out[first + t] = torch.einsum("hnp,hn->hp", S, Cc) + p.d_skip[:, None] * v
+            state["S"][slot] = S
+            if K > 1:
+                state["tail"][slot][1:] = hist[n:n + K - 1]
+        z = x[:, at["z"]:at["z"] + inner]
+        return out.reshape(T, inner) * (z / (1.0 + torch.exp(-z)))
+
     # ---- around a sublayer
     def rmsnorm_grouped(self, x, w, groups, eps, out_dtype=None):
         T, E = x.shape
@@ -360,7 +387,10 @@ class TorchOps:
         y = torch.einsum("thk,hnk->thn", x.to(torch.float32).view(x.shape[0], H, -1)[..., :K], w.to(torch.float32))
         y = y.reshape(x.shape[0], H * N)
         if gate is not None:
-            y = y * torch.sigmoid(gate[0][:, gate[1]:gate[1] + H * N])
+            if gate[2:] == ("head",):
+                y = y * torch.sigmoid(gate[0][:, gate[1]:gate[1] + H]).repeat_interleave(N, dim=1)
+            else:
+                y = y * torch.sigmoid(gate[0][:, gate[1]:gate[1] + H * N])
         return y.to(self.dtype)
 
     # ---- routed experts
@@ -368,7 +398,8 @@ class TorchOps:
         w = torch.cat([torch.cat([self.to_compute(g), self.to_compute(u)], dim=0) for g, u in zip(gates, ups)], dim=0)
         return _W(w, w.shape[0], w.shape[1])
 
-    def route_scored(self, h, router, correction, top, groups, keep, scoring="softmax", extra_rows=0, router_tc=None):
+    def route_scored(self, h, router, correction, top, groups, keep, scoring="softmax", extra_rows=0, router_tc=None,
+                     normalize=None, weight_scale=1.0):
         z = h.to(torch.float32) @ router.T
         n = router.shape[0] - extra_rows
         extra = z[:, n:].clone() if extra_rows else None
@@ -384,6 +415,9 @@ class TorchOps:
         weights = s.gather(1, ids)
         if scoring == "softmax_chosen":
             weights = torch.softmax(weights, dim=-1)
+        if normalize is not None:
+            weights = weights / (weights.sum(-1, keepdim=True) + normalize)
+        weights = weights * weight_scale
         return ids.to(torch.int32), weights, extra
 
     def route(self, h, router, correction, top, groups, keep):
@@ -417,7 +451,7 @@ class TorchOps:
                     mid = (torch.clamp(up @ xin, min=0.0) ** 2).to(self.dtype).to(torch.float32)
                 out[t] += (down @ mid) if weight_on_input else w * (down @ mid)
         if shared is not None:
-            out += torch.sigmoid(shared[1][:, :1]) * shared[0]
+            out += shared[0] if shared[1] is None else torch.sigmoid(shared[1][:, :1]) * shared[0]
         if accumulate_into is not None:
             accumulate_into += out
             return accumulate_into
@@ -460,14 +494,14 @@ class TorchOps:
                 view.v[page, :, p % view.page_size, :] = v[t].to(view.v.dtype)
         return q.to(self.dtype)
 
-    def attention(self, q, meta, view, n_heads, scale, window, sinks=None, softcap=0.0):
+    def attention(self, q, meta, view, n_heads, scale, window, sinks=None, softcap=0.0, keep_first=0):
         T, H, D = q.shape
         G = H // view.n_kv_heads
         out = torch.zeros(T, H * D, dtype=torch.float32)
         for t in range(T):
             p, slot = int(meta.tok_pos[t]), int(meta.tok_slot[t])
             lo = max(0, p - window + 1) if window else 0
-            idx = torch.arange(lo, p + 1)
+            idx = torch.cat([torch.arange(0, min(keep_first, lo)), torch.arange(lo, p + 1)])
             pages = view.page_table[slot, idx // view.page_size].long()
             ks = view.k[pages, :, idx % view.page_size, :].to(torch.float32)   # [n, Kh, D]
             vs = view.v[pages, :, idx % view.page_size, :].to(torch.float32)
@@ -490,6 +524,13 @@ class TorchOps:
         y = y.float()
         x += y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * w
         return x.to(self.dtype) if want_rounded else None
+
+    def norm_add_norm(self, x, y, w, eps, next_w, next_eps):
+        y = y.float()
+        if x is None:
+            x = torch.zeros_like(y)
+        x += y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * w
+        return x, self.rmsnorm(x, next_w, next_eps)
 
     def token_gate(self, a, table, ids):
         a = a.float()
