@@ -593,6 +593,25 @@ def _busavik_shape(width, heads, dim, rot, q_rank, kv_rank, experts, top, expert
     return cfg
 
 
+def _bafulorn_shape(width, heads, kv, dim, lat_heads, lat_dim, kv_rank, ssm_heads, ssm_vdim, ssm_state, ssm_groups, window, keep,
+                    ff, experts, top, expert_ff, shared_ff, layers, vocab=32000):
+    """Layer sizes in the manner of a real model: of every three layers the first is a state-space layer (its inner width twice
+    the model's), the second attention through latents, the third grouped attention whose values are its keys, both
+    windowed; every other layer's feed-forward is dense, the others route `top` of `experts` experts beside a shared one."""
+    ssm = {"type": "mamba2", "mixer": {"heads": ssm_heads, "vdim": ssm_vdim, "state": ssm_state, "groups": ssm_groups, "conv": 4,
+                                       "norm_groups": ssm_groups}}
+    lat = {"type": "latent_attention", "mixer": {"heads": lat_heads, "dim": lat_dim, "vdim": lat_dim, "kv_rank": kv_rank,
+                                                 "scale": lat_dim ** -0.5, "mask": {"size": window}}}
+    att = {"type": "attention", "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window, "keep_first": keep},
+        "rot": {"base": 500000.0, "dims": dim, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "scale": 2.5},
+           "shared": {"ff": shared_ff}}
+    return {"architecture": "Bafulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "max_positions": 8192, "layers": [dict((ssm, lat, att)[i % 3], mlp=moe if i % 2 else {"kind": "dense", "ff": ff})
+                                              for i in range(layers)]}
+
+
 DESIGN_SIZES = {
     # name: (the design's configuration, the configuration of equal width, layer runs and feed-forward size beside it)
     "w2048": (_safuvik_shape(2048, 16, 4, 128, 64, 1024, 16, 8, 128, 256, 5632, 6), _llama_like(2048, 16, 4, 128, 5632, 6)),
@@ -617,6 +636,12 @@ DESIGN_SIZES = {
                       _nifarax_shape(2048, 8, 128, 256, 16, 128, 768, 128, 32, 4, 1408, 1408, 6)),
     "busavik_w4096": (_busavik_shape(4096, 32, 128, 64, 1536, 192, 64, 8, 1792, 1792, 3, dense_every=3, ff=14336),
                       _nifarax_shape(4096, 16, 128, 256, 32, 128, 1536, 256, 64, 8, 1792, 1792, 3)),
+    # Bafulorn beside Gozotar (attention through latents, grouped attention whose values are keys, a matrix memory with
+    # decays; results under norms): 6 layers beside 6, 3 beside 3; cached latents as wide as Gozotar's cached rows
+    "bafulorn_w2048": (_bafulorn_shape(2048, 16, 4, 128, 16, 128, 128, 64, 64, 128, 8, 1024, 64, 5632, 32, 4, 1408, 1408, 6),
+                       _gozotar_shape(2048, 16, 4, 128, 128, 16, 128, 32, 96, 8, 128, 256, 5632, 6)),
+    "bafulorn_w4096": (_bafulorn_shape(4096, 32, 8, 128, 32, 128, 256, 128, 64, 128, 8, 1024, 64, 14336, 64, 8, 1792, 1792, 3),
+                       _gozotar_shape(4096, 32, 8, 128, 128, 32, 128, 64, 192, 16, 128, 256, 14336, 3)),
 }
 
 
@@ -628,7 +653,7 @@ class DesignTimer(KernelTimer):
                              "gated_recurrence", "matrix_memory", "layernorm", "add_rows", "gated_delta", "route", "routed_experts",
                              "rmsnorm_grouped", "input_filter", "gated_add", "softcap", "gated_linear_attention",
                              "latent_norm_append", "per_head_linear", "route_scored", "qk_prepare", "latent_rotate_append",
-                             "retention", "norm_add", "round_rows", "token_gate", "embed_pairs", "tanh_norm", "latent_queries")
+                             "retention", "norm_add", "norm_add_norm", "state_space", "round_rows", "token_gate", "embed_pairs", "tanh_norm", "latent_queries")
 
     @staticmethod
     def _describe(name, a, kw, sync=True):
@@ -686,6 +711,15 @@ class DesignTimer(KernelTimer):
                     el(proj) + T * p.n_heads * p.value_dim * 2, 0.0)
         if name == "norm_add":
             return f"normed result added to the residual stream [{a[0].shape[0]} rows]", 3 * el(a[0]) + a[0].numel() * 2, 0.0
+        if name == "norm_add_norm":
+            y, fresh = a[1], a[0] is None
+            return (f"{'normed embedding' if fresh else 'normed result added to the residual stream'}, next norm [{y.shape[0]} rows]",
+                    (2 if fresh else 3) * el(y) + y.numel() * 2, 0.0)
+        if name == "state_space":
+            proj, p = a[0], a[1]
+            T, inner = proj.shape[0], p.n_heads * p.value_dim
+            return (f"state space: convolution, recurrence, gate [{T} rows, {p.n_heads} heads of {p.state_dim}x{p.value_dim}]",
+                    el(proj) + T * inner * 4, 0.0)
         if name == "round_rows":
             return f"residual rows rounded [{a[0].shape[0]} rows]", el(a[0]) + a[0].numel() * 2, 0.0
         if name == "token_gate":
@@ -832,7 +866,7 @@ def main():
     ap.add_argument("--workload", default=None, choices=sorted(WORKLOADS),
                     help="run one of the other generation workloads end to end instead (one short line)")
     ap.add_argument("--design", default=None, choices=sorted(DESIGN_SIZES),
-                    help="instead of the headline: prefill and decode of another design (Safuvik; vaderax_*: Vaderax; nifarax_*; gozotar_*: Gozotar beside Nifarax; busavik_*: Busavik beside Nifarax) beside the Llama decoder of "
+                    help="instead of the headline: prefill and decode of another design (Safuvik; vaderax_*: Vaderax; nifarax_*; gozotar_*: Gozotar beside Nifarax; busavik_*: Busavik beside Nifarax; bafulorn_*: Bafulorn beside Gozotar) beside the Llama decoder of "
                          "equal size at these layer sizes, nifarax_*: Nifarax beside Vaderax (uses --batch, --context, --prefill-tokens, "
                          "--steps)")
     args = ap.parse_args()

@@ -52,7 +52,16 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(TO* __restrict__ u, int64
     }
   };
   int last_first = -1;
-  for (int t = t0; t < t1; ++t) {
+  constexpr int AHEAD = 8;                               // rows on their way at a time
+  for (int ta = t0; ta < t1; ta += AHEAD) {
+  float in[AHEAD][V];
+#pragma unroll
+  for (int r = 0; r < AHEAD; ++r)
+    if (ta + r < t1) load(x + (int64_t)(ta + r) * ldx + x_off + c, in[r]);
+#pragma unroll
+  for (int r = 0; r < AHEAD; ++r) {
+    const int t = ta + r;
+    if (t >= t1) break;
     const int first = tok_first != nullptr ? tok_first[t] : t;
     if (first != last_first) {                           // a new run, or the block's first row: fetch the rows before
       last_first = first;
@@ -69,8 +78,9 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(TO* __restrict__ u, int64
         }
       }
     }
-    load(x + (int64_t)t * ldx + x_off + c, hist[0]);
     float y[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) hist[0][i] = in[r][i];
 #pragma unroll
     for (int i = 0; i < V; ++i) {
       float acc = b[i];
@@ -90,6 +100,7 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(TO* __restrict__ u, int64
     for (int d = K - 1; d > 0; --d)
 #pragma unroll
       for (int i = 0; i < V; ++i) hist[d][i] = hist[d - 1][i];
+  }
   }
 }
 
@@ -121,18 +132,20 @@ constexpr int STEP_NT = 256;
 constexpr int STEP_COLS = 64;
 constexpr int STEP_HELD = 8;            // state rows a thread holds at a time
 
-template <int V>
-__global__ void __launch_bounds__(STEP_NT) ssd_step_kernel(
+// KT: the convolution's taps (0: any number, from K).
+template <int V, int KT>
+__global__ void __launch_bounds__(STEP_NT, 3) ssd_step_kernel(
     float* __restrict__ out, const float* __restrict__ rows, int64_t ld, int z_off, int x_off, int dt_off,
     const float* __restrict__ taps, const float* __restrict__ conv_bias, const float* __restrict__ dt_bias,
     const float* __restrict__ A_log, const float* __restrict__ D_skip, float* __restrict__ state, float* __restrict__ tail,
-    const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, int H, int P, int N, int G, int K, int cols) {
+    const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, int H, int P, int N, int G, int K_, int cols) {
   rb_pdl_launch_dependents();
   extern __shared__ float s_step[];
   float* sx = s_step;                   // [cols] x
   float* sB = sx + STEP_COLS;           // [N]
   float* sC = sB + N;                   // [N]
   float* red = sC + N;                  // [NL][pw]
+  const int K = KT > 0 ? KT : K_;
   const int t = blockIdx.x, h = blockIdx.y, tile = blockIdx.z, p0 = tile * cols;
   const int pw = min(cols, P - p0);                          // columns of this block
   const int groups_of = H / G, grp = h / groups_of;
@@ -143,6 +156,25 @@ __global__ void __launch_bounds__(STEP_NT) ssd_step_kernel(
   const bool mine = nl < NL;
   const int slot = tok_slot[t], pos = tok_pos[t];
   const float a = expf(A_log[h]), dtb = dt_bias[h], skip = D_skip[h];
+  const int n_ch = pw + 2 * N;                               // channels this block convolves: its x, the group's B and C
+  auto channel = [&](int i) {
+    return i < pw ? h * P + p0 + i : (i < pw + N ? inner + grp * N + (i - pw) : inner + G * N + grp * N + (i - pw - N));
+  };
+  // the weights of a thread's first two channels do not depend on the kernel before this one
+  constexpr int CPT = KT > 0 ? 2 : 1, KW = KT > 0 ? KT : 1;
+  float w[CPT][KW], cb[CPT];
+  if (KT > 0) {
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      const int i = threadIdx.x + j * STEP_NT;
+      if (i < n_ch) {
+        const int c = channel(i);
+        cb[j] = conv_bias[c];
+#pragma unroll
+        for (int d = 0; d < KW; ++d) w[j][d] = taps[(int64_t)c * KW + KW - 1 - d];
+      }
+    }
+  }
   rb_pdl_wait();
   const float* row = rows + (int64_t)t * ld;
   float* S = state + ((int64_t)slot * H + h) * N * P + p0 + pc;
@@ -161,21 +193,52 @@ __global__ void __launch_bounds__(STEP_NT) ssd_step_kernel(
       }
     }
   };
-  fetch(0);                                                  // on its way while the channels are convolved
   const bool write_bc = tile == 0 && h % groups_of == 0;
-  for (int i = threadIdx.x; i < pw + 2 * N; i += STEP_NT) {
-    const bool is_x = i < pw;
-    const int c = is_x ? h * P + p0 + i : (i < pw + N ? inner + grp * N + (i - pw) : inner + G * N + grp * N + (i - pw - N));
+  auto put = [&](int i, int c, float now, float acc) {
+    if (K > 1 && (i < pw || write_bc)) tail[((int64_t)slot * K + pos % K) * C + c] = now;
+    const float y = ssd_silu(acc);
+    if (i < pw) sx[i] = y;
+    else sB[i - pw] = y;                                     // B, then C behind it
+  };
+  const float raw_dt = row[dt_off + h];
+  const float z = threadIdx.x < pw ? row[z_off + h * P + p0 + threadIdx.x] : 0.f;
+  int done = 0;
+  if (KT > 0) {
+    float in[CPT][KW];
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      const int i = threadIdx.x + j * STEP_NT;
+      if (i < n_ch) {
+        const int c = channel(i);
+        in[j][0] = row[x_off + c];
+#pragma unroll
+        for (int d = 1; d < KW; ++d) in[j][d] = d <= pos ? tail[((int64_t)slot * KW + (pos - d) % KW) * C + c] : 0.f;
+      }
+    }
+    fetch(0);                                                // the state is on its way while the channels are convolved
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      const int i = threadIdx.x + j * STEP_NT;
+      if (i < n_ch) {
+        float acc = cb[j];
+#pragma unroll
+        for (int d = 0; d < KW; ++d) acc = fmaf(w[j][d], in[j][d], acc);
+        put(i, channel(i), in[j][0], acc);
+      }
+    }
+    done = CPT * STEP_NT;
+  } else {
+    fetch(0);
+  }
+  for (int i = done + threadIdx.x; i < n_ch; i += STEP_NT) {
+    const int c = channel(i);
     const float now = row[x_off + c];
     float acc = fmaf(taps[(int64_t)c * K + K - 1], now, conv_bias[c]);
     for (int d = 1; d < K && d <= pos; ++d)
       acc = fmaf(taps[(int64_t)c * K + K - 1 - d], tail[((int64_t)slot * K + (pos - d) % K) * C + c], acc);
-    if (K > 1 && (is_x || write_bc)) tail[((int64_t)slot * K + pos % K) * C + c] = now;
-    const float y = ssd_silu(acc);
-    if (is_x) sx[i] = y;
-    else sB[i - pw] = y;                                     // B, then C behind it
+    put(i, c, now, acc);
   }
-  const float dt = ssd_softplus(row[dt_off + h] + dtb);
+  const float dt = ssd_softplus(raw_dt + dtb);
   const float decay = expf(-a * dt);
   __syncthreads();
   float y[V], xdt[V];
@@ -207,10 +270,11 @@ __global__ void __launch_bounds__(STEP_NT) ssd_step_kernel(
       if (pc + k < pw) red[nl * pw + pc + k] = y[k];
   }
   __syncthreads();
-  for (int p = threadIdx.x; p < pw; p += STEP_NT) {
+  if (threadIdx.x < pw) {
+    const int p = threadIdx.x;
     float acc = skip * sx[p];
     for (int i = 0; i < NL; ++i) acc += red[i * pw + p];
-    out[(int64_t)t * inner + h * P + p0 + p] = acc * ssd_silu(row[z_off + h * P + p0 + p]);
+    out[(int64_t)t * inner + h * P + p0 + p] = acc * ssd_silu(z);
   }
 }
 
@@ -293,6 +357,7 @@ __global__ void __launch_bounds__(SCAN_NT) ssd_scan_kernel(
 constexpr int CH = 64;                  // tokens of a chunk
 constexpr int CH_NT = 128;              // four warps of 16 rows
 constexpr int CH_P = 64;                // value columns of a block
+constexpr int SL = 64;                  // state rows that the output kernel holds at a time
 constexpr int LDX = CH_P + 8;           // row stride of tiles of columns: ldmatrix rows in different banks
 
 __device__ __forceinline__ uint32_t s_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -311,11 +376,13 @@ __device__ __forceinline__ uint32_t pack_pair(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<const uint32_t*>(&v);
 }
-// v as three bfloat16 terms; what is left of v after the first two is exact in float32
-__device__ __forceinline__ void split3(float v, float& hi, float& mid, float& lo) {
-  hi = __bfloat162float(__float2bfloat16_rn(v));
-  mid = __bfloat162float(__float2bfloat16_rn(v - hi));
-  lo = v - hi - mid;
+// Two values as three pairs of bfloat16 terms each; what is left of a value after its first two terms is exact in float32.
+__device__ __forceinline__ void split3(float a, float b, uint32_t& hi, uint32_t& mid, uint32_t& lo) {
+  hi = pack_pair(a, b);
+  a -= __uint_as_float(hi << 16);
+  b -= __uint_as_float(hi & 0xffff0000u);
+  mid = pack_pair(a, b);
+  lo = pack_pair(a - __uint_as_float(mid << 16), b - __uint_as_float(mid & 0xffff0000u));
 }
 
 // One warp: dt and L of the chunk's tokens into s_dt [64] and s_L [64] (float64).
@@ -341,16 +408,18 @@ __device__ __forceinline__ void chunk_decays(const float* __restrict__ rows, int
 }
 
 // A tile [64 rows][width] of bfloat16 values from u's columns col.., zeros beyond row m and column `live`.  vec: 16-byte
-// pieces (every column and stride a multiple of 8 values).
+// pieces (every column and stride a multiple of 8 values), which are only asked for: see tiles_landed.
+__device__ __forceinline__ void tiles_landed() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 __device__ __forceinline__ void load_tile(__nv_bfloat16* dst, int ldd, int width, const __nv_bfloat16* __restrict__ u, int64_t ldu,
                                           int64_t row0, int m, int col, int live, bool vec) {
   if (vec) {
     const int w8 = width >> 3;
     for (int i = threadIdx.x; i < CH * w8; i += CH_NT) {
       const int r = i / w8, c = (i - r * w8) << 3;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (r < m && c < live) v = *reinterpret_cast<const uint4*>(u + (row0 + r) * ldu + col + c);
-      *reinterpret_cast<uint4*>(dst + r * ldd + c) = v;
+      const bool in = r < m && c < live;
+      const int bytes = in ? 16 : 0;                                    // none: the piece is filled with zeros
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(s_addr(dst + r * ldd + c)),
+                   "l"(in ? u + (row0 + r) * ldu + col + c : u), "r"(bytes) : "memory");
     }
   } else {
     for (int i = threadIdx.x; i < CH * width; i += CH_NT) {
@@ -360,8 +429,10 @@ __device__ __forceinline__ void load_tile(__nv_bfloat16* dst, int ldd, int width
   }
 }
 
+// FULL: every block has all of its 64 columns.
 // grid (chunks, H, tiles of 64 columns).  sums [chunks][H][N][P], ends [chunks][H].
-__global__ void __launch_bounds__(CH_NT) ssd_chunk_sum_kernel(
+template <bool FULL>
+__global__ void __launch_bounds__(CH_NT, 4) ssd_chunk_sum_kernel(
     float* __restrict__ sums, float* __restrict__ ends, const __nv_bfloat16* __restrict__ u, int64_t ldu,
     const float* __restrict__ rows, int64_t ld, int dt_off, const float* __restrict__ dt_bias, const float* __restrict__ A_log,
     const int* __restrict__ chunk_row, const int* __restrict__ chunk_len, int H, int P, int N, int G, int vec) {
@@ -379,9 +450,10 @@ __global__ void __launch_bounds__(CH_NT) ssd_chunk_sum_kernel(
   rb_pdl_wait();
   const int64_t row0 = chunk_row[chunk];
   const int m = chunk_len[chunk];
-  if (warp == 0) chunk_decays(rows, ld, dt_off + h, row0, m, a, dtb, s_L, s_dt, lane);
   load_tile(sB, LDB, NP, u, ldu, row0, m, inner + grp * N, N, vec != 0);
   load_tile(sX, LDX, CH_P, u, ldu, row0, m, h * P + p0, pw, vec != 0);
+  if (warp == 0) chunk_decays(rows, ld, dt_off + h, row0, m, a, dtb, s_L, s_dt, lane);
+  tiles_landed();
   __syncthreads();
   const double L_end = s_L[CH - 1];
   for (int i = threadIdx.x; i < CH * (CH_P / 2); i += CH_NT) {          // x in place: its owner reads it first
@@ -389,12 +461,11 @@ __global__ void __launch_bounds__(CH_NT) ssd_chunk_sum_kernel(
     __nv_bfloat16* at = sX + r * LDX + c;
     const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(at));
     const float w = s_dt[r] * expf((float)(L_end - s_L[r]));
-    float h0, m0, l0, h1, m1, l1;
-    split3(x.x * w, h0, m0, l0);
-    split3(x.y * w, h1, m1, l1);
-    *reinterpret_cast<uint32_t*>(at) = pack_pair(h0, h1);
-    *reinterpret_cast<uint32_t*>(at + CH * LDX) = pack_pair(m0, m1);
-    *reinterpret_cast<uint32_t*>(at + 2 * CH * LDX) = pack_pair(l0, l1);
+    uint32_t hi, mid, lo;
+    split3(x.x * w, x.y * w, hi, mid, lo);
+    *reinterpret_cast<uint32_t*>(at) = hi;
+    *reinterpret_cast<uint32_t*>(at + CH * LDX) = mid;
+    *reinterpret_cast<uint32_t*>(at + 2 * CH * LDX) = lo;
   }
   if (threadIdx.x == 0 && blockIdx.z == 0) ends[(int64_t)chunk * H + h] = expf((float)L_end);
   __syncthreads();
@@ -406,14 +477,14 @@ __global__ void __launch_bounds__(CH_NT) ssd_chunk_sum_kernel(
     for (int i = 0; i < CH_P / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
     for (int kk = 0; kk < CH / 16; ++kk) {
-      if (kk * 16 >= m) break;
+      if (!FULL && kk * 16 >= m) break;
       uint32_t A[4];
       ldsm4t(A, s_addr(sB + (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * LDB + nb + ((lane >> 3) & 1) * 8));
 #pragma unroll
       for (int part = 0; part < 3; ++part) {
 #pragma unroll
         for (int dn = 0; dn < CH_P / 8; dn += 2) {
-          if (dn * 8 >= pw) break;
+          if (!FULL && dn * 8 >= pw) break;
           uint32_t b[4];
           ldsm4t(b, s_addr(sX + part * CH * LDX + (kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDX + (dn + (lane >> 4)) * 8));
           mma_16816(acc[dn], A, b[0], b[1]);
@@ -441,19 +512,29 @@ __global__ void __launch_bounds__(CH_NT) ssd_chunk_sum_kernel(
   }
 }
 
-// grid (runs, H, pieces of a state), 128 threads, V values each: sums[chunk] <- the state the chunk starts from.
+// grid (runs, H, pieces of a state), 128 threads, V values each: sums[chunk] <- the state the chunk starts from; and
+// the ring of the convolution's last inputs is brought up to the run's end (tail [n_slots, K, C], null with one tap).
 template <int V>
 __global__ void __launch_bounds__(128) ssd_chunk_walk_kernel(float* __restrict__ sums, const float* __restrict__ ends,
                                                              float* __restrict__ state, const int* __restrict__ seq_first,
                                                              const int* __restrict__ seq_count,
                                                              const int* __restrict__ run_chunk0, const int* __restrict__ tok_slot,
-                                                             int H, int64_t NP_) {
+                                                             int H, int64_t NP_, float* __restrict__ tail,
+                                                             const float* __restrict__ rows, int64_t ld, int x_off,
+                                                             const int* __restrict__ tok_pos, int C, int K) {
   rb_pdl_launch_dependents();
   const int run = blockIdx.x, h = blockIdx.y;
   const int64_t e = ((int64_t)blockIdx.z * 128 + threadIdx.x) * V;
   rb_pdl_wait();
+  const int first = seq_first[run], n_tok = seq_count[run], n_chunks = (n_tok + CH - 1) / CH, chunk0 = run_chunk0[run];
+  if (K > 1) {
+    // the ring of the convolution's inputs moves on to the run's end (the convolution is done)
+    const int slot = tok_slot[first], last = first + n_tok - 1, pos = tok_pos[last];
+    for (int c = (h * gridDim.z + blockIdx.z) * 128 + threadIdx.x; c < C; c += H * gridDim.z * 128)
+      for (int back = 0; back < K - 1 && back < n_tok; ++back)
+        tail[((int64_t)slot * K + (pos - back) % K) * C + c] = rows[(int64_t)(last - back) * ld + x_off + c];
+  }
   if (e >= NP_) return;
-  const int first = seq_first[run], n_chunks = (seq_count[run] + CH - 1) / CH, chunk0 = run_chunk0[run];
   float* st = state + ((int64_t)tok_slot[first] * H + h) * NP_ + e;
   float S[V];
 #pragma unroll
@@ -492,7 +573,8 @@ __global__ void __launch_bounds__(128) ssd_chunk_walk_kernel(float* __restrict__
 }
 
 // grid (chunks, H, tiles of 64 columns).  starts: what the walk left.  out [T, H * P] = v (see the top of the file).
-__global__ void __launch_bounds__(CH_NT) ssd_chunk_out_kernel(
+template <bool FULL>
+__global__ void __launch_bounds__(CH_NT, 3) ssd_chunk_out_kernel(
     float* __restrict__ out, const float* __restrict__ starts, const __nv_bfloat16* __restrict__ u, int64_t ldu,
     const float* __restrict__ rows, int64_t ld, int z_off, int dt_off, const float* __restrict__ dt_bias,
     const float* __restrict__ A_log, const float* __restrict__ D_skip, const int* __restrict__ chunk_row,
@@ -505,7 +587,7 @@ __global__ void __launch_bounds__(CH_NT) ssd_chunk_out_kernel(
   __nv_bfloat16* sC = reinterpret_cast<__nv_bfloat16*>(s_dt + CH);      // [64][LDB]
   __nv_bfloat16* sB = sC + CH * LDB;                                    // [64][LDB]
   __nv_bfloat16* sX = sB + CH * LDB;                                    // [64][LDX]
-  __nv_bfloat16* sS = sX + CH * LDX;                                    // three of [NP][LDX]: the state in three terms
+  __nv_bfloat16* sS = sX + CH * LDX;                                    // three of [64][LDX]: 64 state rows in three terms
   const int chunk = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * CH_P, pw = min(CH_P, P - p0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
   const int inner = H * P, grp = h / (H / G);
@@ -513,67 +595,84 @@ __global__ void __launch_bounds__(CH_NT) ssd_chunk_out_kernel(
   rb_pdl_wait();
   const int64_t row0 = chunk_row[chunk];
   const int m = chunk_len[chunk];
-  if (warp == 0) chunk_decays(rows, ld, dt_off + h, row0, m, a, dtb, s_L, s_dt, lane);
+  const float* start = starts + ((int64_t)chunk * H + h) * N * P + p0;
+  // a thread's part of 64 state rows: four columns of every eighth row, fetched ahead
+  constexpr int HELD = SL * (CH_P / 4) / CH_NT;
+  const bool quads = P % 4 == 0;
+  const int sc = (threadIdx.x % (CH_P / 4)) * 4, sr = threadIdx.x / (CH_P / 4);
+  float4 held[HELD];
+  auto fetch = [&](int n0) {
+#pragma unroll
+    for (int i = 0; i < HELD; ++i) {
+      const int n = n0 + sr + i * (CH_NT / (CH_P / 4));
+      held[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (n < N && sc < pw) {
+        const float* src = start + (int64_t)n * P + sc;
+        if (quads) {
+          held[i] = *reinterpret_cast<const float4*>(src);
+        } else {
+          held[i].x = src[0];
+          if (sc + 1 < pw) held[i].y = src[1];
+          if (sc + 2 < pw) held[i].z = src[2];
+          if (sc + 3 < pw) held[i].w = src[3];
+        }
+      }
+    }
+  };
+  fetch(0);
   load_tile(sC, LDB, NP, u, ldu, row0, m, inner + G * N + grp * N, N, vec != 0);
   load_tile(sB, LDB, NP, u, ldu, row0, m, inner + grp * N, N, vec != 0);
   load_tile(sX, LDX, CH_P, u, ldu, row0, m, h * P + p0, pw, vec != 0);
-  const float* start = starts + ((int64_t)chunk * H + h) * N * P + p0;
-  const int part_elems = NP * LDX;
-  if (P % 4 == 0) {
-    for (int i = threadIdx.x; i < NP * (CH_P / 4); i += CH_NT) {
-      const int n = i / (CH_P / 4), c = (i % (CH_P / 4)) * 4;
-      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (n < N && c < pw) f = *reinterpret_cast<const float4*>(start + (int64_t)n * P + c);
-      float hi[4], mid[4], lo[4];
-      split3(f.x, hi[0], mid[0], lo[0]); split3(f.y, hi[1], mid[1], lo[1]);
-      split3(f.z, hi[2], mid[2], lo[2]); split3(f.w, hi[3], mid[3], lo[3]);
-      __nv_bfloat16* at = sS + n * LDX + c;
-      *reinterpret_cast<uint2*>(at) = make_uint2(pack_pair(hi[0], hi[1]), pack_pair(hi[2], hi[3]));
-      *reinterpret_cast<uint2*>(at + part_elems) = make_uint2(pack_pair(mid[0], mid[1]), pack_pair(mid[2], mid[3]));
-      *reinterpret_cast<uint2*>(at + 2 * part_elems) = make_uint2(pack_pair(lo[0], lo[1]), pack_pair(lo[2], lo[3]));
-    }
-  } else {
-    for (int i = threadIdx.x; i < NP * CH_P; i += CH_NT) {
-      const int n = i / CH_P, c = i % CH_P;
-      float hi, mid, lo;
-      split3(n < N && c < pw ? start[(int64_t)n * P + c] : 0.f, hi, mid, lo);
-      __nv_bfloat16* at = sS + n * LDX + c;
-      at[0] = __float2bfloat16_rn(hi);
-      at[part_elems] = __float2bfloat16_rn(mid);
-      at[2 * part_elems] = __float2bfloat16_rn(lo);
-    }
-  }
-  __syncthreads();
+  if (warp == 0) chunk_decays(rows, ld, dt_off + h, row0, m, a, dtb, s_L, s_dt, lane);
+  constexpr int part_elems = SL * LDX;
   const int rb = warp * 16;                                             // this warp's 16 tokens
-  if (rb >= m) return;
+  const bool active = rb < m;
   float acc[CH_P / 8][4], G_[CH / 8][4];
 #pragma unroll
   for (int i = 0; i < CH_P / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
   for (int i = 0; i < CH / 8; ++i) G_[i][0] = G_[i][1] = G_[i][2] = G_[i][3] = 0.f;
-  for (int kk = 0; kk < NP / 16; ++kk) {
-    uint32_t A[4];
-    ldsm4(A, s_addr(sC + (rb + (lane & 7) + ((lane >> 3) & 1) * 8) * LDB + kk * 16 + (lane >> 4) * 8));
+  for (int n0 = 0; n0 < NP; n0 += SL) {                                 // 64 state rows at a time
+    if (n0 > 0) __syncthreads();                                        // everybody has left the slice before
 #pragma unroll
-    for (int part = 0; part < 3; ++part) {                              // S0^T C
+    for (int i = 0; i < HELD; ++i) {
+      uint2 hi, mid, lo;
+      split3(held[i].x, held[i].y, hi.x, mid.x, lo.x);
+      split3(held[i].z, held[i].w, hi.y, mid.y, lo.y);
+      __nv_bfloat16* at = sS + (sr + i * (CH_NT / (CH_P / 4))) * LDX + sc;
+      *reinterpret_cast<uint2*>(at) = hi;
+      *reinterpret_cast<uint2*>(at + part_elems) = mid;
+      *reinterpret_cast<uint2*>(at + 2 * part_elems) = lo;
+    }
+    if (n0 == 0) tiles_landed();
+    __syncthreads();
+    if (n0 + SL < NP) fetch(n0 + SL);                                   // on its way while this slice is multiplied
+    if (!active) continue;
+    for (int kk = n0 / 16; kk < min(NP, n0 + SL) / 16; ++kk) {
+      uint32_t A[4];
+      ldsm4(A, s_addr(sC + (rb + (lane & 7) + ((lane >> 3) & 1) * 8) * LDB + kk * 16 + (lane >> 4) * 8));
 #pragma unroll
-      for (int dn = 0; dn < CH_P / 8; dn += 2) {
-        if (dn * 8 >= pw) break;
+      for (int part = 0; part < 3; ++part) {                            // S0^T C
+#pragma unroll
+        for (int dn = 0; dn < CH_P / 8; dn += 2) {
+          if (!FULL && dn * 8 >= pw) break;
+          uint32_t b[4];
+          ldsm4t(b, s_addr(sS + part * part_elems + (kk * 16 - n0 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDX + (dn + (lane >> 4)) * 8));
+          mma_16816(acc[dn], A, b[0], b[1]);
+          mma_16816(acc[dn + 1], A, b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < CH / 8; j += 2) {                             // C B^T, half of it where the rows are early
+        if (j == CH / 16 && rb < CH / 2) break;
         uint32_t b[4];
-        ldsm4t(b, s_addr(sS + part * part_elems + (kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDX + (dn + (lane >> 4)) * 8));
-        mma_16816(acc[dn], A, b[0], b[1]);
-        mma_16816(acc[dn + 1], A, b[2], b[3]);
+        ldsm4(b, s_addr(sB + (j * 8 + (lane >> 4) * 8 + (lane & 7)) * LDB + kk * 16 + ((lane >> 3) & 1) * 8));
+        mma_16816(G_[j], A, b[0], b[1]);
+        mma_16816(G_[j + 1], A, b[2], b[3]);
       }
     }
-#pragma unroll
-    for (int j = 0; j < CH / 8; j += 2) {                               // C B^T, up to the diagonal
-      if (j * 8 > rb + 15) break;
-      uint32_t b[4];
-      ldsm4(b, s_addr(sB + (j * 8 + (lane >> 4) * 8 + (lane & 7)) * LDB + kk * 16 + ((lane >> 3) & 1) * 8));
-      mma_16816(G_[j], A, b[0], b[1]);
-      mma_16816(G_[j + 1], A, b[2], b[3]);
-    }
   }
+  if (!active) return;
   const int i0 = rb + g, i1 = rb + g + 8;
   const double L0 = s_L[i0], L1 = s_L[i1];
   {
@@ -598,15 +697,12 @@ __global__ void __launch_bounds__(CH_NT) ssd_chunk_out_kernel(
       const float v01 = j + 1 <= i0 ? c[1] * d1 * expf((float)(L0 - Lj1)) : 0.f;
       const float v10 = j <= i1 ? c[2] * d0 * expf((float)(L1 - Lj0)) : 0.f;
       const float v11 = j + 1 <= i1 ? c[3] * d1 * expf((float)(L1 - Lj1)) : 0.f;
-      float h0, m0, l0, h1, m1, l1;
-      split3(v00, h0, m0, l0); split3(v01, h1, m1, l1);
-      Mp[0][2 * q] = pack_pair(h0, h1); Mp[1][2 * q] = pack_pair(m0, m1); Mp[2][2 * q] = pack_pair(l0, l1);
-      split3(v10, h0, m0, l0); split3(v11, h1, m1, l1);
-      Mp[0][2 * q + 1] = pack_pair(h0, h1); Mp[1][2 * q + 1] = pack_pair(m0, m1); Mp[2][2 * q + 1] = pack_pair(l0, l1);
+      split3(v00, v01, Mp[0][2 * q], Mp[1][2 * q], Mp[2][2 * q]);
+      split3(v10, v11, Mp[0][2 * q + 1], Mp[1][2 * q + 1], Mp[2][2 * q + 1]);
     }
 #pragma unroll
     for (int dn = 0; dn < CH_P / 8; dn += 2) {
-      if (dn * 8 >= pw) break;
+      if (!FULL && dn * 8 >= pw) break;
       uint32_t b[4];
       ldsm4t(b, s_addr(sX + (kt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDX + (dn + (lane >> 4)) * 8));
 #pragma unroll
@@ -626,7 +722,7 @@ __global__ void __launch_bounds__(CH_NT) ssd_chunk_out_kernel(
 #pragma unroll
     for (int dn = 0; dn < CH_P / 8; ++dn) {
       const int p = dn * 8 + t4 * 2;
-      if (p >= pw) break;
+      if (!FULL && p >= pw) break;
       const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + i * LDX + p));
       const float y0 = fmaf(skip, x.x, acc[dn][2 * half]), y1 = fmaf(skip, x.y, acc[dn][2 * half + 1]);
       if (pairs) {
@@ -646,7 +742,7 @@ inline int chunk_sum_smem(int N) {
 }
 inline int chunk_out_smem(int N) {
   const int NP = (N + 15) & ~15;
-  return CH * 12 + (2 * CH * (NP + 8) + CH * LDX + 3 * NP * LDX) * 2;
+  return CH * 12 + (2 * CH * (NP + 8) + CH * LDX + 3 * SL * LDX) * 2;
 }
 
 }  // namespace
@@ -694,9 +790,17 @@ RB_EXPORT int rb_ssd_step(float* out, const float* rows, int64_t ld, int z_off, 
   const dim3 grid(T, H, (P + cols - 1) / cols);
   const size_t smem = (size_t)(STEP_COLS + 2 * N + 4 * STEP_NT) * sizeof(float);
   RB_REQUIRE(smem <= 48 * 1024, "rb_ssd_step: a state of %d rows is more than a block's shared memory holds", N);
-#define GO(V) RB_LAUNCH("ssd_step_kernel", (ssd_step_kernel<V>), grid, STEP_NT, smem, stream, out, rows, ld, z_off, x_off, dt_off, taps, conv_bias, dt_bias, A_log, D_skip, state, tail, tok_slot, tok_pos, H, P, N, G, K, cols)
-  if (P % 4 == 0) GO(4);
-  else GO(1);
+#define GO(V, KT) RB_LAUNCH("ssd_step_kernel", (ssd_step_kernel<V, KT>), grid, STEP_NT, smem, stream, out, rows, ld, z_off, x_off, dt_off, taps, conv_bias, dt_bias, A_log, D_skip, state, tail, tok_slot, tok_pos, H, P, N, G, K, cols)
+#define PICK(V)                \
+  do {                         \
+    if (K == 2) GO(V, 2);      \
+    else if (K == 3) GO(V, 3); \
+    else if (K == 4) GO(V, 4); \
+    else GO(V, 0);             \
+  } while (0)
+  if (P % 4 == 0) PICK(4);
+  else PICK(1);
+#undef PICK
 #undef GO
   RB_CHECK_LAUNCH("rb_ssd_step");
   return 0;
@@ -737,36 +841,42 @@ RB_EXPORT long long rb_ssd_chunk_floats(int P, int N) { return (long long)P * N 
 
 // Runs of several tokens in chunks of 64.  chunk_row, chunk_len: every chunk of every run, the runs' chunks in order;
 // run_chunk0[r]: the first chunk of run r.  scratch: n_chunks * H * rb_ssd_chunk_floats(P, N) floats.
-RB_EXPORT int rb_ssd_chunked(float* out, const void* u, int64_t ldu, const float* rows, int64_t ld, int z_off, int dt_off,
-                             const float* dt_bias, const float* A_log, const float* D_skip, float* state, float* scratch,
-                             const int* seq_first, const int* seq_count, const int* run_chunk0, const int* chunk_row,
-                             const int* chunk_len, const int* tok_slot, int n_runs, int n_chunks, int H, int P, int N, int G,
-                             cudaStream_t stream) {
+// It also brings the ring of the convolution's last inputs (columns x_off .. of rows) up to the runs' ends.
+RB_EXPORT int rb_ssd_chunked(float* out, const void* u, int64_t ldu, const float* rows, int64_t ld, int z_off, int x_off, int dt_off,
+                             const float* dt_bias, const float* A_log, const float* D_skip, float* state, float* tail,
+                             float* scratch, const int* seq_first, const int* seq_count, const int* run_chunk0,
+                             const int* chunk_row, const int* chunk_len, const int* tok_slot, const int* tok_pos, int n_runs,
+                             int n_chunks, int H, int P, int N, int G, int K, cudaStream_t stream) {
   if (n_runs == 0 || n_chunks == 0) return 0;
-  RB_REQUIRE(H > 0 && H <= 65535 && G > 0 && H % G == 0 && rb_ssd_chunked_supports(P, N) && (uintptr_t)scratch % 16 == 0,
+  const int C = H * P + 2 * G * N;
+  RB_REQUIRE(H > 0 && H <= 65535 && G > 0 && H % G == 0 && rb_ssd_chunked_supports(P, N) && (uintptr_t)scratch % 16 == 0 &&
+                 (K == 1 || tail != nullptr),
              "rb_ssd_chunked: bad sizes H=%d P=%d N=%d G=%d", H, P, N, G);
+  const bool full = P % CH_P == 0;
   const int vec = P % 8 == 0 && N % 8 == 0 && ldu % 8 == 0 && (uintptr_t)u % 16 == 0;
   static RbOncePerDevice configured;
   if (configured.first()) {
-    RB_CUDA(cudaFuncSetAttribute(ssd_chunk_sum_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
-    RB_CUDA(cudaFuncSetAttribute(ssd_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
+    RB_CUDA(cudaFuncSetAttribute(ssd_chunk_sum_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
+    RB_CUDA(cudaFuncSetAttribute(ssd_chunk_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
+    RB_CUDA(cudaFuncSetAttribute(ssd_chunk_sum_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
+    RB_CUDA(cudaFuncSetAttribute(ssd_chunk_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
   }
   const int64_t NPv = (int64_t)N * P;
   float* sums = scratch;
   float* ends = scratch + (int64_t)n_chunks * H * NPv;
   const dim3 grid(n_chunks, H, (P + CH_P - 1) / CH_P);
   const __nv_bfloat16* ub = (const __nv_bfloat16*)u;
-  RB_LAUNCH("ssd_chunk_sum_kernel", (ssd_chunk_sum_kernel), grid, CH_NT, chunk_sum_smem(N), stream, sums, ends, ub, ldu, rows, ld, dt_off,
+  RB_LAUNCH("ssd_chunk_sum_kernel", (full ? ssd_chunk_sum_kernel<true> : ssd_chunk_sum_kernel<false>), grid, CH_NT, chunk_sum_smem(N), stream, sums, ends, ub, ldu, rows, ld, dt_off,
             dt_bias, A_log, chunk_row, chunk_len, H, P, N, G, vec);
   RB_CHECK_LAUNCH("rb_ssd_chunked");
   if (NPv % 4 == 0)
     RB_LAUNCH("ssd_chunk_walk_kernel", (ssd_chunk_walk_kernel<4>), dim3(n_runs, H, (NPv / 4 + 127) / 128), 128, 0, stream, sums, ends, state,
-              seq_first, seq_count, run_chunk0, tok_slot, H, NPv);
+              seq_first, seq_count, run_chunk0, tok_slot, H, NPv, tail, rows, ld, x_off, tok_pos, C, K);
   else
     RB_LAUNCH("ssd_chunk_walk_kernel", (ssd_chunk_walk_kernel<1>), dim3(n_runs, H, (NPv + 127) / 128), 128, 0, stream, sums, ends, state,
-              seq_first, seq_count, run_chunk0, tok_slot, H, NPv);
+              seq_first, seq_count, run_chunk0, tok_slot, H, NPv, tail, rows, ld, x_off, tok_pos, C, K);
   RB_CHECK_LAUNCH("rb_ssd_chunked");
-  RB_LAUNCH("ssd_chunk_out_kernel", (ssd_chunk_out_kernel), grid, CH_NT, chunk_out_smem(N), stream, out, sums, ub, ldu, rows, ld, z_off,
+  RB_LAUNCH("ssd_chunk_out_kernel", (full ? ssd_chunk_out_kernel<true> : ssd_chunk_out_kernel<false>), grid, CH_NT, chunk_out_smem(N), stream, out, sums, ub, ldu, rows, ld, z_off,
             dt_off, dt_bias, A_log, D_skip, chunk_row, chunk_len, H, P, N, G, vec);
   RB_CHECK_LAUNCH("rb_ssd_chunked");
   return 0;

@@ -297,12 +297,62 @@ inline int flat_blocks(int64_t n, int threads) {
   return (int)(want < most ? want : most);
 }
 
+// The same for parts of 256 values and more: a block per row and part, NV times four values a thread in registers.
+template <typename TO, int NV>
+__global__ void __launch_bounds__(256) rmsnorm_parts_kernel(TO* __restrict__ out, const float* __restrict__ x,
+                                                            const float* __restrict__ w, int E, int per, float eps) {
+  rb_pdl_launch_dependents();
+  __shared__ float scratch[33];
+  const int64_t at = (int64_t)blockIdx.x * E + (int64_t)blockIdx.y * per;
+  float v[NV][4], ww[NV][4];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int e = (i * blockDim.x + threadIdx.x) * 4;
+    if (e < per) rb_load4(w + blockIdx.y * per + e, ww[i]);
+  }
+  rb_pdl_wait();
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int e = (i * blockDim.x + threadIdx.x) * 4;
+    v[i][0] = v[i][1] = v[i][2] = v[i][3] = 0.f;
+    if (e < per) rb_load4(x + at + e, v[i]);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) ss = fmaf(v[i][k], v[i][k], ss);
+  }
+  ss = rb_block_sum(ss, scratch);
+  const float r = 1.0f / sqrtf(ss / (float)per + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int e = (i * blockDim.x + threadIdx.x) * 4;
+    if (e < per) {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[i][k] = v[i][k] * r * ww[i][k];
+      rb_store4(out + at + e, v[i]);
+    }
+  }
+}
+
 }  // namespace
 
 RB_EXPORT int rb_rmsnorm_grouped(void* out, int out_dtype, const float* x, const float* w, int T, int E, int groups,
                                  float eps, cudaStream_t stream) {
   if (T == 0) return 0;
   RB_REQUIRE(groups >= 1 && E > 0 && E % groups == 0, "rb_rmsnorm_grouped: a row of %d values is not %d equal parts", E, groups);
+  {
+    const int per = E / groups, n4 = per / 4;
+    if (per % 4 == 0 && per >= 256 && n4 <= 4 * 256 && groups <= 65535 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+        (uintptr_t)out % 16 == 0) {
+      const int nv = n4 <= 256 ? 1 : (n4 <= 512 ? 2 : 4), nt = ((n4 + nv - 1) / nv + 31) / 32 * 32;
+#define GO(TT, N) RB_LAUNCH("rmsnorm_parts_kernel", (rmsnorm_parts_kernel<TT, N>), dim3(T, groups), nt, 0, stream, (TT*)out, x, w, E, per, eps)
+      if (out_dtype == RB_F32) { if (nv == 1) GO(float, 1); else if (nv == 2) GO(float, 2); else GO(float, 4); }
+      else if (out_dtype == RB_BF16) { if (nv == 1) GO(__nv_bfloat16, 1); else if (nv == 2) GO(__nv_bfloat16, 2); else GO(__nv_bfloat16, 4); }
+      else RB_FAIL("rb_rmsnorm_grouped: unknown dtype %d", out_dtype);
+#undef GO
+      RB_CHECK_LAUNCH("rb_rmsnorm_grouped");
+      return 0;
+    }
+  }
   const int threads = groups >= 8 ? 256 : 32 * groups;
   const int vec = (E / groups) % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0;
   if (out_dtype == RB_F32)

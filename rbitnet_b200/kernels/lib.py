@@ -96,7 +96,7 @@ _SIGNATURES = {
     "rb_ssd_conv": [P, I, L, P, L, I, P, P, P, P, P, P, I, I, I, P],
     "rb_ssd_step": [P, P, L, I, I, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
     "rb_ssd_scan": [P, P, I, L, P, L, I, I, P, P, P, P, P, P, P, I, I, I, I, I, P],
-    "rb_ssd_chunked": [P, P, L, P, L, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
+    "rb_ssd_chunked": [P, P, L, P, L, I, I, I, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
     "rb_ssd_chunked_supports": [I, I],
     "rb_round_rows": [P, I, P, L, P],
     "rb_norm_add_norm": [P, P, P, F, I, I, I, P, I, P, F, P],

@@ -1131,18 +1131,18 @@ class CudaOps:
         self.lib.call("rb_ssd_conv", _ptr(u), self.code, u.stride(0), _ptr(proj), proj.stride(0), at["x"], _ptr(p.conv_w),
                       _ptr(p.conv_b), _ptr(tail), _ptr(tok_first), _ptr(meta.tok_slot), _ptr(meta.tok_pos), T, C, K,
                       self._stream())
-        if K > 1:
-            self.lib.call("rb_conv_tail_update", _ptr(tail), _ptr(proj), proj.stride(0), at["x"], F32, c_void_p(0), _ptr(first),
-                          _ptr(count), _ptr(meta.tok_slot), _ptr(meta.tok_pos), n_runs, C, K, self._stream())
         if self.dtype == torch.bfloat16 and self.ssd_in_chunks and self.lib.raw("rb_ssd_chunked_supports")(P, N):
             run_chunk0, chunk_row, chunk_len, n_chunks = self._delta_chunks(meta, 64)
             scratch = torch.empty((n_chunks * H * self.lib.raw("rb_ssd_chunk_floats")(P, N),), dtype=torch.float32,
                                   device=self.device)
-            self.lib.call("rb_ssd_chunked", _ptr(out), _ptr(u), u.stride(0), _ptr(proj), proj.stride(0), at["z"], at["dt"],
-                          _ptr(p.dt_bias), _ptr(p.a_log), _ptr(p.d_skip), _ptr(state["S"]), _ptr(scratch), _ptr(first), _ptr(count),
-                          _ptr(run_chunk0), _ptr(chunk_row), _ptr(chunk_len), _ptr(meta.tok_slot), n_runs, n_chunks, H, P, N, G,
-                          self._stream(), launches=3)
+            self.lib.call("rb_ssd_chunked", _ptr(out), _ptr(u), u.stride(0), _ptr(proj), proj.stride(0), at["z"], at["x"], at["dt"],
+                          _ptr(p.dt_bias), _ptr(p.a_log), _ptr(p.d_skip), _ptr(state["S"]), _ptr(tail), _ptr(scratch), _ptr(first),
+                          _ptr(count), _ptr(run_chunk0), _ptr(chunk_row), _ptr(chunk_len), _ptr(meta.tok_slot),
+                          _ptr(meta.tok_pos), n_runs, n_chunks, H, P, N, G, K, self._stream(), launches=3)
         else:
+            if K > 1:
+                self.lib.call("rb_conv_tail_update", _ptr(tail), _ptr(proj), proj.stride(0), at["x"], F32, c_void_p(0), _ptr(first),
+                              _ptr(count), _ptr(meta.tok_slot), _ptr(meta.tok_pos), n_runs, C, K, self._stream())
             self.lib.call("rb_ssd_scan", _ptr(out), _ptr(u), self.code, u.stride(0), _ptr(proj), proj.stride(0), at["z"], at["dt"],
                           _ptr(p.dt_bias), _ptr(p.a_log), _ptr(p.d_skip), _ptr(state["S"]), _ptr(first), _ptr(count),
                           _ptr(meta.tok_slot), n_runs, H, P, N, G, self._stream())

@@ -107,7 +107,8 @@ def attention(h, m, w):
     T, H, G, D = h.shape[0], m["heads"], m["kv_heads"], m["dim"]
     q = (h @ w["q"].T + w["q.b"]).view(T, H, D)
     k = (h @ w["k"].T + w["k.b"]).view(T, G, D)
-    o = softmax_attention(rotate(q, m["rot"]), rotate(k, m["rot"]), k, float(m["scale"]), visible(T, m.get("mask")))
+    turned = [rotate(x, m["rot"]) if m.get("rot") else x for x in (q, k)]
+    o = softmax_attention(*turned, k, float(m["scale"]), visible(T, m.get("mask")))
     return o.reshape(T, -1) @ w["o"].T + w["o.b"]
 
 
