@@ -20,6 +20,10 @@ namespace {
 
 __device__ __forceinline__ float ssd_softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 __device__ __forceinline__ float ssd_silu(float v) { return v / (1.0f + expf(-v)); }
+// The same two with the hardware's exponential and reciprocal, for the chunked kernels (error a few units of float32, far
+// below that of the bfloat16 channels they work on).
+__device__ __forceinline__ float ssd_exp_fast(float v) { return __expf(v); }
+__device__ __forceinline__ float ssd_silu_fast(float v) { return __fdividef(v, 1.0f + __expf(-v)); }
 
 // ---------------------------------------------------------------- short convolution and SiLU
 // u[t, c] = silu(bias[c] + sum_d taps[c, K-1-d] x_(t-d)[c]), zeros before a sequence's start, rows before a run from the
@@ -86,7 +90,7 @@ __global__ void __launch_bounds__(128) ssd_conv_kernel(TO* __restrict__ u, int64
       float acc = b[i];
 #pragma unroll
       for (int d = 0; d < K; ++d) acc = fmaf(w[d][i], hist[d][i], acc);
-      y[i] = ssd_silu(acc);
+      y[i] = sizeof(TO) == 2 ? ssd_silu_fast(acc) : ssd_silu(acc);
     }
     TO* dst = u + (int64_t)t * ldu + c;
     if (V == 4) {
@@ -357,6 +361,7 @@ __global__ void __launch_bounds__(SCAN_NT) ssd_scan_kernel(
 constexpr int CH = 64;                  // tokens of a chunk
 constexpr int CH_NT = 128;              // four warps of 16 rows
 constexpr int CH_P = 64;                // value columns of a block
+constexpr int LDZ = CH_P + 8;           // row stride of the tile of z (float32)
 constexpr int SL = 64;                  // state rows that the output kernel holds at a time
 constexpr int LDX = CH_P + 8;           // row stride of tiles of columns: ldmatrix rows in different banks
 
@@ -460,7 +465,7 @@ __global__ void __launch_bounds__(CH_NT, 4) ssd_chunk_sum_kernel(
     const int r = i / (CH_P / 2), c = (i % (CH_P / 2)) * 2;
     __nv_bfloat16* at = sX + r * LDX + c;
     const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(at));
-    const float w = s_dt[r] * expf((float)(L_end - s_L[r]));
+    const float w = s_dt[r] * ssd_exp_fast((float)(L_end - s_L[r]));
     uint32_t hi, mid, lo;
     split3(x.x * w, x.y * w, hi, mid, lo);
     *reinterpret_cast<uint32_t*>(at) = hi;
@@ -672,7 +677,18 @@ __global__ void __launch_bounds__(CH_NT, 3) ssd_chunk_out_kernel(
       }
     }
   }
-  if (!active) return;
+  // z comes into the state's place while the chunk's own tokens are multiplied
+  float* sZ = reinterpret_cast<float*>(sS);                             // [64][LDZ]
+  const bool staged = FULL && vec != 0 && ld % 4 == 0 && z_off % 4 == 0;
+  if (staged) {
+    __syncthreads();                                                    // everybody has left the last slice
+    for (int i = threadIdx.x; i < CH * (CH_P / 4); i += CH_NT) {
+      const int r = i / (CH_P / 4), c = (i % (CH_P / 4)) * 4;
+      if (r < m)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s_addr(sZ + r * LDZ + c)),
+                     "l"(rows + (row0 + r) * ld + z_off + h * P + p0 + c) : "memory");
+    }
+  }
   const int i0 = rb + g, i1 = rb + g + 8;
   const double L0 = s_L[i0], L1 = s_L[i1];
   {
@@ -685,7 +701,7 @@ __global__ void __launch_bounds__(CH_NT, 3) ssd_chunk_out_kernel(
   }
 #pragma unroll
   for (int kt = 0; kt < CH / 16; ++kt) {                                // 16 earlier tokens at a time
-    if (kt * 16 > rb + 15) break;
+    if (kt * 16 > rb + 15 || !active) break;
     uint32_t Mp[3][4];
 #pragma unroll
     for (int q = 0; q < 2; ++q) {
@@ -693,10 +709,10 @@ __global__ void __launch_bounds__(CH_NT, 3) ssd_chunk_out_kernel(
       const double Lj0 = s_L[j], Lj1 = s_L[j + 1];
       const float d0 = s_dt[j], d1 = s_dt[j + 1];
       const float* c = G_[2 * kt + q];
-      const float v00 = j <= i0 ? c[0] * d0 * expf((float)(L0 - Lj0)) : 0.f;
-      const float v01 = j + 1 <= i0 ? c[1] * d1 * expf((float)(L0 - Lj1)) : 0.f;
-      const float v10 = j <= i1 ? c[2] * d0 * expf((float)(L1 - Lj0)) : 0.f;
-      const float v11 = j + 1 <= i1 ? c[3] * d1 * expf((float)(L1 - Lj1)) : 0.f;
+      const float v00 = j <= i0 ? c[0] * d0 * ssd_exp_fast((float)(L0 - Lj0)) : 0.f;
+      const float v01 = j + 1 <= i0 ? c[1] * d1 * ssd_exp_fast((float)(L0 - Lj1)) : 0.f;
+      const float v10 = j <= i1 ? c[2] * d0 * ssd_exp_fast((float)(L1 - Lj0)) : 0.f;
+      const float v11 = j + 1 <= i1 ? c[3] * d1 * ssd_exp_fast((float)(L1 - Lj1)) : 0.f;
       split3(v00, v01, Mp[0][2 * q], Mp[1][2 * q], Mp[2][2 * q]);
       split3(v10, v11, Mp[0][2 * q + 1], Mp[1][2 * q + 1], Mp[2][2 * q + 1]);
     }
@@ -712,6 +728,11 @@ __global__ void __launch_bounds__(CH_NT, 3) ssd_chunk_out_kernel(
       }
     }
   }
+  if (staged) {
+    tiles_landed();
+    __syncthreads();
+  }
+  if (!active) return;
   const bool pairs = P % 2 == 0 && ld % 2 == 0 && z_off % 2 == 0;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
@@ -726,11 +747,11 @@ __global__ void __launch_bounds__(CH_NT, 3) ssd_chunk_out_kernel(
       const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + i * LDX + p));
       const float y0 = fmaf(skip, x.x, acc[dn][2 * half]), y1 = fmaf(skip, x.y, acc[dn][2 * half + 1]);
       if (pairs) {
-        const float2 zz = *reinterpret_cast<const float2*>(z + p);
-        *reinterpret_cast<float2*>(dst + p) = make_float2(y0 * ssd_silu(zz.x), y1 * ssd_silu(zz.y));
+        const float2 zz = staged ? *reinterpret_cast<const float2*>(sZ + i * LDZ + p) : *reinterpret_cast<const float2*>(z + p);
+        *reinterpret_cast<float2*>(dst + p) = make_float2(y0 * ssd_silu_fast(zz.x), y1 * ssd_silu_fast(zz.y));
       } else {
-        dst[p] = y0 * ssd_silu(z[p]);
-        if (p + 1 < pw) dst[p + 1] = y1 * ssd_silu(z[p + 1]);
+        dst[p] = y0 * ssd_silu_fast(z[p]);
+        if (p + 1 < pw) dst[p + 1] = y1 * ssd_silu_fast(z[p + 1]);
       }
     }
   }
