@@ -341,7 +341,8 @@ RB_EXPORT int rb_rmsnorm_grouped(void* out, int out_dtype, const float* x, const
   RB_REQUIRE(groups >= 1 && E > 0 && E % groups == 0, "rb_rmsnorm_grouped: a row of %d values is not %d equal parts", E, groups);
   {
     const int per = E / groups, n4 = per / 4;
-    if (per % 4 == 0 && per >= 256 && n4 <= 4 * 256 && groups <= 65535 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+    // (with many rows and several parts a warp per part is faster)
+    if (per % 4 == 0 && per >= 256 && (groups < 4 || T <= 64) && n4 <= 4 * 256 && groups <= 65535 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
         (uintptr_t)out % 16 == 0) {
       const int nv = n4 <= 256 ? 1 : (n4 <= 512 ? 2 : 4), nt = ((n4 + nv - 1) / nv + 31) / 32 * 32;
 #define GO(TT, N) RB_LAUNCH("rmsnorm_parts_kernel", (rmsnorm_parts_kernel<TT, N>), dim3(T, groups), nt, 0, stream, (TT*)out, x, w, E, per, eps)

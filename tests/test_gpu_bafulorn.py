@@ -305,8 +305,6 @@ def test_attention_with_kept_first_positions(H, Kh, D, shared, window, keep):
             "prompts": [(300, 300), (400, 37), (64, 64), (193, 2), (128, 1)], "long prompt": [(700, 500)]}
     for dtype in (torch.float32, torch.bfloat16):
         ops = _ops(dtype)
-        if dtype == torch.float32 and not (H <= 8 and not shared):
-            continue                                                   # the float32 kernel knows no sharing
         for what, seqs in runs.items():
             need = CacheNeed(Kh, D, None, streams=((Kh, D),) if shared else None)
             cache = SequenceCache({0: need}, {}, {}, 64 * 40, 1024, dtype, ops.device)
