@@ -89,7 +89,8 @@ template <int D> __device__ __forceinline__ uint32_t tile_off(int row, int col) 
   return (uint32_t)((col >> 6) * (TILE * 128) + row * 128 + (((((col & 63) >> 3) ^ (row & 7))) << 4) + (col & 7) * 2);
 }
 
-template <int D, int NS>
+// KEEP: with a window, the first p.keep keys stay visible (a kernel of its own, so that the others do not pay for it).
+template <int D, int NS, bool KEEP>
 __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK,
                                                                       const __grid_constant__ CUtensorMap tmV, Params p) {
   rb_pdl_launch_dependents();
@@ -110,8 +111,10 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
   const int slot = p.tok_slot[tok0];
   const int pos0 = p.tok_pos[tok0];
   const int key_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-  const RbKeyTiles tiles(key_lo, pos0, p.keep, TILE);
-  int kt_begin = 0, kt_end = tiles.n;         // numbers of the visited tiles, see RbKeyTiles
+  // with kept keys kt counts the visited tiles (see RbKeyTiles), else it is a tile's own number
+  const RbKeyTiles tiles(key_lo, pos0, KEEP ? p.keep : 0, TILE);
+  auto tile_of = [&](int kt) { return KEEP ? tiles.at(kt) : kt; };
+  int kt_begin = KEEP ? 0 : tiles.first, kt_end = kt_begin + tiles.n;
   if (p.n_splits > 1) {
     // the tiles are dealt evenly: part z takes [z*n/parts, (z+1)*n/parts), sizes that differ by at most one
     const int n = kt_end - kt_begin, z = blockIdx.z;
@@ -127,7 +130,7 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
 
   // one thread asks for a tile: keys and values of 64 positions of this kv head, D/64 boxes each
   auto request = [&](int i, int buf) {
-    const int key0 = tiles.at(i) * TILE;
+    const int key0 = tile_of(i) * TILE;
     const int page = p.page_table[(int64_t)slot * p.max_pages + key0 / p.page_size];
     const int row = (page * p.n_kv_heads + kvh) * p.page_size + key0 % p.page_size;
     mbar_expect_tx(&full[buf], 2 * S::TILE_BYTES);
@@ -143,7 +146,7 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
   int n_early = 0;                     // tiles requested before the wait (thread 0's count)
   if (threadIdx.x == 0) {
     for (int i = 0; i < NS - 1; ++i)
-      if (kt_begin + i < kt_end && tiles.at(kt_begin + i) != newest && n_early == i) {
+      if (kt_begin + i < kt_end && tile_of(kt_begin + i) != newest && n_early == i) {
         request(kt_begin + i, i);
         n_early = i + 1;
       }
@@ -190,7 +193,7 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
     if (!failed && !mbar_wait(&full[buf], (uint32_t)((i / NS) & 1), 14)) failed = true;
     const uint32_t tK = smem_u32(smem + S::OFF_K + buf * S::TILE_BYTES);
     const uint32_t tV = smem_u32(smem + S::OFF_V + buf * S::TILE_BYTES);
-    const int key_base = tiles.at(kt) * TILE + kw0;
+    const int key_base = tile_of(kt) * TILE + kw0;
     if (key_base <= pos0) {
       // ---- S = Q K^T: two accumulators per 8-key tile, over even and odd steps of d, so that the
       // chain of dependent products is half as long
@@ -214,7 +217,7 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
         for (int c = 0; c < 4; ++c) {
           const int h = c >> 1;
           const int key = key_base + n * 8 + t4 * 2 + (c & 1);
-          const bool ok = row_ok[h] && key <= pos0 && (key >= key_lo || key < p.keep);
+          const bool ok = row_ok[h] && key <= pos0 && (key >= key_lo || (KEEP && key < p.keep));
           const float sc = s[n][c] + s2[n][c];
           const float v = !ok ? -INFINITY : (p.softcap > 0.f ? cap_log2 * tanhf(sc * scale_over_cap) : sc * p.scale_log2);
           s[n][c] = v;
@@ -364,9 +367,9 @@ __global__ void __launch_bounds__(WARPS_D * 32) attn_decode_tma_kernel(const __g
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
-template <int D, int NS>
+template <int D, int NS, bool KEEP>
 int launch_ns(const CUtensorMap& tk, const CUtensorMap& tv, const Params& p, int B, int Kh, cudaStream_t stream) {
-  auto kernel = attn_decode_tma_kernel<D, NS>;
+  auto kernel = attn_decode_tma_kernel<D, NS, KEEP>;
   constexpr int smem = Smem<D, NS>::BYTES;
   static RbOncePerDevice configured;
   if (configured.first()) {
@@ -415,7 +418,7 @@ inline bool cluster_of_16_runs() {
   static int answer = -1;
   if (answer < 0) {
     answer = 0;
-    auto kernel = attn_decode_tma_kernel<128, 3>;
+    auto kernel = attn_decode_tma_kernel<128, 3, false>;
     constexpr int smem = Smem<128, 3>::BYTES;
     if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) == cudaSuccess &&
         cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess) {
@@ -442,8 +445,8 @@ template <int D>
 int launch(const CUtensorMap& tk, const CUtensorMap& tv, const Params& p, int B, int Kh, cudaStream_t stream) {
   // the deeper ring when the whole grid runs at once with it, or when the shallower one holds no more CTAs
   if ((long long)B * Kh * p.n_splits <= places(D, 3) || places(D, 2) <= places(D, 3))
-    return launch_ns<D, 3>(tk, tv, p, B, Kh, stream);
-  return launch_ns<D, 2>(tk, tv, p, B, Kh, stream);
+    return p.keep > 0 ? launch_ns<D, 3, true>(tk, tv, p, B, Kh, stream) : launch_ns<D, 3, false>(tk, tv, p, B, Kh, stream);
+  return p.keep > 0 ? launch_ns<D, 2, true>(tk, tv, p, B, Kh, stream) : launch_ns<D, 2, false>(tk, tv, p, B, Kh, stream);
 }
 
 }  // namespace decode_tma

@@ -137,7 +137,8 @@ struct TcSmem {
   static_assert(BYTES <= 227 * 1024, "shared memory");
 };
 
-template <int D, bool SHARED>
+// KEEP: with a window, the first p.keep keys stay visible (a kernel of its own, so that the others do not pay for it).
+template <int D, bool SHARED, bool KEEP>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, TcAttnParams p) {
   using S = TcSmem<D, SHARED>;
@@ -195,8 +196,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   const int n_rows = ntok * G;
   const int key_hi = pos0 + ntok - 1;
   const int key_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-  const RbKeyTiles tiles(key_lo, key_hi, p.keep, TILE_KEYS);
-  int kt_begin = 0, kt_end = tiles.n;                      // numbers of the visited tiles, see RbKeyTiles
+  // with kept keys kt counts the visited tiles (see RbKeyTiles), else it is a tile's own number
+  const RbKeyTiles tiles(key_lo, key_hi, KEEP ? p.keep : 0, TILE_KEYS);
+  auto tile_of = [&](int kt) { return KEEP ? tiles.at(kt) : kt; };
+  int kt_begin = KEEP ? 0 : tiles.first, kt_end = kt_begin + tiles.n;
   if (p.n_splits > 1) {                                    // this CTA's range of the key tiles (it may be empty)
     const int per = (kt_end - kt_begin + p.n_splits - 1) / p.n_splits;
     kt_begin += (int)blockIdx.z * per;
@@ -260,7 +263,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         int row[TILE_KEYS / PIECE];
 #pragma unroll
         for (int h = 0; h < TILE_KEYS / PIECE; ++h) {      // a tile is two pieces of 64 positions
-          const int key0 = tiles.at(kt) * TILE_KEYS + h * PIECE;
+          const int key0 = tile_of(kt) * TILE_KEYS + h * PIECE;
           const int pi = min(key0 / p.page_size, p.max_pages - 1);       // past the sequence: any page, masked later
           const int page = p.page_table[(int64_t)slot * p.max_pages + pi];
           row[h] = (page * p.n_kv_heads + kvh) * p.page_size + key0 % p.page_size;
@@ -387,11 +390,11 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
           sv[c] = fmaf(-2.0f * cap_b, rc, cap_b);
         }
       }
-      const int key0 = tiles.at(kt) * TILE_KEYS, key_base = key0 + half * HK;
+      const int key0 = tile_of(kt) * TILE_KEYS, key_base = key0 + half * HK;
       // a tile that every row of the CTA sees whole needs no mask (all tiles but those on the
       // diagonal, at the window's edge and at the end of the first keys that stay visible)
       const bool whole = key0 + TILE_KEYS - 1 <= pos0 &&
-                         (p.window <= 0 || key0 >= max(0, key_hi - p.window + 1) || key0 + TILE_KEYS <= p.keep);
+                         (p.window <= 0 || key0 >= max(0, key_hi - p.window + 1) || (KEEP && key0 + TILE_KEYS <= p.keep));
       float m_half;
       if (whole) {
         float t0 = sv[0], t1 = sv[1], t2 = sv[2], t3 = sv[3];          // four chains of three-input maxima
@@ -407,8 +410,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
 #pragma unroll
         for (int c = 0; c < HK; c += 2) {
           const int key = key_base + c;
-          sv[c] = (row_ok && key <= row_pos && (key >= row_lo || key < p.keep)) ? sv[c] : -INFINITY;
-          sv[c + 1] = (row_ok && key + 1 <= row_pos && (key + 1 >= row_lo || key + 1 < p.keep)) ? sv[c + 1] : -INFINITY;
+          sv[c] = (row_ok && key <= row_pos && (key >= row_lo || (KEEP && key < p.keep))) ? sv[c] : -INFINITY;
+          sv[c + 1] = (row_ok && key + 1 <= row_pos && (key + 1 >= row_lo || (KEEP && key + 1 < p.keep))) ? sv[c + 1] : -INFINITY;
           t0 = fmaxf(t0, sv[c]); t1 = fmaxf(t1, sv[c + 1]);
         }
         m_half = fmaxf(t0, t1) * p.scale_log2;
@@ -542,9 +545,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   }
 }
 
-template <int D, bool SHARED>
-int launch_tc(const CUtensorMap& tk, const CUtensorMap& tv, const TcAttnParams& p, int Kh, cudaStream_t stream) {
-  auto kernel = attn_tc_kernel<D, SHARED>;
+template <int D, bool SHARED, bool KEEP>
+int launch_tc_keep(const CUtensorMap& tk, const CUtensorMap& tv, const TcAttnParams& p, int Kh, cudaStream_t stream) {
+  auto kernel = attn_tc_kernel<D, SHARED, KEEP>;
   constexpr int smem = TcSmem<D, SHARED>::BYTES;
   static RbOncePerDevice configured;
   if (configured.first()) {
@@ -552,6 +555,10 @@ int launch_tc(const CUtensorMap& tk, const CUtensorMap& tv, const TcAttnParams& 
   }
   RB_LAUNCH("rb_attention_prefill_tc", (kernel), dim3(Kh, p.n_tiles, p.n_splits), THREADS, smem, stream, tk, tv, p);
   return 0;
+}
+template <int D, bool SHARED>
+int launch_tc(const CUtensorMap& tk, const CUtensorMap& tv, const TcAttnParams& p, int Kh, cudaStream_t stream) {
+  return p.keep > 0 ? launch_tc_keep<D, SHARED, true>(tk, tv, p, Kh, stream) : launch_tc_keep<D, SHARED, false>(tk, tv, p, Kh, stream);
 }
 
 }  // namespace

@@ -142,9 +142,11 @@ __device__ __forceinline__ float stored_value(const GemmParams& p, float v) {
 // The gated epilogue's value, with the hardware's exponential and reciprocal: their error (a few units of
 // float32) is far below the rounding to bfloat16 that follows.
 __device__ __forceinline__ float gated_value(const GemmParams& p, float g, float up) {
-  // gelu_tanh(g) = g/2 (1 + tanh(s)) = g / (1 + e^(-2 s)), s = sqrt(2/pi) (g + 0.044715 g^3)
-  if (p.act_kind == 1) return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * g * (1.0f + 0.044715f * g * g))) * up;
-  if (p.act_kind == 2) return fmaxf(g, 0.f) * up;
+  if (p.act_kind != 0) {
+    if (p.act_kind == 2) return fmaxf(g, 0.f) * up;
+    // gelu_tanh(g) = g/2 (1 + tanh(s)) = g / (1 + e^(-2 s)), s = sqrt(2/pi) (g + 0.044715 g^3)
+    return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * g * (1.0f + 0.044715f * g * g))) * up;
+  }
   if (p.act_limit > 0.f) {
     g = fminf(g, p.act_limit);
     up = fminf(fmaxf(up, -p.act_limit), p.act_limit);
