@@ -185,7 +185,7 @@ def one_key_stands_out(make_engine, tol, kind, n, far, window, keep, seen, cuts,
 
 #: (length, far position, window, kept positions, whether the last position sees it): keys far away, at page borders, just
 #: inside and just outside a window, the last kept position and the one after it
-KEYS = [(300, 299 - 95, 96, 0, True), (300, 299 - 96, 96, 0, False), (200, 199 - 63, 64, 0, True), (200, 199 - 64, 64, 0, False),
+KEYS = [(300, 299 - 90, 91, 0, True), (300, 299 - 91, 91, 0, False), (200, 199 - 63, 64, 0, True), (200, 199 - 64, 64, 0, False),
         (260, 128, 132, 0, True), (260, 127, 132, 0, False), (300, 2, None, 0, True), (700, 63, None, 0, True)]
 KEPT_KEYS = [(300, 9, 50, 10, True), (300, 10, 50, 10, False), (300, 0, 50, 1, True), (300, 1, 50, 1, False), (200, 63, 20, 64, True),
              (200, 64, 20, 64, False), (330, 69, 64, 70, True), (330, 70, 64, 70, False), (190, 130, 60, 7, True), (190, 129, 60, 7, False),
